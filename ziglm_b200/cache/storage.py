@@ -11,11 +11,12 @@ and narrows only the read range for windowed layers (src/model.zig:661).
 
 Beside the pages lies fixed-size state per sequence: for a place in the schedule
 that asks for it, a tensor [n_slots, *shape] that is zeroed when a slot is handed
-out.  This architecture asks for none; a mixer with a recurrent state would.
+out (a tuple of such tensors for a place that asks for several).  The Llama
+architecture asks for none; a mixer with a recurrent state does.
 """
 from __future__ import annotations
 
-from typing import Dict, List, Optional, Sequence, Tuple
+from typing import Dict, List, Optional, Sequence, Tuple, Union
 
 import torch
 
@@ -46,7 +47,7 @@ class CacheStorage:
     """All groups, the slot table above them, and the per-sequence state."""
 
     def __init__(self, kv_needs: Sequence[Optional[KVNeed]], reads_from: Sequence[Optional[int]],
-                 state_needs: Sequence[Optional[StateNeed]], max_tokens: int, n_slots: int, max_len: int,
+                 state_needs: Sequence[Union[StateNeed, Tuple[StateNeed, ...], None]], max_tokens: int, n_slots: int, max_len: int,
                  dtype: torch.dtype, device: torch.device, page_size: int = PAGE_SIZE,
                  window_pool_tokens: Optional[int] = None):
         """kv_needs[s], state_needs[s]: what place s of the schedule keeps.  reads_from[s]: the place
@@ -77,16 +78,21 @@ class CacheStorage:
         self.slots = SlotTable(n_slots, [g.pages for g in self.groups], max_len)
         for g in self.groups:
             g.pages.mirror(n_slots, self.max_pages_per_seq)
-        self.states: Dict[int, torch.Tensor] = {}
+        self.states: Dict[int, Union[torch.Tensor, Tuple[torch.Tensor, ...]]] = {}
+
+        def zeros(need: StateNeed) -> torch.Tensor:
+            return torch.zeros((n_slots,) + tuple(need.shape), dtype=need.dtype, device=device)
+
         for s, need in enumerate(state_needs):
             if need is not None:
-                self.states[s] = torch.zeros((n_slots,) + tuple(need.shape), dtype=need.dtype, device=device)
+                self.states[s] = tuple(zeros(n) for n in need) if isinstance(need, tuple) else zeros(need)
 
     # ------------------------------------------------------------------ slots
     def alloc_slot(self) -> int:
         slot = self.slots.alloc()
-        for st in self.states.values():
-            st[slot].zero_()
+        for held in self.states.values():
+            for st in held if isinstance(held, tuple) else (held,):
+                st[slot].zero_()
         return slot
 
     def free_slot(self, slot: int) -> None:

@@ -18,6 +18,7 @@ from .tumatar import TumatarConfig
 from .tikalix import TikalixConfig
 from .vilazen import VilazenConfig
 from .lipadra import LipadraConfig
+from .mopilorn import MopilornConfig
 from .spec import ModelSpec
 
 _ARCHITECTURES: Dict[str, Any] = {}
@@ -70,3 +71,4 @@ register_architecture(TumatarConfig.ARCHITECTURE, TumatarConfig)
 register_architecture(TikalixConfig.ARCHITECTURE, TikalixConfig)
 register_architecture(VilazenConfig.ARCHITECTURE, VilazenConfig)
 register_architecture(LipadraConfig.ARCHITECTURE, LipadraConfig)
+register_architecture(MopilornConfig.ARCHITECTURE, MopilornConfig)

@@ -116,8 +116,15 @@ class ModelSpec:
     # added at the start of every pass through a repeated run of layers, say)
     place_hooks: Mapping[int, HookSpec] = field(default_factory=dict)
     options: Mapping[str, Any] = field(default_factory=dict)
+    # copies of the residual a token is carried by (hyper-connections): every block then works on rows of
+    # streams * width, all copies equal to the embedding at first, and their sum is what the final norm reads
+    streams: int = 1
 
     def __post_init__(self) -> None:
+        if self.streams < 1:
+            raise ValueError(f"a token needs at least one residual stream, found {self.streams}")
+        if self.streams > 1 and (self.embed_hook is not None or self.place_hooks):
+            raise ValueError("hooks on the residual are not combined with several residual streams")
         for i in self.schedule:
             if not 0 <= i < len(self.layers):
                 raise ValueError(f"schedule names layer {i}, but there are {len(self.layers)} layers")

@@ -607,6 +607,14 @@ __global__ void scale_kernel(float* __restrict__ x, long n, float factor) {
     if (i < n) x[i] *= factor;
 }
 
+// x <- cap tanh(x / cap)
+__global__ void soft_cap_kernel(float* __restrict__ x, long n, float cap) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) x[i] = cap * tanhf(x[i] / cap);
+}
+
 // y += x (float), used by parts that cannot fold their residual sum into a product
 __global__ void add_kernel(float* __restrict__ y, const float* __restrict__ x, long n) {
     const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -1014,6 +1022,13 @@ ZLM_EXPORT int zlm_add_row(float* x, const void* table_row, int dtype, int T, in
 ZLM_EXPORT int zlm_scale(float* x, long n, float factor, cudaStream_t stream) {
     if (n <= 0) return 0;
     cudaError_t e = launch_pdl(scale_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, x, n, factor);
+    return e == cudaSuccess ? launch_status() : (int)e;
+}
+
+ZLM_EXPORT int zlm_soft_cap(float* x, long n, float cap, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (!(cap > 0.f)) return ZLM_ERR_BAD_ARG;
+    cudaError_t e = launch_pdl(soft_cap_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, x, n, cap);
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 

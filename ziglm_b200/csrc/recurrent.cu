@@ -104,6 +104,68 @@ __global__ void conv_vec_kernel(const __nv_bfloat16* __restrict__ x, long x_stri
     *reinterpret_cast<uint4*>(u + (long)t * C + c) = o;
 }
 
+// A causal convolution a channel that keeps its own inputs: ring float [slots][K][C], row p mod K the inputs of
+// position p.  y_t = act(sum_j taps[K-1-j] x_(t-j)), zeros before the start of the sequence.
+// grid (channels, tiles of `tile` tokens, sequences).  A thread takes W channels for a tile's tokens; only a sequence's
+// first tile (tile >= K - 1) reads the ring, and it writes the ring when it has read it: the step's last inputs are
+// rows of x.
+template <typename T, int W>
+__global__ void __launch_bounds__(128)
+conv_ring_kernel(const T* __restrict__ x, long x_stride, const float* __restrict__ taps, float* __restrict__ ring_all,
+                 const int* __restrict__ slots, const int* __restrict__ past_lens, const int* __restrict__ cu_seqlens,
+                 T* __restrict__ y, long y_stride, int C, int K, int act, int tile) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int b = blockIdx.z;
+    const int first = cu_seqlens[b], n_new = cu_seqlens[b + 1] - first;
+    const int lo = blockIdx.y * tile, hi = min(n_new, lo + tile);
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * W;
+    if (lo >= n_new || c >= C) return;
+    const int past = past_lens[b];
+    float* ring = ring_all + (long)slots[b] * K * C + c;
+    auto load = [&](const T* p, float (&f)[W]) {
+        if constexpr (W == 1) f[0] = to_float(*p);
+        else if constexpr (sizeof(T) == 4) {
+            const float4 v = *reinterpret_cast<const float4*>(p);
+            f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+        } else {
+            const uint2 raw = *reinterpret_cast<const uint2*>(p);
+            const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+            const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+            f[0] = u.x; f[1] = u.y; f[2] = v.x; f[3] = v.y;
+        }
+    };
+    for (int i = lo; i < hi; ++i) {
+        const T* xr = x + (long)(first + i) * x_stride + c;
+        float acc[W];
+#pragma unroll
+        for (int e = 0; e < W; ++e) acc[e] = 0.f;
+        for (int j = K - 1; j >= 0; --j) {                // oldest input first
+            float xv[W];
+            if (i - j >= 0) load(xr - (long)j * x_stride, xv);
+            else {
+                const int p = past + i - j;
+#pragma unroll
+                for (int e = 0; e < W; ++e) xv[e] = p >= 0 ? ring[(long)(p % K) * C + e] : 0.f;
+            }
+            const float* w = taps + (long)(K - 1 - j) * C + c;
+#pragma unroll
+            for (int e = 0; e < W; ++e) acc[e] = fmaf(w[e], xv[e], acc[e]);
+        }
+        T* yr = y + (long)(first + i) * y_stride + c;
+#pragma unroll
+        for (int e = 0; e < W; ++e) yr[e] = from_float<T>(act == 1 ? silu_f(round_to<T>(acc[e])) : acc[e]);
+    }
+    if (lo != 0) return;
+    for (int j = min(K, n_new) - 1; j >= 0; --j) {
+        const int i = n_new - 1 - j;
+        float xv[W];
+        load(x + (long)(first + i) * x_stride + c, xv);
+#pragma unroll
+        for (int e = 0; e < W; ++e) ring[(long)((past + i) % K) * C + e] = xv[e];
+    }
+}
+
 // grid (sequences, ceil(C / channels a block takes)), block (channels: 32 or 16, chunks)
 template <typename T>
 __global__ void __launch_bounds__(RC_MAX_THREADS)
@@ -369,6 +431,31 @@ ZLM_EXPORT int zlm_causal_conv(const void* x, int dtype, long x_stride, const fl
                        act);
     else
         return ZLM_ERR_UNSUPPORTED;
+    return e == cudaSuccess ? launch_status() : (int)e;
+}
+
+// The convolution with a ring: x rows with stride x_stride, taps float [K, C] (the current token's row last), ring float
+// [slots, K, C], y rows with stride y_stride (may not be x); act: 0 none, 1 silu; max_new: the most tokens a sequence
+// brings.
+ZLM_EXPORT int zlm_causal_conv_ring(const void* x, int dtype, long x_stride, const float* taps, float* ring,
+                                    const int* slots, const int* past_lens, const int* cu_seqlens, void* y, long y_stride,
+                                    int n_seqs, int max_new, int C, int K, int act, cudaStream_t stream) {
+    if (n_seqs <= 0 || max_new <= 0) return 0;
+    if (C <= 0 || K <= 0 || x == y) return ZLM_ERR_BAD_ARG;
+    const int tile = K - 1 > 8 ? K - 1 : 8;
+    const int tiles = (max_new + tile - 1) / tile;
+    if (tiles > 65535 || n_seqs > 65535) return ZLM_ERR_UNSUPPORTED;
+    const bool wide = C % 4 == 0 && x_stride % 4 == 0 && y_stride % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0;
+    const int per_block = 128 * (wide ? 4 : 1);
+    dim3 grid((C + per_block - 1) / per_block, tiles, n_seqs);
+    cudaError_t e;
+#define ZLM_CRING(TT, WW)                                                                                              \
+    e = launch_pdl(conv_ring_kernel<TT, WW>, grid, dim3(128), 0, stream, (const TT*)x, x_stride, taps, ring, slots, past_lens, \
+                   cu_seqlens, (TT*)y, y_stride, C, K, act, tile)
+    if (dtype == ZLM_F32) { if (wide) ZLM_CRING(float, 4); else ZLM_CRING(float, 1); }
+    else if (dtype == ZLM_BF16) { if (wide) ZLM_CRING(__nv_bfloat16, 4); else ZLM_CRING(__nv_bfloat16, 1); }
+    else return ZLM_ERR_UNSUPPORTED;
+#undef ZLM_CRING
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 

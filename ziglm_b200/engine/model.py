@@ -83,7 +83,7 @@ class Model:
                            for local in hook_class(hook_spec.kind).declare(hook_spec)})
 
     def kernel_libraries(self) -> Tuple[str, ...]:
-        libs = ("elementwise",) + self.final_norm.kernel_libraries()
+        libs = ("elementwise",) + (("streams",) if self.spec.streams > 1 else ()) + self.final_norm.kernel_libraries()
         for b in self.blocks:
             libs += b.kernel_libraries()
         if self.head is not None:
@@ -119,8 +119,11 @@ class Model:
     def forward(self, step: StepContext) -> Optional[torch.Tensor]:
         """Run the step's tokens through the layers; float32 logits [n_want, vocab] or None."""
         spec = self.spec
-        x = step.ws.buf("residual", (step.n_tokens, spec.width), torch.float32)
-        kernels.embed(self.embedding, step.tokens, x, spec.embedding_scale)
+        x = step.ws.buf("residual", (step.n_tokens, spec.streams * spec.width), torch.float32)
+        if spec.streams > 1:
+            kernels.embed_streams(self.embedding, step.tokens, x, spec.streams, spec.embedding_scale)
+        else:
+            kernels.embed(self.embedding, step.tokens, x, spec.embedding_scale)
         if self.embed_hook is not None:
             self.embed_hook.forward(step, x)
         carried = None           # the next block's first norm, half done by the block before (steps of few tokens)

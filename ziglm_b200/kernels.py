@@ -71,6 +71,7 @@ _PROTOTYPES = {
         "zlm_head_norm_gate": [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int,
                                c_float, c_int, c_float, c_void_p],
         "zlm_scale": [c_void_p, c_long, c_float, c_void_p],
+        "zlm_soft_cap": [c_void_p, c_long, c_float, c_void_p],
         "zlm_add": [c_void_p, c_void_p, c_long, c_void_p],
         "zlm_convert": [c_void_p, c_int, c_void_p, c_int, c_long, c_void_p],
         "zlm_fill_normal": [c_void_p, c_int, c_long, ctypes.c_ulonglong, c_float, c_float, c_void_p],
@@ -82,11 +83,29 @@ _PROTOTYPES = {
     "recurrent": {
         "zlm_causal_conv": [c_void_p, c_int, c_long, c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p,
                             c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+        "zlm_causal_conv_ring": [c_void_p, c_int, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_long,
+                                 c_int, c_int, c_int, c_int, c_int, c_void_p],
         "zlm_selective_scan": [c_void_p, c_int, c_void_p, c_void_p, c_long, c_int, c_int, c_void_p, c_long, c_void_p, c_long,
                                c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                c_int, c_int, c_void_p],
         "zlm_gated_scan": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_long, c_void_p, c_long, c_void_p, c_float,
                            c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    },
+    "streams": {
+        "zlm_stream_norm": [c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+        "zlm_stream_mix": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p,
+                           c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
+        "zlm_embed_streams": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
+    },
+    "delta_rule": {
+        "zlm_delta_prep": [c_void_p, c_int, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_long,
+                           c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                           c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+        "zlm_delta_scan": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_long,
+                           c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "zlm_delta_decode": [c_void_p, c_int, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_long,
+                             c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                             c_float, c_void_p, c_long, c_int, c_void_p, c_long, c_void_p],
     },
     "linear_attention": {
         "zlm_linear_attention_chunk": [],
@@ -470,6 +489,81 @@ def scale_(x: torch.Tensor, factor: float) -> None:
     _check(_fn("elementwise", "zlm_scale")(x.data_ptr(), x.numel(), float(factor), _stream()), "scale_")
 
 
+def soft_cap_(x: torch.Tensor, cap: float) -> None:
+    """x <- cap * tanh(x / cap), float32, in place."""
+    _cuda(x, "x", torch.float32)
+    _check(_fn("elementwise", "zlm_soft_cap")(x.data_ptr(), x.numel(), float(cap), _stream()), "soft_cap_")
+
+
+# -------------------------------------------------------------- residual streams
+def embed_streams(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, streams: int, scale: float = 1.0) -> None:
+    """out[t] = ``streams`` copies, one behind the other, of float(table[tokens[t], :]) * scale; out float32 [T, streams * d]."""
+    _cuda(table, "table"); _cuda(tokens, "tokens", torch.int32); _cuda(out, "out", torch.float32)
+    T, width = out.shape
+    d = table.shape[1]
+    if width != streams * d or tokens.numel() < T:
+        raise KernelError("embed_streams: shapes do not match")
+    _check(_fn("streams", "zlm_embed_streams")(table.data_ptr(), code(table.dtype), tokens.data_ptr(), out.data_ptr(), T,
+                                               streams, d, scale, _stream()), "embed_streams")
+
+
+def stream_norm(x: torch.Tensor, streams: int, gather: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
+                out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+    """out[r] = norm(u) * weight with u = sum_a gather[a] * x[rows[r] or r, stream a] and norm(u) = u / sqrt(mean(u^2) + eps).
+    x float32 [n, streams * d]; gather float32 [streams], None: every stream counts once; weight float32 [d]."""
+    _cuda(x, "x", torch.float32); _cuda(weight, "weight", torch.float32); _cuda(out, "out")
+    n, d = out.shape
+    if x.shape[1] != streams * d or weight.numel() != d or (rows is None and x.shape[0] < n):
+        raise KernelError("stream_norm: shapes do not match")
+    if gather is not None:
+        _cuda(gather, "gather", torch.float32)
+        if gather.numel() != streams:
+            raise KernelError("stream_norm: one number is needed for each stream")
+    if rows is not None:
+        _cuda(rows, "rows", torch.int32)
+        if rows.numel() < n:
+            raise KernelError("stream_norm: fewer row indices than output rows")
+    _check(_fn("streams", "zlm_stream_norm")(x.data_ptr(), _ptr(gather), streams, weight.data_ptr(), float(eps), _ptr(rows),
+                                             out.data_ptr(), code(out.dtype), n, d, _stream()), "stream_norm")
+
+
+def stream_mix(x: torch.Tensor, streams: int, coef: torch.Tensor, branches, norm_weights=None, norm_eps: float = 0.0,
+               factor: float = 1.0, nxt=None) -> None:
+    """New streams in place: x[t, b] <- sum_a mix[a, b] x[t, a] + out[b] y[t], all at once from the old ones.  ``coef``
+    float32 [streams^2 + streams]: mix row by row ([from, to]), then out.  ``branches``: one float32 [T, d] tensor, y, or
+    two, and then y = factor * sum_i norm(branch_i) * norm_weights[i] with ``norm_eps``.  ``nxt`` = (gather, weight, eps,
+    h): also the rows h [T, d] that ``stream_norm`` would make of the new streams."""
+    _cuda(x, "x", torch.float32); _cuda(coef, "coef", torch.float32)
+    T = x.shape[0]
+    d = x.shape[1] // streams
+    if x.shape[1] != streams * d or coef.numel() != streams * streams + streams or len(branches) not in (1, 2):
+        raise KernelError("stream_mix: shapes do not match")
+    for b in branches:
+        _cuda(b, "branch", torch.float32)
+        if b.shape != (T, d):
+            raise KernelError("stream_mix: a branch must be [T, d]")
+    b2 = w1 = w2 = None
+    if len(branches) == 2:
+        if norm_weights is None or len(norm_weights) != 2:
+            raise KernelError("stream_mix: two branches are normed, each with a weight")
+        w1, w2 = norm_weights
+        _cuda(w1, "w1", torch.float32); _cuda(w2, "w2", torch.float32)
+        if w1.numel() != d or w2.numel() != d:
+            raise KernelError("stream_mix: a branch's weight must hold d numbers")
+        b2 = branches[1]
+    gather = weight = h = None
+    eps = 0.0
+    if nxt is not None:
+        gather, weight, eps, h = nxt
+        _cuda(gather, "gather", torch.float32); _cuda(weight, "weight", torch.float32); _cuda(h, "h")
+        if gather.numel() != streams or weight.numel() != d or h.shape != (T, d):
+            raise KernelError("stream_mix: the next sublayer's rows do not match")
+    _check(_fn("streams", "zlm_stream_mix")(
+        x.data_ptr(), coef.data_ptr(), streams, branches[0].data_ptr(), _ptr(w1), _ptr(b2), _ptr(w2), float(norm_eps),
+        float(factor), _ptr(gather), _ptr(weight), float(eps), _ptr(h), code(h.dtype) if h is not None else F32, T, d,
+        _stream()), "stream_mix")
+
+
 # ---------------------------------------------------------- block-diagonal product
 BLOCK_EPILOGUES = {None: 0, "sigmoid": 1, "sigmoid_gate": 2}
 
@@ -527,6 +621,111 @@ def causal_conv(x: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, state: 
         x.data_ptr(), code(x.dtype), _row_stride(x), taps.data_ptr(), bias.data_ptr(), state.data_ptr(), state.stride(0),
         step.seq_of_token.data_ptr(), step.cu_seqlens.data_ptr(), step.slots.data_ptr(), u.data_ptr(), T, C, K,
         1 if activation == "silu" else 0, _stream()), "causal_conv")
+
+
+def causal_conv_ring(x: torch.Tensor, taps: torch.Tensor, ring: torch.Tensor, step, y: torch.Tensor,
+                     activation: Optional[str] = None) -> None:
+    """y[t, c] = act(sum_j taps[K-1-j, c] * x[t-j, c]) over each sequence of the step, zeros before its start.  The inputs
+    before the step are in the sequence's ``ring`` [slots, K, C] (float32; row p mod K: position p), which the kernel also
+    brings up to date.  taps float32 [K, C] (the current token's row last); x and y may be column slices."""
+    _rows(x, "x"); _rows(y, "y"); _cuda(taps, "taps", torch.float32); _cuda(ring, "ring", torch.float32)
+    T, C = x.shape
+    K = taps.shape[0]
+    if taps.shape != (K, C) or y.shape != (T, C) or y.dtype != x.dtype or tuple(ring.shape[1:]) != (K, C):
+        raise KernelError("causal_conv_ring: shapes or types do not match")
+    if activation not in (None, "silu"):
+        raise KernelError(f"causal_conv_ring: activation {activation!r} is not known (silu)")
+    _check(_fn("recurrent", "zlm_causal_conv_ring")(
+        x.data_ptr(), code(x.dtype), _row_stride(x), taps.data_ptr(), ring.data_ptr(), step.slots.data_ptr(),
+        step.past_lens.data_ptr(), step.cu_seqlens.data_ptr(), y.data_ptr(), _row_stride(y), step.n_seqs, step.max_new, C, K,
+        1 if activation == "silu" else 0, _stream()), "causal_conv_ring")
+
+
+# -------------------------------------------------------------------- delta rule
+def delta_state_size(dim: int) -> int:
+    """Elements a value column of the delta rule's state holds: the key size as a multiple of four."""
+    return -(-dim // 4) * 4
+
+
+def _delta_args(proj, taps, ring, n_heads, n_kv, dim, value_dim, a, b, rate, dt_bias):
+    """Checks what the delta rule's kernels have in common; (taps a channel, whether the decay is one a key channel)."""
+    _rows(proj, "proj"); _rows(a, "a"); _rows(b, "b")
+    for t, n in ((taps, "taps"), (ring, "ring"), (rate, "rate"), (dt_bias, "dt_bias")):
+        _cuda(t, n, torch.float32)
+    C = 2 * n_kv * dim + n_heads * value_dim
+    T, K = proj.shape[0], taps.shape[0]
+    per_channel = dt_bias.numel() == n_heads * dim and a.shape[1] == n_heads * dim
+    if not per_channel and (dt_bias.numel() != n_heads or a.shape[1] != n_heads):
+        raise KernelError("delta rule: the decays are one a head or one a key channel")
+    if (n_heads <= 0 or n_kv <= 0 or n_heads % n_kv or proj.shape[1] < C or taps.shape != (K, C)
+            or tuple(ring.shape[1:]) != (K, C) or a.shape[0] != T or b.shape != (T, n_heads) or rate.numel() != n_heads
+            or a.dtype != torch.float32 or b.dtype != torch.float32):
+        raise KernelError("delta rule: shapes or types do not match")
+    return K, per_channel
+
+
+def _delta_state(state, n_heads, dim, value_dim):
+    _cuda(state, "state", torch.float32)
+    if tuple(state.shape[1:]) != (n_heads, value_dim, delta_state_size(dim)):
+        raise KernelError("delta rule: the state must be [slots, heads, value_dim, key size as a multiple of four]")
+
+
+def delta_rule(proj: torch.Tensor, taps: torch.Tensor, ring: torch.Tensor, n_heads: int, n_kv: int, dim: int,
+               value_dim: int, a: torch.Tensor, b: torch.Tensor, rate: torch.Tensor, dt_bias: torch.Tensor,
+               state: torch.Tensor, step, out: torch.Tensor) -> None:
+    """The gated delta rule over the step's sequences: with q | k | v the first 2 n_kv dim + n_heads value_dim columns of
+    ``proj`` behind a causal convolution a channel (``taps`` float32 [K, C], inputs kept in ``ring`` [slots, K, C]) and silu,
+    q and k divided by sqrt(sum of their squares + 1e-6) per head, q times dim^-1/2, beta = sigmoid(b),
+    g = exp(-rate softplus(a + dt_bias)) (one a head, or one a key channel when a and dt_bias hold n_heads * dim numbers):
+        S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  out = S^T q
+    Head h uses q/k head h // (n_heads // n_kv).  a, b float32 rows; out float32 [T, n_heads * value_dim]; state float32
+    [slots, n_heads, value_dim, ceil4(dim)]."""
+    K, per_channel = _delta_args(proj, taps, ring, n_heads, n_kv, dim, value_dim, a, b, rate, dt_bias)
+    _delta_state(state, n_heads, dim, value_dim)
+    _rows(out, "out")
+    T = proj.shape[0]
+    if out.dtype != torch.float32 or out.shape != (T, n_heads * value_dim):
+        raise KernelError("delta_rule: out must be float32 [T, heads * value_dim]")
+    dp, vp = delta_state_size(dim), delta_state_size(value_dim)
+    qk = step.ws.buf("delta_qk", (T, 2 * n_kv, dp), torch.float32)
+    v = step.ws.buf("delta_v", (T, n_heads, vp), torch.float32)
+    g = step.ws.buf("delta_g", (T, n_heads, dp if per_channel else 1), torch.float32)
+    beta = step.ws.buf("delta_beta", (T, n_heads), torch.float32)
+    _check(_fn("delta_rule", "zlm_delta_prep")(
+        proj.data_ptr(), code(proj.dtype), _row_stride(proj), taps.data_ptr(), ring.data_ptr(), n_heads, n_kv, dim, value_dim,
+        K, a.data_ptr(), _row_stride(a), int(per_channel), b.data_ptr(), _row_stride(b), rate.data_ptr(), dt_bias.data_ptr(),
+        step.slots.data_ptr(), step.past_lens.data_ptr(), step.cu_seqlens.data_ptr(), step.n_seqs, step.max_new,
+        qk.data_ptr(), v.data_ptr(), g.data_ptr(), beta.data_ptr(), _stream()), "delta_prep")
+    _check(_fn("delta_rule", "zlm_delta_scan")(
+        qk.data_ptr(), v.data_ptr(), g.data_ptr(), int(per_channel), beta.data_ptr(), state.data_ptr(), step.slots.data_ptr(),
+        step.cu_seqlens.data_ptr(), out.data_ptr(), _row_stride(out), step.n_seqs, n_heads, n_kv, dim, value_dim, _stream()),
+        "delta_scan")
+
+
+def delta_rule_decode(proj: torch.Tensor, taps: torch.Tensor, ring: torch.Tensor, n_heads: int, n_kv: int, dim: int,
+                      value_dim: int, a: torch.Tensor, b: torch.Tensor, rate: torch.Tensor, dt_bias: torch.Tensor,
+                      state: torch.Tensor, step, norm_weight: torch.Tensor, eps: float, gate: Optional[torch.Tensor],
+                      gate_kind: Optional[str], out: torch.Tensor) -> None:
+    """``delta_rule`` for a step of one token a sequence, with what stands behind it in the same kernel: every head's output
+    divided by its root mean square (``eps``), times ``norm_weight`` (float32 [value_dim], shared by the heads), times
+    act(gate) (proj's type, [T, n_heads * value_dim]; "sigmoid" or "silu"), into out's rows (proj's type)."""
+    K, per_channel = _delta_args(proj, taps, ring, n_heads, n_kv, dim, value_dim, a, b, rate, dt_bias)
+    _delta_state(state, n_heads, dim, value_dim)
+    _rows(out, "out"); _cuda(norm_weight, "norm_weight", torch.float32)
+    T = proj.shape[0]
+    if (T != step.n_seqs or out.dtype != proj.dtype or out.shape != (T, n_heads * value_dim)
+            or norm_weight.numel() != value_dim or gate_kind not in HEAD_GATES or (gate is None) != (gate_kind is None)):
+        raise KernelError("delta_rule_decode: one row a sequence, out of proj's type, a weight of one head's length")
+    if gate is not None:
+        _rows(gate, "gate")
+        if gate.dtype != proj.dtype or gate.shape != out.shape:
+            raise KernelError("delta_rule_decode: the gate must have out's type and shape")
+    _check(_fn("delta_rule", "zlm_delta_decode")(
+        proj.data_ptr(), code(proj.dtype), _row_stride(proj), taps.data_ptr(), ring.data_ptr(), n_heads, n_kv, dim, value_dim,
+        K, a.data_ptr(), _row_stride(a), int(per_channel), b.data_ptr(), _row_stride(b), rate.data_ptr(), dt_bias.data_ptr(),
+        step.slots.data_ptr(), step.past_lens.data_ptr(), step.n_seqs, state.data_ptr(), norm_weight.data_ptr(), float(eps),
+        _ptr(gate), _row_stride(gate) if gate is not None else 0, HEAD_GATES[gate_kind], out.data_ptr(), _row_stride(out),
+        _stream()), "delta_rule_decode")
 
 
 def selective_scan(u: torch.Tensor, dt_pre: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, n_states: int,

@@ -12,9 +12,9 @@ PositionEncoding``rotary_table() -> (inv_freq, rotary_dim) | None`` for encoding
                 that are a rotation by position (fused into the cache write), and
                 ``apply(step, qkv, n_heads, n_kv_heads, head_dim)`` for any other.
 Mixer           ``cache_needs() -> KVNeed | None``, ``state_needs() -> StateNeed |
-                None``, ``forward(step, io, h, residual)``: adds its output to the
-                float32 ``residual`` in place.  ``io`` is the storage of the place
-                in the schedule that is running (:class:`LayerIO`).
+                tuple of them | None``, ``forward(step, io, h, residual)``: adds its
+                output to the float32 ``residual`` in place.  ``io`` is the storage of
+                the place in the schedule that is running (:class:`LayerIO`).
 FeedForward     ``forward(step, h, residual)``: adds its output to ``residual``.
 Block           ``forward(step, io, x)``: runs its parts on the residual stream x.
 Hook            ``forward(step, x)``: changes x in place; x is the float32 residual
@@ -40,6 +40,11 @@ from dataclasses import dataclass
 from typing import Any, Callable, Dict, Optional, Tuple
 
 import torch
+
+
+class FreeDim(int):
+    """A dimension of a declared tensor that the file gives and config.json does not (the inner size of a product of
+    low rank): the loader takes any size from 1 on; the number itself is what random weights are made with."""
 
 
 @dataclass(frozen=True)
@@ -68,7 +73,8 @@ class KVNeed:
 
 @dataclass(frozen=True)
 class StateNeed:
-    """Fixed-size state a mixer wants kept per sequence (zero when the sequence starts)."""
+    """Fixed-size state a mixer wants kept per sequence (zero when the sequence starts).  A mixer that keeps several
+    (a convolution's last inputs beside a matrix) asks for a tuple of these and finds a tuple of tensors."""
     shape: Tuple[int, ...]
     dtype: torch.dtype = torch.float32
 
@@ -81,7 +87,7 @@ class LayerIO:
     block_table: Optional[torch.Tensor] = None  # int32 [B, stride], rows in batch order
     page_size: int = 0
     writes_cache: bool = True
-    state: Optional[torch.Tensor] = None        # [n_slots, *shape]; index with step.slots
+    state: Any = None        # [n_slots, *shape], index with step.slots; a tuple of them where the mixer asked for several
 
 
 @dataclass

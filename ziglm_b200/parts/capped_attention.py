@@ -2,6 +2,8 @@
 
 For the rows h the mixer reads, H query heads, G key/value heads, query/key size D and value size V:
     q = W_q h + b_q,  k = W_k h + b_k,  v = W_v h + b_v
+    q, k, v <- conv(q), conv(k), conv(v)        a causal convolution a channel over the last taps tokens  (``conv``: taps;
+                                                no bias, zeros before the start; the inputs are a state of the sequence)
     q, k <- q / rms(q) * w_q, k / rms(k) * w_k  q (all heads as one vector) and k likewise  (``qk_norm`` "whole")
     q, k <- rotate(q, k; position)              the first ``rotary_dim`` dimensions of a head, in the pairs of the
                                                 position encoding; cosines and sines times its amplitude
@@ -95,6 +97,9 @@ class CappedAttention(Part):
             raise ValueError(f"capped_attention: sink {o.get('sink')!r} is not known (true, \"zero\")")
         self.has_sink = bool(o.get("sink"))
         self.sink_learned = o.get("sink") is True
+        self.conv = int(o.get("conv") or 0)
+        if self.conv < 0:
+            raise ValueError(f"capped_attention: a convolution of {self.conv} taps")
         self.value_mix = o.get("value_mix")
         if self.value_mix not in (None, "first", "mix"):
             raise ValueError(f"capped_attention: value_mix {self.value_mix!r} is not known (first, mix)")
@@ -108,6 +113,7 @@ class CappedAttention(Part):
                                                    else -(-self.n_heads // 8) * 8)
         self.proj: Optional[Linear] = None      # [q; k; v; g] with every head padded to ``kept``
         self.o: Optional[Linear] = None
+        self.conv_w: Optional[torch.Tensor] = None      # [taps, channels of q, k and v as they are held]
         self.q_norm_w: Optional[torch.Tensor] = None
         self.k_norm_w: Optional[torch.Tensor] = None
         self.sinks: Optional[torch.Tensor] = None
@@ -143,6 +149,9 @@ class CappedAttention(Part):
         if o.get("qk_norm_eps") is not None and o.get("qk_norm") == "head_first":
             p["q_norm.weight"] = ParamDecl((D,), init="ones")
             p["k_norm.weight"] = ParamDecl((D,), init="ones")
+        if o.get("conv"):
+            K = int(o["conv"])
+            p.update({"q.conv": ParamDecl((H * D, K)), "k.conv": ParamDecl((G * D, K)), "v.conv": ParamDecl((G * V, K))})
         if o.get("sink") is True:
             p["sink"] = ParamDecl((H,))
         if o.get("value_mix") is not None:
@@ -178,6 +187,10 @@ class CappedAttention(Part):
         if V != P:
             w_o = _pad_heads(w_o.t().contiguous(), H, V, P).t().contiguous()
         self.o = Linear(w_o)
+        if self.conv:
+            # a channel keeps its taps where it goes: padded and reordered like the rows of the projections
+            self.conv_w = torch.cat([_pad_heads(_order_heads(tensors[f"{n}.conv"].float(), heads, size, ordr), heads, size, P)
+                                     for n, heads, size, ordr in parts], dim=0).t().contiguous()
         if self.norm_kind == "whole":
             self.q_norm_w = _pad_heads(_order_heads(tensors["q_norm.weight"].float(), H, D, order), H, D, P).contiguous()
             self.k_norm_w = _pad_heads(_order_heads(tensors["k_norm.weight"].float(), G, D, order), G, D, P).contiguous()
@@ -191,7 +204,7 @@ class CappedAttention(Part):
             self.mix = float(tensors["vmix"].float().item())
 
     def kernel_libraries(self) -> Tuple[str, ...]:
-        libs = ("attention", "elementwise")
+        libs = ("attention", "elementwise") + (("recurrent",) if self.conv else ())
         libs += kernels.fast_attention_libraries(self.dtype, self.kept, self.n_heads, self.n_kv, softcap=self.softcap,
                                                  keep_first=self.keep_first, sinks=self.has_sink)
         for lin in (self.proj, self.o):
@@ -203,7 +216,14 @@ class CappedAttention(Part):
         return KVNeed(self.n_kv, self.kept, self.window, keep_first=self.keep_first, chunk=self.chunk)
 
     def state_needs(self) -> Optional[StateNeed]:
-        return None
+        return StateNeed((self.conv, (self.n_heads + 2 * self.n_kv) * self.kept), torch.float32) if self.conv else None
+
+    def _plain(self) -> bool:
+        """Nothing but rotation stands between the rows of q, k and v and the scores, and nothing behind the softmax: what
+        the decode kernel that turns the heads and writes the cache itself can do."""
+        return (self.norm_kind is None and self.value_mix is None and not self.softcap and not self.gated
+                and not self.has_sink and self.chunk is None and self.keep_first == 0
+                and float(getattr(self.position, "amplitude", 1.0)) == 1.0)
 
     def forward(self, step, io: LayerIO, h: torch.Tensor, residual: torch.Tensor, accumulate: bool = True):
         T = residual.shape[0]
@@ -211,9 +231,20 @@ class CappedAttention(Part):
         heads_width = (H + 2 * G) * P
         proj = step.ws.buf("cattn_proj", (T, heads_width + self.gate_cols), self.dtype)
         self.proj(h, proj)
+        gate = proj[:, heads_width:] if self.gate == "sigmoid" else None
+        head_gate = proj[:, heads_width:heads_width + H] if self.gate == "sigmoid_head" else None
+        if self.conv:
+            rows = step.ws.buf("cattn_conv", (T, heads_width), self.dtype)
+            kernels.causal_conv_ring(proj[:, :heads_width], self.conv_w, io.state, step, rows)
+            proj = rows
         table = self.position.rotary_table()
         inv_freq, rot = table if table is not None else (None, 0)
         amplitude = float(getattr(self.position, "amplitude", 1.0))
+        out = step.ws.buf("attn_out", (T, H * P), self.dtype)
+        if self.conv and self._plain() and kernels.attention_with_rope(step, proj, out, H, G, P, self.scale, self.window, io,
+                                                                       inv_freq, rot, io.writes_cache):
+            self.o(out, residual, accumulate=accumulate)
+            return None
         k_pages, v_pages = (io.k_pages, io.v_pages) if io.writes_cache else (None, None)
         if self.norm_kind == "whole" or self.value_mix is not None:
             if amplitude != 1.0:
@@ -234,11 +265,8 @@ class CappedAttention(Part):
                                     (self.norm_eps or 0.0) if head_norm else 0.0, step.positions, step.seq_of_token,
                                     io.block_table, k_pages, v_pages, io.page_size, norm_first=first,
                                     q_weight=self.q_norm_w if first else None, k_weight=self.k_norm_w if first else None)
-        out = step.ws.buf("attn_out", (T, H * P), self.dtype)
-        gate = proj[:, heads_width:] if self.gate == "sigmoid" else None
         # the flat decode kernel multiplies by an element gate's sigmoid as it stores, the decode kernel that splits a
         # sequence's keys by a head's gate where it combines the splits; behind the others a kernel does
-        head_gate = proj[:, heads_width:heads_width + H] if self.gate == "sigmoid_head" else None
         gated = kernels.attention(step, proj, out, H, G, P, self.scale, self.window, io, softcap=self.softcap, gate=gate,
                                   keep_first=self.keep_first, sinks=self.sinks, head_gate=head_gate,
                                   head_gate_mult=self.out_scale, chunk=self.chunk)

@@ -4,6 +4,7 @@
               stream at a fixed place (the start of a pass through a repeated run of layers).  Options:
               ``rows`` and ``width`` (the table's shape), ``row``.
 ``scale``     logits *= factor.  Option: ``factor``.
+``soft_cap``  logits <- cap tanh(logits / cap), in float32.  Option: ``cap``.
 ``rmsnorm``   x <- x / sqrt(mean(x^2) + eps) * (w + offset) over every row, in place and in float32: a norm of the
               embedded tokens before the first layer.  Options: ``width``, ``eps``, ``unit_offset`` (the stored weight
               is the gain minus one).
@@ -53,6 +54,20 @@ class Scale(Part):
         kernels.scale_(x, self.factor)
 
 
+class SoftCap(Part):
+    def __init__(self, spec: HookSpec, dtype: torch.dtype, device: torch.device):
+        super().__init__(spec, dtype, device)
+        self.cap = float(spec.options["cap"])
+        if not self.cap > 0.0:
+            raise ValueError(f"soft_cap: the cap must be positive, found {self.cap}")
+
+    def kernel_libraries(self) -> Tuple[str, ...]:
+        return ("elementwise",)
+
+    def forward(self, step, x: torch.Tensor) -> None:
+        kernels.soft_cap_(x, self.cap)
+
+
 class NormRows(Part):
     def __init__(self, spec: HookSpec, dtype: torch.dtype, device: torch.device):
         super().__init__(spec, dtype, device)
@@ -81,3 +96,4 @@ class NormRows(Part):
 register_hook("add_row", AddRow)
 register_hook("rmsnorm", NormRows)
 register_hook("scale", Scale)
+register_hook("soft_cap", SoftCap)

@@ -19,7 +19,7 @@ from typing import Dict, List, Mapping, Optional, Tuple
 
 import torch
 
-from ..parts.base import ParamDecl
+from ..parts.base import FreeDim, ParamDecl
 from .safetensors_io import SafetensorsError, open_model_files
 
 # Buffers some exporters write that are not parameters of any part.
@@ -55,6 +55,12 @@ def storage_dtype(stored: str, kind: str, run_dtype: torch.dtype) -> torch.dtype
     return torch.bfloat16
 
 
+def _shape_fits(found: Tuple[int, ...], declared: Tuple[int, ...]) -> bool:
+    """Equal dimension by dimension, but for those the declaration leaves to the file."""
+    return len(found) == len(declared) and all(f >= 1 if isinstance(d, FreeDim) else f == d
+                                               for f, d in zip(found, declared))
+
+
 def check_against(folder: str, declared: Mapping[str, ParamDecl],
                   found: Mapping[str, Tuple[str, Tuple[int, ...]]], ignored: Tuple[str, ...] = ()) -> None:
     """Raise one WeightError listing every disagreement between ``declared`` and ``found``.  ``ignored``: patterns of
@@ -68,8 +74,10 @@ def check_against(folder: str, declared: Mapping[str, ParamDecl],
         if n not in found:
             continue
         stored, shape = found[n]
-        if tuple(shape) != tuple(decl.shape):
-            wrong.append(f"{n}: expected {list(decl.shape)}, found {list(shape)}")
+        if not _shape_fits(tuple(shape), tuple(decl.shape)):
+            wrong.append(f"{n}: expected {['any' if isinstance(d, FreeDim) else d for d in decl.shape]}, found {list(shape)}"
+                         if any(isinstance(d, FreeDim) for d in decl.shape)
+                         else f"{n}: expected {list(decl.shape)}, found {list(shape)}")
         elif decl.kind == "float" and stored not in _FLOATS:
             wrong.append(f"{n}: expected a floating type, found {stored}")
         elif decl.kind == "int" and stored not in _INTS:
