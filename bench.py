@@ -12,6 +12,7 @@
     python bench.py --case tikalix [--shape 1b|8b] [--layers L]    the Tikalix design beside Llama at equal width, its kernels alone
     python bench.py --case vilazen [--shape 1b|8b] [--layers L]    the Vilazen design beside Llama at equal width, its kernels alone
     python bench.py --case lipadra [--shape 1b|8b] [--layers L]    the Lipadra design beside Tumatar and Llama at equal width, its kernels alone
+    python bench.py --case mopilorn [--shape 1b|8b] [--layers L]   the Mopilorn design beside Vilazen and Llama at equal width, its kernels alone
 
 A "step" is one decode step of a batch of 8 sequences at a context of 4096
 tokens.  ``value`` is decoded tokens a second, timed on the device with CUDA
@@ -1065,6 +1066,161 @@ def run_lipadra(args):
     return 0
 
 
+def run_mopilorn(args):
+    """The Mopilorn design beside the Vilazen design (the library's closest: windowed attention beside linear attention with
+    a matrix-valued state) and the Llama shape, all of the same width and with random weights: a prompt of
+    ``--prompt-tokens`` and decode steps of ``--batch`` sequences at ``--context``, ``--layers`` layers of each (default 4), and
+    every kernel the design adds, alone, against its own roofline (the larger of bytes / measured copy bandwidth, FLOPs /
+    measured bf16 peak and float32 FMA work / (2 x 128 lanes x 148 SMs x the clock)), each beside the library's like kernel
+    timed in the same run on operands of the same size."""
+    import torch
+    from types import SimpleNamespace
+    from ziglm_b200 import kernels
+    from ziglm_b200.config.shapes import shape
+    from ziglm_b200.engine.workspace import Workspace
+    torch.cuda.set_device(0)
+    pk = peaks()
+    size = "8b" if args.shape == "8b" else "1b"
+    layers = args.layers or 4
+    T, batch, context = args.prompt_tokens, args.batch, args.context
+    max_seq = max(context, T) + 64
+    gen = torch.Generator().manual_seed(7)
+    out = {"case": "mopilorn", "width_of": "llama-" + size, "dtype": "bf16", "layers": layers, "prompt_tokens": T,
+           "batch": batch, "context": context, "data": "synthetic", "l2": "a 256 MiB buffer is rewritten before every timed call",
+           "peaks": pk["source"], "models": {}}
+    with ClockSampler() as clocks:
+        for name in ("mopilorn-" + size, "vilazen-" + size, "llama-" + size):
+            cfg = shape(name)
+            if "layers" in cfg:
+                cfg["layers"] = cfg["layers"][:layers]
+                vocab = cfg["vocab"]
+            else:
+                cfg["num_hidden_layers"] = layers
+                cfg["max_position_embeddings"] = max(cfg["max_position_embeddings"], max_seq)
+                vocab = cfg["vocab_size"]
+            eng = _engine_for(cfg, "bfloat16", batch, max_seq)
+            ids = lambda n: torch.randint(0, vocab, (n,), generator=gen).tolist()
+            pre = _time_prompt(eng, ids(T), args.warmup, args.steps)
+            dec = _time_decode_at(eng, batch, context, args.warmup, args.steps, ids)
+            out["models"][name] = {"prefill_ms": round(pre, 3), "prefill_tok_s": round(T / pre * 1e3, 1),
+                                   "decode_ms": round(dec, 4), "decode_tok_s": round(batch / dec * 1e3, 1)}
+            del eng
+            torch.cuda.empty_cache()
+    out["clocks"] = clocks.summary()
+    # ---- the kernels, alone
+    cfg = shape("mopilorn-" + size)
+    d, S, vocab = cfg["width"], cfg["streams"], cfg["vocab"]
+    left, right, chan = cfg["layers"][0]["mixer"]["left"], cfg["layers"][0]["mixer"]["right"], cfg["layers"][1]["mixer"]
+    dev = torch.device("cuda:0")
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=dev)
+    bf = lambda *sh: (torch.randn(*sh, device=dev) * 0.05).to(torch.bfloat16)
+    f32 = lambda *sh: torch.randn(*sh, device=dev) * 0.05
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    hbm, peak = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    fma = 2.0 * 128 * 148 * 1.9e9
+    rows = []
+
+    def report(what, like, ms, nbytes, flops, fma_flops=0.0):
+        floor = max(nbytes / hbm, flops / peak, fma_flops / fma) * 1e3
+        rows.append({"kernel": what, "like": like, "ms": round(ms, 4), "roofline_ms": round(floor, 4),
+                     "frac_of_roofline": round(floor / ms, 4)})
+
+    def timed(fn):
+        return _timed(fn, args.warmup, args.steps, flush)
+
+    kernels.require(("elementwise", "streams", "recurrent", "delta_rule", "linear_attention"))
+    LH, LD = right["heads"], right["dim"]
+    chunk = kernels.linear_attention_chunk()
+    pows = torch.tensor([[0.97 ** n for n in range(chunk + 1)] for _ in range(LH)], dtype=torch.float64).float().to(dev)
+    for n_tok, tag in ((T, f"prompt of {T}"), (batch, f"decode batch {batch}")):
+        decode = n_tok != T
+        past = context - 1 if decode else 0
+        new = [1] * n_tok if decode else [T]
+        n_seq = len(new)
+        cu = [0]
+        for n in new:
+            cu.append(cu[-1] + n)
+        step = SimpleNamespace(
+            n_tokens=n_tok, n_seqs=n_seq, single_token=decode, max_new=max(new), max_total=past + max(new),
+            positions=i32([past + i for n in new for i in range(n)]), seq_of_token=i32([b for b, n in enumerate(new) for _ in range(n)]),
+            cu_seqlens=i32(cu), past_lens=i32([past] * n_seq), slots=i32(list(range(n_seq))), ws=Workspace(dev))
+        # residual streams, beside the norm that adds a branch and leaves the next rows, and the plain norm
+        x, xs, br, br2 = f32(n_tok, d), f32(n_tok, S * d), f32(n_tok, d), f32(n_tok, d)
+        w, wb, hrow = f32(d) + 1, bf(d), torch.empty(n_tok, d, dtype=torch.bfloat16, device=dev)
+        coef, gather = torch.cat([torch.eye(S).reshape(-1), torch.ones(S)]).to(dev), torch.full((S,), 0.5, device=dev)
+        ms = timed(lambda: kernels.rmsnorm(x, wb, hrow, 1e-6))
+        report(f"rmsnorm, {tag}", "-", ms, n_tok * d * 6, 0)
+        ms = timed(lambda: kernels.stream_norm(xs, S, gather, w, 1e-6, hrow))
+        report(f"stream_norm ({S} streams), {tag}", "rmsnorm", ms, n_tok * d * (4 * S + 2), 0)
+        ms = timed(lambda: kernels.norm_add_scaled(br, wb, 1e-6, 0.5, x, hrow))
+        report(f"norm_add_scaled (x += m norm(branch), and the next rows), {tag}", "rmsnorm", ms, n_tok * d * 14, 0)
+        ms = timed(lambda: kernels.stream_mix(xs, S, coef, [br], nxt=(gather, w, 1e-6, hrow)))
+        report(f"stream_mix ({S} streams, one branch, and the next rows), {tag}", "norm_add_scaled", ms, n_tok * d * (8 * S + 6), 0)
+        ms = timed(lambda: kernels.stream_mix(xs, S, coef, [br, br2], [w, w], 1e-6, 0.5, nxt=(gather, w, 1e-6, hrow)))
+        report(f"stream_mix ({S} streams, two normed branches, and the next rows), {tag}", "norm_add_scaled", ms,
+               n_tok * d * (8 * S + 10), 0)
+        # the convolution with its own ring of inputs, beside the convolution whose inputs a scan keeps
+        C, K = (left["heads"] + 2 * left["kv_heads"]) * left["dim"], left["conv"]
+        proj, y = bf(n_tok, C), torch.empty(n_tok, C, dtype=torch.bfloat16, device=dev)
+        taps, ring = f32(K, C), torch.zeros(n_seq, K, C, device=dev)
+        ms = timed(lambda: kernels.causal_conv(proj, taps, torch.zeros(C, device=dev), ring, step, y))
+        report(f"causal_conv ({C} channels), {tag}", "-", ms, n_tok * C * 4, 0)
+        ms = timed(lambda: kernels.causal_conv_ring(proj, taps, ring, step, y))
+        report(f"causal_conv_ring ({C} channels), {tag}", "causal_conv", ms, n_tok * C * 4, 0)
+        # the delta rule, beside linear attention with a fixed decay and as many heads
+        lproj = bf(n_tok, LH * 3 * LD)
+        state = torch.zeros(n_seq, LH, LD, LD, device=dev)
+        mixed = torch.empty(n_tok, LH * LD, device=dev)
+        la_bytes = n_tok * LH * 3 * LD * 2 + n_tok * LH * LD * 4 + n_seq * LH * LD * LD * 8
+        c = min(chunk, max(new))
+        ms = timed(lambda: kernels.decayed_linear_attention(lproj, 0, LH * LD, 2 * LH * LD, LH, LD, LD, None, pows, state, step,
+                                                            mixed))
+        report(f"decayed_linear_attention ({LH} heads of {LD}), {tag}", "-", ms, la_bytes, 0,
+               2.0 * n_tok * LH * (c * LD + c * LD + 2 * LD * LD))
+        lout, gate = torch.empty(n_tok, LH * LD, dtype=torch.bfloat16, device=dev), bf(n_tok, LH * LD)
+        wl = f32(LH * LD) + 1
+        ms = timed(lambda: kernels.head_norm_gate(mixed, None, gate, lout, LH, 1e-6, "silu", 1.0))
+        report(f"head_norm_gate without a weight, {tag}", "-", ms, n_tok * LH * LD * 8, 0)
+        ms = timed(lambda: kernels.head_norm_gate(mixed, wl, gate, lout, LH, 1e-6, "silu", 1.0))
+        report(f"head_norm_gate with a weight, {tag}", "head_norm_gate", ms, n_tok * LH * LD * 8, 0)
+        for m, kind in ((right, "a decay a head"), (chan, "a decay a key channel")):
+            H, G, D, V, K = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+            per = D if kind.endswith("channel") else 1
+            C = 2 * G * D + H * V
+            dproj, taps, ring = bf(n_tok, C), f32(K, C), torch.zeros(n_seq, K, C, device=dev)
+            a, b, rate, bias = f32(n_tok, H * per), f32(n_tok, H), torch.rand(H, device=dev), f32(H * per)
+            dst = torch.zeros(n_seq, H, V, kernels.delta_state_size(D), device=dev)
+            args_d = (dproj, taps, ring, H, G, D, V, a, b, rate, bias)
+            state_bytes, rule_fma = n_seq * H * D * V * 8, 7.0 * n_tok * H * D * V
+            if decode:
+                ms = timed(lambda: kernels.delta_rule_decode(*args_d, dst, step, wl[:V].contiguous(), 1e-6, gate, "silu", lout))
+                report(f"delta_rule_decode ({H} heads of {D}, {kind}; convolution to gated heads), {tag}",
+                       "decayed_linear_attention", ms, state_bytes + n_tok * (C * 2 + H * per * 4 + H * V * 4) + n_seq * K * C * 4, 0,
+                       rule_fma)
+                continue
+            made = kernels.delta_prep(*args_d, step)
+            ms = timed(lambda: kernels.delta_prep(*args_d, step))
+            report(f"delta_prep ({H} heads of {D}, {kind}), {tag}", "causal_conv", ms,
+                   n_tok * (C * 6 + H * per * 8 + H * 8), 0)
+            chunks = kernels.delta_chunk(made[0], made[2], made[3], H, G, D, step)
+            ms = timed(lambda: kernels.delta_chunk(made[0], made[2], made[3], H, G, D, step))
+            moved = (3 * H * D * 4) if per > 1 else H * 8
+            report(f"delta_chunk ({H} heads of {D}, {kind}), {tag}", "causal_conv", ms,
+                   n_tok * (2 * G * D * 4 + H * per * 4 + moved + H * 64), 0)
+            ms = timed(lambda: kernels.delta_scan(made[0], made[1], chunks, H, G, D, V, dst, step, mixed))
+            report(f"delta_scan ({H} heads of {D}, {kind}), {tag}", "decayed_linear_attention", ms,
+                   state_bytes + n_tok * (C * 4 + H * per * 4 + H * V * 4), 0, rule_fma)
+        z = f32(batch, vocab)
+        ms = timed(lambda: kernels.scale_(z, 1.0))
+        report(f"scale_ ({batch} rows of {vocab} logits), {tag}", "-", ms, batch * vocab * 8, 0)
+        ms = timed(lambda: kernels.soft_cap_(z, 30.0))
+        report(f"soft_cap_ ({batch} rows of {vocab} logits), {tag}", "scale_", ms, batch * vocab * 8, 0)
+    out["kernels"] = rows
+    out["wait_errors"] = wait_errors(kernels)
+    print(json.dumps(out))
+    return 0
+
+
 def run_workload(args):
     """The two workloads beside the headline one, through ``Engine.generate`` (host token ids in, ids out):
 
@@ -1284,13 +1440,14 @@ def main():
                     help="run fewer layers than the configuration has (both numbers are reported)")
     ap.add_argument("--case", default="full",
                     choices=["full", "prefill", "decode", "workload-1b", "workload-13b", "float32", "reference-kernels",
-                             "tumatar", "tikalix", "vilazen", "lipadra"],
+                             "tumatar", "tikalix", "vilazen", "lipadra", "mopilorn"],
                     help="full: the whole measurement; prefill / decode: that phase alone (for profilers and sweeps); "
                          "workload-1b / workload-13b: the two other workloads through Engine.generate; float32: the "
                          "8B shape in true 32-bit; reference-kernels: the reference's CUDA kernels alone, if built; tumatar: the "
                          "Tumatar design beside the Llama shape of the same width (--shape 1b or 8b), and its kernels alone; tikalix: "
                          "the same for the Tikalix design; vilazen: the same for the Vilazen design; lipadra: the Lipadra design "
-                         "beside the Tumatar design and the Llama shape of the same width, and its kernels alone")
+                         "beside the Tumatar design and the Llama shape of the same width, and its kernels alone; mopilorn: the "
+                         "Mopilorn design beside the Vilazen design and the Llama shape likewise")
     ap.add_argument("--shape", default="8b", choices=sorted(SHAPES), help="--case prefill/decode: layer sizes")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="--case prefill/decode")
     ap.add_argument("--repeats", type=int, default=2, help="workload cases: timed repetitions after one warm-up")
@@ -1320,6 +1477,8 @@ def main():
         return run_vilazen(args)
     if args.case == "lipadra":
         return run_lipadra(args)
+    if args.case == "mopilorn":
+        return run_mopilorn(args)
     if args.case != "full":
         return run_case(args)
     return run_ours(args)

@@ -146,6 +146,31 @@ SHAPES["lipadra-1b"] = _lipadra(2048, 128256, 4, 32, 8, 64, 16, 2048)
 SHAPES["lipadra-8b"] = _lipadra(4096, 128256, 8, 32, 8, 128, 16, 3584)
 
 
+def _mopilorn(width: int, vocab: int, pairs: int, heads: int, kv_heads: int, dim: int, ff: int) -> Dict[str, Any]:
+    """A Mopilorn stack of ``pairs`` times (windowed attention beside a delta rule with a decay a head, a delta rule with a
+    decay a key channel) with the attention heads of the Llama shape of that width: keys and values of one size, half of
+    every head rotated with frequencies stretched eightfold, windows of 1,024 positions, convolutions of four taps, delta
+    rules over heads of 128 (two share the q and k of one in the parallel layer), products of rank 128, two residual
+    streams."""
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "conv": 4,
+            "rot": {"dims": dim // 2, "base": 500000.0,
+                    "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}},
+            "mask": {"size": 1024}}
+    delta_heads = width // 128
+    right = {"heads": delta_heads, "kv_heads": delta_heads // 2, "dim": 128, "vdim": 128, "conv": 4}
+    channel = {"heads": delta_heads, "kv_heads": delta_heads, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128,
+               "gate_rank": 128}
+    mlp = {"kind": "dense", "ff": ff}
+    two = ({"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": mlp},
+           {"type": "channel_delta", "mixer": channel, "mlp": mlp})
+    return {"architecture": "Mopilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": 2,
+            "logit_softcap": 30.0, "layers": [copy.deepcopy(x) for _ in range(pairs) for x in two]}
+
+
+SHAPES["mopilorn-1b"] = _mopilorn(2048, 128256, 8, 32, 8, 64, 8192)
+SHAPES["mopilorn-8b"] = _mopilorn(4096, 128256, 16, 32, 8, 128, 14336)
+
+
 def shape(name: str) -> Dict[str, Any]:
     """A copy of the named config.json dictionary."""
     try:

@@ -16,20 +16,26 @@
 // before it waits for the projection, makes q, k, v, g and beta, updates S in place, norms the head's output over V,
 // applies weight and gate and writes the rows the output projection reads.
 //
-// Any other step is two kernels.  dr_prep makes q, k, v, g, beta of every token in float and writes the ring.  dr_scan
-// walks a sequence's tokens with S in registers: a column of S is spread over L lanes of a warp (4 NI elements a lane)
-// and the columns of a head over blocks, which need nothing from each other.  A token would cost two dependent
-// reductions over those lanes; the walk keeps the write of the token before pending instead,
-//     Sbar_t = diag(g_t) (Sbar_(t-1) + k_(t-1) u_(t-1)),     u_t = beta_t (v_t - r_t - c_t u_(t-1)),
-//     r_(t+1) = (g_(t+1) k_(t+1)) . Sbar_t,  c_t = (g_t k_t) . k_(t-1),   o_t = q_t . Sbar_t + (q_t . k_t) u_t,
-// so the reduction that u_(t+1) needs starts before u_t is known, and both reductions of a token run side by side.
-// Tokens come in chunks through shared memory (cp.async, two stages); c and q . k are taken once a chunk.  Every sum is
-// float FMA; nothing that enters the recurrence passes through a 16-bit type behind the projection.
+// Any other step is three kernels, over chunks of DR_C tokens of a sequence.  dr_prep makes q, k, v, g, beta of every
+// token in float and writes the ring.  Behind a state S0 a chunk unrolls to (products of decays: from where to where)
+//     R_t = (G_0t k_t) . S0            A_tj = beta_t (G_jt k_t) . k_j   (j < t)     u = (I + A)^-1 beta (v - R)
+//     o_t = (G_0t q_t) . S0 + sum_(j <= t) B_tj u_j,  B_tj = (G_jt q_t) . k_j       S = G_0n S0 + sum_j (G_jn k_j) u_j^T
+// with G_jt the product of the decays of the tokens behind j up to t: never a quotient, so a strong decay is a zero and not
+// an overflow.  dr_chunk makes everything of this that does not depend on S, all chunks and heads side by side: the
+// weighted keys and queries, T = (I + A)^-1 diag(beta) and B.  dr_scan walks the chunks with S in registers, so a chunk is
+// three float products of which none waits for the token before: a column of S is spread over 16 lanes of a warp, a
+// lane holding two columns, the columns of a head over blocks, which need nothing from each other; the sums over the
+// lanes are scattered so that lane (t, column) ends with R_t and o_t of its column.  The chunks come through shared memory
+// (cp.async, three stages).  Every sum is float FMA (two at a time, fma.rn.f32x2); nothing that enters the recurrence
+// passes through a 16-bit type behind the projection.
 #include "common.cuh"
 
 namespace zlm {
 
-constexpr int DR_THREADS = 128;      // of the scan: 128 / L value columns a block
+constexpr int DR_C = 8;              // tokens of a chunk
+constexpr int DR_L = 16;             // lanes that share a column of the state in dr_scan
+constexpr int DR_THREADS = 128;      // of dr_chunk (DR_C tokens x DR_L lanes) and of dr_scan
+constexpr int DR_VT = 16;            // value columns of a block of dr_scan: two a lane, two times DR_L lanes a warp
 constexpr int DR_PREP_WARPS = 4;
 
 __device__ __forceinline__ float dr_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
@@ -101,7 +107,6 @@ __global__ void __launch_bounds__(DR_PREP_WARPS * 32)
 dr_prep_kernel(DrIn<T> in, int channel_decay, int tile, float* __restrict__ qk_out, float* __restrict__ v_out,
                float* __restrict__ g_out, float* __restrict__ beta_out) {
     extern __shared__ float dr_sm[];
-    pdl_launch_dependents();
     pdl_wait();
     const int b = blockIdx.z;
     const int first = in.cu_seqlens[b], n_new = in.cu_seqlens[b + 1] - first;
@@ -195,165 +200,347 @@ template <int L> __device__ __forceinline__ float dr_sum(float v) {
     return v;
 }
 
-__host__ __device__ constexpr int dr_chunk(int DS) { return 2048 / DS > 16 ? 16 : 2048 / DS; }      // tokens of a chunk
-static inline size_t dr_scan_floats(int L, int NI, bool ch) {
-    const int DS = 4 * L * NI, TC = dr_chunk(DS), VT = DR_THREADS / L;
-    const size_t stage = (size_t)TC * ((ch ? 3 : 2) * DS + VT + (ch ? 1 : 2));
-    return 2 * ((stage + 3) / 4 * 4) + (ch ? (size_t)TC * DS : 0) + 2 * TC + (size_t)TC * VT;
+// The place of a chunk among all chunks of the step: sequence b's chunks lie behind those of the sequences before it.
+__device__ __forceinline__ long dr_chunk_index(int first, int b, int chunk) { return (long)(first / DR_C) + b + chunk; }
+
+// grid (chunks of the longest sequence, heads, sequences); thread (j, l): token j of the chunk, lane l of its D elements.
+// qk: float [T][2 G][Dp]; g: [T][H][Dp] (CH) or [T][H]; beta: [T][H].
+// wk, wq, we: float [T][H][Dp], the chunk's weighted keys and queries G_0t k_t, G_0t q_t and G_jn k_j (CH);
+// ws: float [T][H][2], G_0t and G_jn (not CH).  gam: [chunks][H][Dp] or [chunks][H], G_0n.
+// tb: float [T][H][2 DR_C], row t of T, then row t of B; rows behind the chunk's last token are not written.
+template <int NI, bool CH>
+__global__ void __launch_bounds__(DR_THREADS)
+dr_chunk_kernel(const float* __restrict__ qk, const float* __restrict__ g, const float* __restrict__ beta,
+                const int* __restrict__ cu_seqlens, float* __restrict__ wk, float* __restrict__ wq, float* __restrict__ we,
+                float* __restrict__ ws, float* __restrict__ gam, float* __restrict__ tb, int H, int G, int Dp) {
+    constexpr int D4 = DR_L * NI;                          // float4 of a padded row
+    extern __shared__ __align__(16) float dr_sm[];
+    float4* k4 = reinterpret_cast<float4*>(dr_sm);         // [DR_C][D4]
+    float4* q4 = k4 + DR_C * D4;
+    float4* g4 = q4 + DR_C * D4;                           // CH
+    __shared__ float a_s[DR_C][DR_C], b_s[DR_C][DR_C], g_s[DR_C], beta_s[DR_C];
+    pdl_wait();
+    const int b = blockIdx.z, h = blockIdx.y, kv = h / (H / G);
+    const int first = cu_seqlens[b], n_new = cu_seqlens[b + 1] - first;
+    const int at = blockIdx.x * DR_C, n = min(DR_C, n_new - at);
+    if (n <= 0) return;
+    const int tid = threadIdx.x, j = tid / DR_L, l = tid % DR_L, d4 = Dp / 4;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const long t0 = first + at;
+    for (int idx = tid; idx < DR_C * D4; idx += DR_THREADS) {
+        const int t = idx / D4, i = idx - t * D4;
+        const bool in = t < n && i < d4;
+        k4[idx] = in ? reinterpret_cast<const float4*>(qk + ((t0 + t) * 2 * G + G + kv) * Dp)[i] : zero;
+        q4[idx] = in ? reinterpret_cast<const float4*>(qk + ((t0 + t) * 2 * G + kv) * Dp)[i] : zero;
+        if constexpr (CH) g4[idx] = in ? reinterpret_cast<const float4*>(g + ((t0 + t) * H + h) * Dp)[i] : zero;
+    }
+    if (tid < DR_C) {
+        beta_s[tid] = tid < n ? beta[(t0 + tid) * H + h] : 0.f;
+        if constexpr (!CH) g_s[tid] = tid < n ? g[(t0 + tid) * H + h] : 0.f;
+    }
+    if (tid < DR_C * DR_C) (&a_s[0][0])[tid] = (&b_s[0][0])[tid] = 0.f;
+    __syncthreads();
+    // token j's key, decayed from one later token to the next: its products with their k and q
+    float4 w[NI];
+    float wsc = 1.f;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) w[i] = k4[j * D4 + l + DR_L * i];
+    for (int t = 0; t < n; ++t) {                          // every thread takes every round: shuffles inside
+        const bool on = t >= j;
+        float ka = 0.f, qa = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const float4 kk = k4[t * D4 + l + DR_L * i], qq = q4[t * D4 + l + DR_L * i];
+            if constexpr (CH) {
+                if (t > j) {
+                    const float4 gg = g4[t * D4 + l + DR_L * i];
+                    w[i].x *= gg.x; w[i].y *= gg.y; w[i].z *= gg.z; w[i].w *= gg.w;
+                }
+            }
+            ka = fmaf(kk.x, w[i].x, ka); ka = fmaf(kk.y, w[i].y, ka); ka = fmaf(kk.z, w[i].z, ka); ka = fmaf(kk.w, w[i].w, ka);
+            qa = fmaf(qq.x, w[i].x, qa); qa = fmaf(qq.y, w[i].y, qa); qa = fmaf(qq.z, w[i].z, qa); qa = fmaf(qq.w, w[i].w, qa);
+        }
+        if constexpr (!CH) { if (t > j) wsc *= g_s[t]; }
+        ka = dr_sum<DR_L>(ka);
+        qa = dr_sum<DR_L>(qa);
+        if (on && l == 0) {
+            b_s[t][j] = qa * wsc;
+            if (t > j) a_s[t][j] = beta_s[t] * (ka * wsc);
+        }
+    }
+    if (j < n) {
+        const long row = (t0 + j) * H + h;
+        if constexpr (CH) {
+            // from the state to token j, and from token j to the chunk's end (what w has become)
+            float4 G0[NI];
+#pragma unroll
+            for (int i = 0; i < NI; ++i) G0[i] = g4[l + DR_L * i];
+            for (int t = 1; t <= j; ++t) {
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    const float4 gg = g4[t * D4 + l + DR_L * i];
+                    G0[i].x *= gg.x; G0[i].y *= gg.y; G0[i].z *= gg.z; G0[i].w *= gg.w;
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                if (l + DR_L * i >= d4) continue;
+                const float4 kk = k4[j * D4 + l + DR_L * i], qq = q4[j * D4 + l + DR_L * i];
+                reinterpret_cast<float4*>(wk + row * Dp)[l + DR_L * i] =
+                    make_float4(G0[i].x * kk.x, G0[i].y * kk.y, G0[i].z * kk.z, G0[i].w * kk.w);
+                reinterpret_cast<float4*>(wq + row * Dp)[l + DR_L * i] =
+                    make_float4(G0[i].x * qq.x, G0[i].y * qq.y, G0[i].z * qq.z, G0[i].w * qq.w);
+                reinterpret_cast<float4*>(we + row * Dp)[l + DR_L * i] = w[i];
+                if (j == n - 1)
+                    reinterpret_cast<float4*>(gam + (dr_chunk_index(first, b, blockIdx.x) * H + h) * Dp)[l + DR_L * i] = G0[i];
+            }
+        } else if (l == 0) {
+            float g0 = 1.f;
+            for (int t = 0; t <= j; ++t) g0 *= g_s[t];
+            ws[row * 2] = g0;
+            ws[row * 2 + 1] = wsc;
+            if (j == n - 1) gam[dr_chunk_index(first, b, blockIdx.x) * H + h] = g0;
+        }
+    }
+    __syncthreads();
+    // column c of T: (I + A) x = beta_c e_c, downwards
+    if (tid < DR_C) {
+        float x[DR_C];
+#pragma unroll
+        for (int t = 0; t < DR_C; ++t) {
+            float acc = t == tid ? beta_s[t] : 0.f;
+#pragma unroll
+            for (int u = 0; u < t; ++u) acc = fmaf(-a_s[t][u], x[u], acc);
+            x[t] = acc;
+            if (t < n) tb[((t0 + t) * H + h) * (2 * DR_C) + tid] = acc;
+        }
+    } else if (tid >= 64) {
+        const int i = tid - 64, t = i / DR_C;
+        if (t < n) tb[((t0 + t) * H + h) * (2 * DR_C) + DR_C + i % DR_C] = b_s[t][i % DR_C];
+    }
 }
 
-// grid (value tiles, heads, sequences).  qk: float [T][2 G][Dp], v: [T][H][Vp], g: [T][H][Dp] or [T][H], beta: [T][H];
-// out: float [T][H * V] rows.
-template <int L, int NI, bool CH>
+// Two floats at a time.
+typedef unsigned long long dr_f2;
+__device__ __forceinline__ dr_f2 dr_fma2(dr_f2 a, dr_f2 b, dr_f2 c) {
+    dr_f2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ dr_f2 dr_mul2(dr_f2 a, dr_f2 b) {
+    dr_f2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ dr_f2 dr_pack2(float x, float y) {
+    dr_f2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(x), "f"(y));
+    return d;
+}
+__device__ __forceinline__ float dr_both(dr_f2 v) {
+    float x, y;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v));
+    return x + y;
+}
+
+// The sums over 16 lanes of 16 numbers a lane, scattered: lane m is left with the sum of number m.
+__device__ __forceinline__ float dr_scatter16(float (&a)[16], int l) {
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) {
+        const bool up = (l & o) != 0;
+#pragma unroll
+        for (int i = 0; i < o; ++i) {
+            const float give = up ? a[i] : a[i + o], keep = up ? a[i + o] : a[i];
+            a[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+    }
+    return a[0];
+}
+
+constexpr int DR_STAGES = 3;
+// floats of a stage: the rows k, q (and, with a decay a channel, the keys for the state), the values, T and B, the decays
+__host__ __device__ constexpr int dr_stage(int NI, bool ch) {
+    return DR_C * (64 * NI * (ch ? 3 : 2) + DR_VT + 2 * DR_C + (ch ? 0 : 2)) + (ch ? 64 * NI : 4);
+}
+
+// grid (value tiles, heads, sequences).  CH: kr, qr, er are wk, wq, we of dr_chunk (rows [T][H][Dp]); else kr is qk (rows
+// [T][2 G][Dp]) and ws holds the weights.  v: [T][H][Vp]; out: float rows of H V numbers.
+template <int NI, bool CH>
 __global__ void __launch_bounds__(DR_THREADS)
-dr_scan_kernel(const float* __restrict__ qk, const float* __restrict__ v, const float* __restrict__ g,
-               const float* __restrict__ beta, float* __restrict__ state, const int* __restrict__ slots,
+dr_scan_kernel(const float* __restrict__ kr, const float* __restrict__ qr, const float* __restrict__ er,
+               const float* __restrict__ ws, const float* __restrict__ gam, const float* __restrict__ tb,
+               const float* __restrict__ v, float* __restrict__ state, const int* __restrict__ slots,
                const int* __restrict__ cu_seqlens, float* __restrict__ out, long out_stride, int H, int G, int Dp, int V,
                int Vp) {
-    constexpr int DS = 4 * L * NI, TC = dr_chunk(DS), VT = DR_THREADS / L, D4 = DS / 4;
-    constexpr int STAGE = (TC * ((CH ? 3 : 2) * DS + VT + (CH ? 1 : 2)) + 3) / 4 * 4;
+    constexpr int DS = 64 * NI, D4 = DS / 4, STAGE = dr_stage(NI, CH), ROWS = CH ? 3 : 2;
     extern __shared__ __align__(16) float dr_sm[];
-    float* kg_s = dr_sm + 2 * STAGE;                       // [TC][DS] g k (CH)
-    float* c_s = kg_s + (CH ? TC * DS : 0);                // [TC]
-    float* qd_s = c_s + TC;                                // [TC]
-    float* o_s = qd_s + TC;                                // [TC][VT]
-    pdl_launch_dependents();
-    const int tid = threadIdx.x, l = tid % L, col = tid / L;
-    const int b = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * VT;
-    const int kv = h / (H / G);
-    const int d4 = Dp / 4;
-    const int vcol = v0 + col;
-    const bool live = vcol < V;
-    // what stands behind the live elements of a row stays zero
-    for (int i = tid; i < 2 * STAGE; i += DR_THREADS) dr_sm[i] = 0.f;
-    if constexpr (CH) for (int i = tid; i < TC * DS; i += DR_THREADS) kg_s[i] = 0.f;
-    float* st = state + (((long)slots[b] * H + h) * V + (live ? vcol : 0)) * Dp;
-    float4 S[NI];
+    const int tid = threadIdx.x, lane = tid & 31, l = lane & 15;
+    const int b = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * DR_VT;
+    const int kv = h / (H / G), d4 = Dp / 4;
+    const int col0 = (tid >> 5) * 4 + (lane >> 4) * 2;      // this lane's two columns of the tile
+    const int my_t = l >> 1, my_col = col0 + (l & 1);       // what the scattered sums leave this lane with
+    // what stands behind the live elements of a row, and behind a short chunk's last token, is zero or finite
+    for (int i = tid; i < DR_STAGES * STAGE; i += DR_THREADS) dr_sm[i] = 0.f;
+    float* st = state + ((long)slots[b] * H + h) * V * Dp;
+    dr_f2 S[2][2 * NI];
 #pragma unroll
-    for (int i = 0; i < NI; ++i)
-        S[i] = (live && l + L * i < d4) ? reinterpret_cast<const float4*>(st)[l + L * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int c = 0; c < 2; ++c) {
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            ulonglong2 s = make_ulonglong2(0, 0);
+            if (v0 + col0 + c < V && l + DR_L * i < d4)
+                s = reinterpret_cast<const ulonglong2*>(st + (long)(v0 + col0 + c) * Dp)[l + DR_L * i];
+            S[c][2 * i] = s.x; S[c][2 * i + 1] = s.y;
+        }
+    }
     pdl_wait();
     __syncthreads();
     const int first = cu_seqlens[b], n_new = cu_seqlens[b + 1] - first;
-    auto fetch = [&](int at, int stage) {
-        float* sm = dr_sm + stage * STAGE;
-        const int n = min(TC, n_new - at);
-        for (int idx = tid; idx < n * d4; idx += DR_THREADS) {
-            const int j = idx / d4, i = idx - j * d4;
-            const long t = first + at + j;
-            dr_cp16(sm + j * DS + 4 * i, qk + (t * 2 * G + kv) * Dp + 4 * i);
-            dr_cp16(sm + (TC + j) * DS + 4 * i, qk + (t * 2 * G + G + kv) * Dp + 4 * i);
-            if constexpr (CH) dr_cp16(sm + (2 * TC + j) * DS + 4 * i, g + (t * H + h) * Dp + 4 * i);
-        }
-        float* v_s = sm + (CH ? 3 : 2) * TC * DS;
-        for (int idx = tid; idx < n * (VT / 4); idx += DR_THREADS) {
-            const int j = idx / (VT / 4), i = idx - j * (VT / 4);
-            if (v0 + 4 * i < Vp) dr_cp16(v_s + j * VT + 4 * i, v + ((first + at + j) * (long)H + h) * Vp + v0 + 4 * i);
-        }
-        float* s_s = v_s + TC * VT;
-        for (int j = tid; j < n; j += DR_THREADS) {
-            const long t = first + at + j;
-            s_s[j] = beta[t * H + h];
-            if constexpr (!CH) s_s[TC + j] = g[t * H + h];
+    const int n_chunks = (n_new + DR_C - 1) / DR_C;
+    auto fetch = [&](int chunk) {
+        if (chunk < n_chunks) {
+            float* sm = dr_sm + (chunk % DR_STAGES) * STAGE;
+            const int at = chunk * DR_C, n = min(DR_C, n_new - at);
+            for (int idx = tid; idx < n * d4; idx += DR_THREADS) {
+                const int j = idx / d4, i = 4 * (idx - j * d4);
+                const long t = first + at + j;
+                if constexpr (CH) {
+                    dr_cp16(sm + j * DS + i, kr + (t * H + h) * Dp + i);
+                    dr_cp16(sm + (DR_C + j) * DS + i, qr + (t * H + h) * Dp + i);
+                    dr_cp16(sm + (2 * DR_C + j) * DS + i, er + (t * H + h) * Dp + i);
+                } else {
+                    dr_cp16(sm + j * DS + i, kr + (t * 2 * G + G + kv) * Dp + i);
+                    dr_cp16(sm + (DR_C + j) * DS + i, kr + (t * 2 * G + kv) * Dp + i);
+                }
+            }
+            float* v_s = sm + ROWS * DR_C * DS;
+            if (tid < n * (DR_VT / 4)) {
+                const int j = tid / (DR_VT / 4), i = 4 * (tid % (DR_VT / 4));
+                if (v0 + i < Vp) dr_cp16(v_s + j * DR_VT + i, v + ((first + at + j) * (long)H + h) * Vp + v0 + i);
+            }
+            float* tb_s = v_s + DR_C * DR_VT;
+            if (tid >= 64 && tid - 64 < n * (2 * DR_C / 4)) {
+                const int j = (tid - 64) / (2 * DR_C / 4), i = 4 * ((tid - 64) % (2 * DR_C / 4));
+                dr_cp16(tb_s + j * 2 * DR_C + i, tb + ((first + at + j) * (long)H + h) * (2 * DR_C) + i);
+            }
+            float* g_s = tb_s + DR_C * 2 * DR_C;
+            const float* gsrc = gam + (dr_chunk_index(first, b, chunk) * H + h) * (CH ? Dp : 1);
+            if constexpr (CH) {
+                for (int i = tid; i < d4; i += DR_THREADS) dr_cp16(g_s + 4 * i, gsrc + 4 * i);
+            } else {
+                if (tid == 0) g_s[0] = gsrc[0];
+                if (tid >= 32 && tid - 32 < n) {
+                    const float* w = ws + ((first + at + tid - 32) * (long)H + h) * 2;
+                    g_s[4 + tid - 32] = w[0];
+                    g_s[4 + DR_C + tid - 32] = w[1];
+                }
+            }
+            // a short chunk: the rows of T and B behind its last token must be zero
+            if (n < DR_C) for (int i = n * 2 * DR_C + tid; i < DR_C * 2 * DR_C; i += DR_THREADS) tb_s[i] = 0.f;
         }
         dr_cp_commit();
     };
-    fetch(0, 0);
-    for (int at = 0, stage = 0; at < n_new; at += TC, stage ^= 1) {
-        const int n = min(TC, n_new - at);
-        if (at + TC < n_new) { fetch(at + TC, stage ^ 1); dr_cp_wait<1>(); } else { dr_cp_wait<0>(); }
-        __syncthreads();
-        const float4* q4 = reinterpret_cast<const float4*>(dr_sm + stage * STAGE);
-        const float4* k4 = q4 + TC * D4;
-        const float4* g4 = k4 + TC * D4;                   // CH
-        const float* v_s = dr_sm + stage * STAGE + (CH ? 3 : 2) * TC * DS;
-        const float* b_s = v_s + TC * VT;
-        const float* g_s = b_s + TC;                       // !CH
-        const float4* kg4 = CH ? reinterpret_cast<const float4*>(kg_s) : k4;
-        // q . k of a token, (g k) . k of the token before, and g k
-        for (int t0 = 0; t0 < n; t0 += VT) {
-            const int t = t0 + col;
-            float qd = 0.f, cc = 0.f;
-            if (t < n) {
+    fetch(0);
+    fetch(1);
+    for (int chunk = 0; chunk < n_chunks; ++chunk) {
+        dr_cp_wait<1>();
+        __syncthreads();                                   // this chunk is here, and everyone is done with the one before
+        fetch(chunk + 2);
+        const float* sm = dr_sm + (chunk % DR_STAGES) * STAGE;
+        const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(sm);
+        const ulonglong2* q2 = k2 + DR_C * D4;
+        const ulonglong2* e2 = CH ? q2 + DR_C * D4 : k2;
+        const float* v_s = sm + ROWS * DR_C * DS;
+        const float* tb_s = v_s + DR_C * DR_VT;
+        const float* g_s = tb_s + DR_C * 2 * DR_C;
+        float part[16];
+        // R: the chunk's keys on the state
+#pragma unroll
+        for (int t = 0; t < DR_C; ++t) {
+            dr_f2 a0 = 0, a1 = 0;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const ulonglong2 kk = k2[t * D4 + l + DR_L * i];
+                a0 = dr_fma2(kk.x, S[0][2 * i], a0); a1 = dr_fma2(kk.x, S[1][2 * i], a1);
+                a0 = dr_fma2(kk.y, S[0][2 * i + 1], a0); a1 = dr_fma2(kk.y, S[1][2 * i + 1], a1);
+            }
+            part[2 * t] = dr_both(a0); part[2 * t + 1] = dr_both(a1);
+        }
+        float R = dr_scatter16(part, l);
+        if constexpr (!CH) R *= g_s[4 + my_t];
+        const float e = v_s[my_t * DR_VT + my_col] - R;
+        // the queries on the state, while the solution is on its way
+#pragma unroll
+        for (int t = 0; t < DR_C; ++t) {
+            dr_f2 a0 = 0, a1 = 0;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const ulonglong2 qq = q2[t * D4 + l + DR_L * i];
+                a0 = dr_fma2(qq.x, S[0][2 * i], a0); a1 = dr_fma2(qq.x, S[1][2 * i], a1);
+                a0 = dr_fma2(qq.y, S[0][2 * i + 1], a0); a1 = dr_fma2(qq.y, S[1][2 * i + 1], a1);
+            }
+            part[2 * t] = dr_both(a0); part[2 * t + 1] = dr_both(a1);
+        }
+        float o = dr_scatter16(part, l);
+        if constexpr (!CH) o *= g_s[4 + my_t];
+        // u = T e: lane (t, column) takes row t
+        float u = 0.f;
+        {
+            const float4 t0 = *reinterpret_cast<const float4*>(tb_s + my_t * 2 * DR_C);
+            const float4 t1 = *reinterpret_cast<const float4*>(tb_s + my_t * 2 * DR_C + 4);
+            const float tr[DR_C] = {t0.x, t0.y, t0.z, t0.w, t1.x, t1.y, t1.z, t1.w};
+            const int base = (lane & 16) | (l & 1);
+#pragma unroll
+            for (int j = 0; j < DR_C; ++j) u = fmaf(tr[j], __shfl_sync(0xffffffffu, e, base + 2 * j), u);
+        }
+        // o += B u, and the state: G_0n S + sum_j (G_jn k_j) u_j
+        {
+            const float4 t0 = *reinterpret_cast<const float4*>(tb_s + my_t * 2 * DR_C + DR_C);
+            const float4 t1 = *reinterpret_cast<const float4*>(tb_s + my_t * 2 * DR_C + DR_C + 4);
+            const float br[DR_C] = {t0.x, t0.y, t0.z, t0.w, t1.x, t1.y, t1.z, t1.w};
+            const float uw = CH ? u : u * g_s[4 + DR_C + my_t];
+            if constexpr (CH) {
+                const ulonglong2* gg2 = reinterpret_cast<const ulonglong2*>(g_s);
 #pragma unroll
                 for (int i = 0; i < NI; ++i) {
-                    const float4 kk = k4[t * D4 + l + L * i], qq = q4[t * D4 + l + L * i];
-                    float4 kg = kk;
-                    if constexpr (CH) {
-                        const float4 gg = g4[t * D4 + l + L * i];
-                        kg = make_float4(kk.x * gg.x, kk.y * gg.y, kk.z * gg.z, kk.w * gg.w);
-                        reinterpret_cast<float4*>(kg_s)[t * D4 + l + L * i] = kg;
-                    }
-                    qd = fmaf(qq.x, kk.x, qd); qd = fmaf(qq.y, kk.y, qd); qd = fmaf(qq.z, kk.z, qd); qd = fmaf(qq.w, kk.w, qd);
-                    if (t > 0) {
-                        const float4 kp = k4[(t - 1) * D4 + l + L * i];
-                        cc = fmaf(kg.x, kp.x, cc); cc = fmaf(kg.y, kp.y, cc); cc = fmaf(kg.z, kp.z, cc); cc = fmaf(kg.w, kp.w, cc);
+                    const ulonglong2 gg = gg2[l + DR_L * i];
+#pragma unroll
+                    for (int c = 0; c < 2; ++c) {
+                        S[c][2 * i] = dr_mul2(S[c][2 * i], gg.x);
+                        S[c][2 * i + 1] = dr_mul2(S[c][2 * i + 1], gg.y);
                     }
                 }
-            }
-            qd = dr_sum<L>(qd);
-            cc = dr_sum<L>(cc);
-            if (t < n && l == 0) {
-                qd_s[t] = qd;
-                c_s[t] = CH ? cc : cc * g_s[t];
-            }
-        }
-        __syncthreads();
-        float r, u = 0.f;
-        {
-            float p0 = 0.f, p1 = 0.f;
+            } else {
+                const dr_f2 gg = dr_pack2(g_s[0], g_s[0]);
 #pragma unroll
-            for (int i = 0; i < NI; ++i) {
-                const float4 kk = kg4[l + L * i];
-                p0 = fmaf(kk.x, S[i].x, p0); p1 = fmaf(kk.y, S[i].y, p1);
-                p0 = fmaf(kk.z, S[i].z, p0); p1 = fmaf(kk.w, S[i].w, p1);
+                for (int i = 0; i < 2 * NI; ++i) { S[0][i] = dr_mul2(S[0][i], gg); S[1][i] = dr_mul2(S[1][i], gg); }
             }
-            r = dr_sum<L>(p0 + p1);
-            if constexpr (!CH) r *= g_s[0];
-        }
-        for (int t = 0; t < n; ++t) {
-            float o0 = 0.f, o1 = 0.f, p0 = 0.f, p1 = 0.f;
-            const int tn = t + 1 < n ? t + 1 : t, tp = t > 0 ? t - 1 : 0;        // u is zero where there is no token before
-            const float gt = CH ? 0.f : g_s[t];
+            const int base = lane & 16;
 #pragma unroll
-            for (int i = 0; i < NI; ++i) {
-                const float4 kp = k4[tp * D4 + l + L * i];
-                float4 s = S[i];
-                s.x = fmaf(kp.x, u, s.x); s.y = fmaf(kp.y, u, s.y); s.z = fmaf(kp.z, u, s.z); s.w = fmaf(kp.w, u, s.w);
-                if constexpr (CH) {
-                    const float4 gg = g4[t * D4 + l + L * i];
-                    s.x *= gg.x; s.y *= gg.y; s.z *= gg.z; s.w *= gg.w;
-                } else {
-                    s.x *= gt; s.y *= gt; s.z *= gt; s.w *= gt;
+            for (int j = 0; j < DR_C; ++j) {
+                const float u0 = __shfl_sync(0xffffffffu, uw, base + 2 * j), u1 = __shfl_sync(0xffffffffu, uw, base + 2 * j + 1);
+                const dr_f2 p0 = dr_pack2(u0, u0), p1 = dr_pack2(u1, u1);
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    const ulonglong2 kk = e2[j * D4 + l + DR_L * i];
+                    S[0][2 * i] = dr_fma2(kk.x, p0, S[0][2 * i]); S[0][2 * i + 1] = dr_fma2(kk.y, p0, S[0][2 * i + 1]);
+                    S[1][2 * i] = dr_fma2(kk.x, p1, S[1][2 * i]); S[1][2 * i + 1] = dr_fma2(kk.y, p1, S[1][2 * i + 1]);
                 }
-                S[i] = s;
-                const float4 kn = kg4[tn * D4 + l + L * i], qq = q4[t * D4 + l + L * i];
-                p0 = fmaf(kn.x, s.x, p0); p1 = fmaf(kn.y, s.y, p1); p0 = fmaf(kn.z, s.z, p0); p1 = fmaf(kn.w, s.w, p1);
-                o0 = fmaf(qq.x, s.x, o0); o1 = fmaf(qq.y, s.y, o1); o0 = fmaf(qq.z, s.z, o0); o1 = fmaf(qq.w, s.w, o1);
+                if constexpr (CH) o = fmaf(br[j], (l & 1) ? u1 : u0, o);
+                else o = fmaf(br[j], __shfl_sync(0xffffffffu, u, base + (l & 1) + 2 * j), o);
             }
-            u = b_s[t] * (v_s[t * VT + col] - fmaf(c_s[t], u, r));
-            r = dr_sum<L>(p0 + p1);
-            if constexpr (!CH) r *= g_s[tn];
-            const float o = fmaf(qd_s[t], u, dr_sum<L>(o0 + o1));
-            if (l == 0) o_s[t * VT + col] = o;
         }
-        // the last token's write
-#pragma unroll
-        for (int i = 0; i < NI; ++i) {
-            const float4 kp = k4[(n - 1) * D4 + l + L * i];
-            S[i].x = fmaf(kp.x, u, S[i].x); S[i].y = fmaf(kp.y, u, S[i].y);
-            S[i].z = fmaf(kp.z, u, S[i].z); S[i].w = fmaf(kp.w, u, S[i].w);
-        }
-        __syncthreads();
-        for (int idx = tid; idx < n * VT; idx += DR_THREADS) {
-            const int j = idx / VT, c = idx - j * VT;
-            if (v0 + c < V) out[(long)(first + at + j) * out_stride + (long)h * V + v0 + c] = o_s[idx];
-        }
+        const int t = chunk * DR_C + my_t;
+        if (t < n_new && v0 + my_col < V) out[(long)(first + t) * out_stride + (long)h * V + v0 + my_col] = o;
     }
-    if (live) {
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        if (v0 + col0 + c >= V) continue;
 #pragma unroll
         for (int i = 0; i < NI; ++i)
-            if (l + L * i < d4) reinterpret_cast<float4*>(st)[l + L * i] = S[i];
+            if (l + DR_L * i < d4)
+                reinterpret_cast<ulonglong2*>(st + (long)(v0 + col0 + c) * Dp)[l + DR_L * i] =
+                    make_ulonglong2(S[c][2 * i], S[c][2 * i + 1]);
     }
 }
 
@@ -476,9 +663,8 @@ static inline bool dr_shape(int Dp, int& L, int& NI) {
     for (int ni : {1, 2, 3, 4, 6, 8})
         if (4 * 8 * ni >= Dp) { NI = ni; return true; }
     L = 32;
-    for (int ni : {4, 8})
-        if (4 * 32 * ni >= Dp) { NI = ni; return true; }
-    return false;
+    NI = 4;
+    return 4 * 32 * NI >= Dp;
 }
 
 }  // namespace zlm
@@ -496,10 +682,7 @@ using namespace zlm;
             default: F(8, 8); break;                                                                                  \
         }                                                                                                             \
     } else {                                                                                                          \
-        switch (NI) {                                                                                                 \
-            case 4: F(32, 4); break;                                                                                  \
-            default: F(32, 8); break;                                                                                 \
-        }                                                                                                             \
+        F(32, 4);                                                                                                     \
     }
 
 template <typename T>
@@ -555,32 +738,77 @@ ZLM_EXPORT int zlm_delta_prep(const void* proj, int dtype, long proj_stride, con
     return ZLM_ERR_UNSUPPORTED;
 }
 
-// state: float [slots][H][V][Dp]; out: float rows of H V numbers.
-ZLM_EXPORT int zlm_delta_scan(const float* qk, const float* v, const float* g, int channel_decay, const float* beta,
-                              float* state, const int* slots, const int* cu_seqlens, float* out, long out_stride, int n_seqs,
-                              int H, int G, int D, int V, cudaStream_t stream) {
-    if (n_seqs <= 0) return 0;
-    if (H <= 0 || G <= 0 || H % G || D <= 0 || V <= 0) return ZLM_ERR_BAD_ARG;
-    const int Dp = (D + 3) / 4 * 4, Vp = (V + 3) / 4 * 4;
-    int L, NI;
-    if (!dr_shape(Dp, L, NI) || H > 65535 || n_seqs > 65535) return ZLM_ERR_UNSUPPORTED;
-    const int VT = DR_THREADS / L;
-    dim3 grid((V + VT - 1) / VT, H, n_seqs);
-    const size_t smem = dr_scan_floats(L, NI, channel_decay != 0) * sizeof(float);
-    cudaError_t e = cudaSuccess;
-#define ZLM_DR_SCAN(LL, NN)                                                                                            \
+// The float4 a lane of DR_L holds of a row of Dp elements, or 0: too long.
+static inline int dr_scan_ni(int Dp) {
+    for (int ni : {1, 2, 3, 4, 8})
+        if (4 * DR_L * ni >= Dp) return ni;
+    return 0;
+}
+
+#define ZLM_DR_NI(F)                                                                                                   \
+    switch (ni) {                                                                                                      \
+        case 1: F(1); break;                                                                                           \
+        case 2: F(2); break;                                                                                           \
+        case 3: F(3); break;                                                                                           \
+        case 4: F(4); break;                                                                                           \
+        default: F(8); break;                                                                                          \
+    }
+// Launch kernel k with smem bytes of shared memory, raising its limit once.
+#define ZLM_DR_RAISED(k, which, grid, ...)                                                                             \
     do {                                                                                                               \
-        auto* k = channel_decay ? dr_scan_kernel<LL, NN, true> : dr_scan_kernel<LL, NN, false>;                        \
-        static size_t raised[2] = {0, 0};                                                                              \
-        if (smem > 48 * 1024 && raised[channel_decay ? 1 : 0] < smem) {                                                \
+        static size_t raised[2] = {40 * 1024, 40 * 1024};                                                              \
+        if (raised[which] < smem) {                                                                                    \
             e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                       \
             if (e != cudaSuccess) return (int)e;                                                                       \
-            raised[channel_decay ? 1 : 0] = smem;                                                                      \
+            raised[which] = smem;                                                                                      \
         }                                                                                                              \
-        e = launch_pdl(k, grid, dim3(DR_THREADS), smem, stream, qk, v, g, beta, state, slots, cu_seqlens, out, out_stride, H, \
-                       G, Dp, V, Vp);                                                                                  \
+        e = launch_pdl(k, grid, dim3(DR_THREADS), smem, stream, __VA_ARGS__);                                          \
     } while (0)
-    ZLM_DR_SHAPES(ZLM_DR_SCAN)
+
+// What a chunk contributes apart from the state (see dr_chunk_kernel for the operands; we null: one decay a head).
+ZLM_EXPORT int zlm_delta_chunk(const float* qk, const float* g, int channel_decay, const float* beta, const int* cu_seqlens,
+                               float* wk, float* wq, float* we, float* ws, float* gam, float* tb, int n_seqs, int max_new,
+                               int H, int G, int D, cudaStream_t stream) {
+    if (n_seqs <= 0 || max_new <= 0) return 0;
+    if (H <= 0 || G <= 0 || H % G || D <= 0) return ZLM_ERR_BAD_ARG;
+    const int Dp = (D + 3) / 4 * 4, ni = dr_scan_ni(Dp), which = channel_decay ? 1 : 0;
+    if (ni == 0 || H > 65535 || n_seqs > 65535) return ZLM_ERR_UNSUPPORTED;
+    const size_t smem = (size_t)DR_C * 64 * ni * (which ? 3 : 2) * sizeof(float);
+    dim3 grid((max_new + DR_C - 1) / DR_C, H, n_seqs);
+    cudaError_t e = cudaSuccess;
+#define ZLM_DR_CHUNK(NN)                                                                                               \
+    do {                                                                                                               \
+        auto* k = which ? dr_chunk_kernel<NN, true> : dr_chunk_kernel<NN, false>;                                      \
+        ZLM_DR_RAISED(k, which, grid, qk, g, beta, cu_seqlens, wk, wq, we, ws, gam, tb, H, G, Dp);                     \
+    } while (0)
+    ZLM_DR_NI(ZLM_DR_CHUNK)
+#undef ZLM_DR_CHUNK
+    return e == cudaSuccess ? launch_status() : (int)e;
+}
+
+// The tokens of a chunk, and the chunks a step of T tokens of n_seqs sequences can have at most (sizes ``gam``).
+ZLM_EXPORT int zlm_delta_chunks(int T, int n_seqs) { return T / DR_C + n_seqs + 1; }
+ZLM_EXPORT int zlm_delta_chunk_tokens() { return DR_C; }
+
+// state: float [slots][H][V][Dp]; out: float rows of H V numbers; the other operands as dr_chunk left them.
+ZLM_EXPORT int zlm_delta_scan(const float* kr, const float* qr, const float* er, const float* ws, const float* gam,
+                              const float* tb, const float* v, int channel_decay, float* state, const int* slots,
+                              const int* cu_seqlens, float* out, long out_stride, int n_seqs, int H, int G, int D, int V,
+                              cudaStream_t stream) {
+    if (n_seqs <= 0) return 0;
+    if (H <= 0 || G <= 0 || H % G || D <= 0 || V <= 0) return ZLM_ERR_BAD_ARG;
+    const int Dp = (D + 3) / 4 * 4, Vp = (V + 3) / 4 * 4, ni = dr_scan_ni(Dp), which = channel_decay ? 1 : 0;
+    if (ni == 0 || H > 65535 || n_seqs > 65535) return ZLM_ERR_UNSUPPORTED;
+    dim3 grid((V + DR_VT - 1) / DR_VT, H, n_seqs);
+    const size_t smem = (size_t)DR_STAGES * dr_stage(ni, which != 0) * sizeof(float);
+    if (smem > 227 * 1024) return ZLM_ERR_UNSUPPORTED;
+    cudaError_t e = cudaSuccess;
+#define ZLM_DR_SCAN(NN)                                                                                                \
+    do {                                                                                                               \
+        auto* k = which ? dr_scan_kernel<NN, true> : dr_scan_kernel<NN, false>;                                        \
+        ZLM_DR_RAISED(k, which, grid, kr, qr, er, ws, gam, tb, v, state, slots, cu_seqlens, out, out_stride, H, G, Dp, V, Vp); \
+    } while (0)
+    ZLM_DR_NI(ZLM_DR_SCAN)
 #undef ZLM_DR_SCAN
     return e == cudaSuccess ? launch_status() : (int)e;
 }

@@ -57,8 +57,8 @@ class GatedDeltaRule(Part):
             raise ValueError(f"gated_delta_rule: {self.n_heads} heads cannot share {self.n_kv} heads of q and k")
         if min(self.dim, self.value_dim, self.taps) <= 0:
             raise ValueError("gated_delta_rule: key size, value size and taps must be positive")
-        if self.dim > 1024:
-            raise ValueError(f"gated_delta_rule: keys of {self.dim} elements are not supported (at most 1024)")
+        if self.dim > 512:
+            raise ValueError(f"gated_delta_rule: keys of {self.dim} elements are not supported (at most 512)")
         self.decay = o.get("decay", "head")
         if self.decay not in ("head", "channel"):
             raise ValueError(f"gated_delta_rule: decay {self.decay!r} is not known (head, channel)")
