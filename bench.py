@@ -1202,12 +1202,12 @@ def run_mopilorn(args):
             ms = timed(lambda: kernels.delta_prep(*args_d, step))
             report(f"delta_prep ({H} heads of {D}, {kind}), {tag}", "causal_conv", ms,
                    n_tok * (C * 6 + H * per * 8 + H * 8), 0)
-            chunks = kernels.delta_chunk(made[0], made[2], made[3], H, G, D, step)
+            records = kernels.delta_chunk(made[0], made[2], made[3], H, G, D, step)
             ms = timed(lambda: kernels.delta_chunk(made[0], made[2], made[3], H, G, D, step))
-            moved = (3 * H * D * 4) if per > 1 else H * 8
+            moved = 3 * H * D * 4
             report(f"delta_chunk ({H} heads of {D}, {kind}), {tag}", "causal_conv", ms,
                    n_tok * (2 * G * D * 4 + H * per * 4 + moved + H * 64), 0)
-            ms = timed(lambda: kernels.delta_scan(made[0], made[1], chunks, H, G, D, V, dst, step, mixed))
+            ms = timed(lambda: kernels.delta_scan(records, made[1], H, D, V, dst, step, mixed))
             report(f"delta_scan ({H} heads of {D}, {kind}), {tag}", "decayed_linear_attention", ms,
                    state_bytes + n_tok * (C * 4 + H * per * 4 + H * V * 4), 0, rule_fma)
         z = f32(batch, vocab)

@@ -203,16 +203,17 @@ template <int L> __device__ __forceinline__ float dr_sum(float v) {
 // The place of a chunk among all chunks of the step: sequence b's chunks lie behind those of the sequences before it.
 __device__ __forceinline__ long dr_chunk_index(int first, int b, int chunk) { return (long)(first / DR_C) + b + chunk; }
 
+// What dr_chunk leaves of a (chunk, head), in floats, rows padded with zeros to DS elements:
+//   G_0t k_t [DR_C][DS], G_0t q_t [DR_C][DS], G_jn k_j [DR_C][DS], G_0n [DS], then per token its row of T and of B [DR_C][2 DR_C]
+// Tokens behind the end of a short chunk are zero in all of them.
+__host__ __device__ constexpr int dr_record(int NI) { return (3 * DR_C + 1) * 64 * NI + 2 * DR_C * DR_C; }
+
 // grid (chunks of the longest sequence, heads, sequences); thread (j, l): token j of the chunk, lane l of its D elements.
-// qk: float [T][2 G][Dp]; g: [T][H][Dp] (CH) or [T][H]; beta: [T][H].
-// wk, wq, we: float [T][H][Dp], the chunk's weighted keys and queries G_0t k_t, G_0t q_t and G_jn k_j (CH);
-// ws: float [T][H][2], G_0t and G_jn (not CH).  gam: [chunks][H][Dp] or [chunks][H], G_0n.
-// tb: float [T][H][2 DR_C], row t of T, then row t of B; rows behind the chunk's last token are not written.
+// qk: float [T][2 G][Dp]; g: [T][H][Dp] (CH) or [T][H]; beta: [T][H]; rec: [chunks][H] records.
 template <int NI, bool CH>
 __global__ void __launch_bounds__(DR_THREADS)
 dr_chunk_kernel(const float* __restrict__ qk, const float* __restrict__ g, const float* __restrict__ beta,
-                const int* __restrict__ cu_seqlens, float* __restrict__ wk, float* __restrict__ wq, float* __restrict__ we,
-                float* __restrict__ ws, float* __restrict__ gam, float* __restrict__ tb, int H, int G, int Dp) {
+                const int* __restrict__ cu_seqlens, float* __restrict__ rec, int H, int G, int Dp) {
     constexpr int D4 = DR_L * NI;                          // float4 of a padded row
     extern __shared__ __align__(16) float dr_sm[];
     float4* k4 = reinterpret_cast<float4*>(dr_sm);         // [DR_C][D4]
@@ -227,12 +228,14 @@ dr_chunk_kernel(const float* __restrict__ qk, const float* __restrict__ g, const
     const int tid = threadIdx.x, j = tid / DR_L, l = tid % DR_L, d4 = Dp / 4;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     const long t0 = first + at;
-    for (int idx = tid; idx < DR_C * D4; idx += DR_THREADS) {
-        const int t = idx / D4, i = idx - t * D4;
-        const bool in = t < n && i < d4;
-        k4[idx] = in ? reinterpret_cast<const float4*>(qk + ((t0 + t) * 2 * G + G + kv) * Dp)[i] : zero;
-        q4[idx] = in ? reinterpret_cast<const float4*>(qk + ((t0 + t) * 2 * G + kv) * Dp)[i] : zero;
-        if constexpr (CH) g4[idx] = in ? reinterpret_cast<const float4*>(g + ((t0 + t) * H + h) * Dp)[i] : zero;
+    // a token's row by the lanes that work on it
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const int c = l + DR_L * i;
+        const bool in = j < n && c < d4;
+        k4[j * D4 + c] = in ? reinterpret_cast<const float4*>(qk + ((t0 + j) * 2 * G + G + kv) * Dp)[c] : zero;
+        q4[j * D4 + c] = in ? reinterpret_cast<const float4*>(qk + ((t0 + j) * 2 * G + kv) * Dp)[c] : zero;
+        if constexpr (CH) g4[j * D4 + c] = in ? reinterpret_cast<const float4*>(g + ((t0 + j) * H + h) * Dp)[c] : zero;
     }
     if (tid < DR_C) {
         beta_s[tid] = tid < n ? beta[(t0 + tid) * H + h] : 0.f;
@@ -246,7 +249,6 @@ dr_chunk_kernel(const float* __restrict__ qk, const float* __restrict__ g, const
 #pragma unroll
     for (int i = 0; i < NI; ++i) w[i] = k4[j * D4 + l + DR_L * i];
     for (int t = 0; t < n; ++t) {                          // every thread takes every round: shuffles inside
-        const bool on = t >= j;
         float ka = 0.f, qa = 0.f;
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
@@ -263,16 +265,18 @@ dr_chunk_kernel(const float* __restrict__ qk, const float* __restrict__ g, const
         if constexpr (!CH) { if (t > j) wsc *= g_s[t]; }
         ka = dr_sum<DR_L>(ka);
         qa = dr_sum<DR_L>(qa);
-        if (on && l == 0) {
+        if (t >= j && l == 0) {
             b_s[t][j] = qa * wsc;
             if (t > j) a_s[t][j] = beta_s[t] * (ka * wsc);
         }
     }
-    if (j < n) {
-        const long row = (t0 + j) * H + h;
+    float4* r4 = reinterpret_cast<float4*>(rec + (dr_chunk_index(first, b, blockIdx.x) * H + h) * dr_record(NI));
+    {
+        // decays from the state to token j, and from token j to the chunk's end (what w has become); a row behind a short
+        // chunk's last token is zero because its k and q are
+        float4 G0[NI];
+        float g0 = 1.f;
         if constexpr (CH) {
-            // from the state to token j, and from token j to the chunk's end (what w has become)
-            float4 G0[NI];
 #pragma unroll
             for (int i = 0; i < NI; ++i) G0[i] = g4[l + DR_L * i];
             for (int t = 1; t <= j; ++t) {
@@ -282,28 +286,23 @@ dr_chunk_kernel(const float* __restrict__ qk, const float* __restrict__ g, const
                     G0[i].x *= gg.x; G0[i].y *= gg.y; G0[i].z *= gg.z; G0[i].w *= gg.w;
                 }
             }
-#pragma unroll
-            for (int i = 0; i < NI; ++i) {
-                if (l + DR_L * i >= d4) continue;
-                const float4 kk = k4[j * D4 + l + DR_L * i], qq = q4[j * D4 + l + DR_L * i];
-                reinterpret_cast<float4*>(wk + row * Dp)[l + DR_L * i] =
-                    make_float4(G0[i].x * kk.x, G0[i].y * kk.y, G0[i].z * kk.z, G0[i].w * kk.w);
-                reinterpret_cast<float4*>(wq + row * Dp)[l + DR_L * i] =
-                    make_float4(G0[i].x * qq.x, G0[i].y * qq.y, G0[i].z * qq.z, G0[i].w * qq.w);
-                reinterpret_cast<float4*>(we + row * Dp)[l + DR_L * i] = w[i];
-                if (j == n - 1)
-                    reinterpret_cast<float4*>(gam + (dr_chunk_index(first, b, blockIdx.x) * H + h) * Dp)[l + DR_L * i] = G0[i];
-            }
-        } else if (l == 0) {
-            float g0 = 1.f;
+        } else {
             for (int t = 0; t <= j; ++t) g0 *= g_s[t];
-            ws[row * 2] = g0;
-            ws[row * 2 + 1] = wsc;
-            if (j == n - 1) gam[dr_chunk_index(first, b, blockIdx.x) * H + h] = g0;
+        }
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int c = j * D4 + l + DR_L * i;
+            const float4 gg = CH ? G0[i] : make_float4(g0, g0, g0, g0);
+            const float4 kk = k4[c], qq = q4[c];
+            r4[c] = make_float4(gg.x * kk.x, gg.y * kk.y, gg.z * kk.z, gg.w * kk.w);
+            r4[DR_C * D4 + c] = make_float4(gg.x * qq.x, gg.y * qq.y, gg.z * qq.z, gg.w * qq.w);
+            r4[2 * DR_C * D4 + c] = make_float4(w[i].x * wsc, w[i].y * wsc, w[i].z * wsc, w[i].w * wsc);
+            if (j == n - 1) r4[3 * DR_C * D4 + l + DR_L * i] = gg;
         }
     }
     __syncthreads();
     // column c of T: (I + A) x = beta_c e_c, downwards
+    float* tb = reinterpret_cast<float*>(r4 + (3 * DR_C + 1) * D4);
     if (tid < DR_C) {
         float x[DR_C];
 #pragma unroll
@@ -312,11 +311,11 @@ dr_chunk_kernel(const float* __restrict__ qk, const float* __restrict__ g, const
 #pragma unroll
             for (int u = 0; u < t; ++u) acc = fmaf(-a_s[t][u], x[u], acc);
             x[t] = acc;
-            if (t < n) tb[((t0 + t) * H + h) * (2 * DR_C) + tid] = acc;
+            tb[t * 2 * DR_C + tid] = acc;                  // behind the last token: beta and A are zero, so is T
         }
     } else if (tid >= 64) {
         const int i = tid - 64, t = i / DR_C;
-        if (t < n) tb[((t0 + t) * H + h) * (2 * DR_C) + DR_C + i % DR_C] = b_s[t][i % DR_C];
+        tb[t * 2 * DR_C + DR_C + i % DR_C] = b_s[t][i % DR_C];
     }
 }
 
@@ -343,8 +342,9 @@ __device__ __forceinline__ float dr_both(dr_f2 v) {
     return x + y;
 }
 
-// The sums over 16 lanes of 16 numbers a lane, scattered: lane m is left with the sum of number m.
-__device__ __forceinline__ float dr_scatter16(float (&a)[16], int l) {
+// The sums over 16 lanes of 16 numbers a lane, scattered: lane m is left with the sum of number m in a[0].  Two sets side
+// by side, so that the rounds of one hide those of the other.
+__device__ __forceinline__ void dr_scatter16(float (&a)[16], float (&b)[16], int l) {
 #pragma unroll
     for (int o = 8; o > 0; o >>= 1) {
         const bool up = (l & o) != 0;
@@ -353,34 +353,34 @@ __device__ __forceinline__ float dr_scatter16(float (&a)[16], int l) {
             const float give = up ? a[i] : a[i + o], keep = up ? a[i + o] : a[i];
             a[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
         }
+#pragma unroll
+        for (int i = 0; i < o; ++i) {
+            const float give = up ? b[i] : b[i + o], keep = up ? b[i + o] : b[i];
+            b[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
     }
-    return a[0];
 }
 
 constexpr int DR_STAGES = 3;
-// floats of a stage: the rows k, q (and, with a decay a channel, the keys for the state), the values, T and B, the decays
-__host__ __device__ constexpr int dr_stage(int NI, bool ch) {
-    return DR_C * (64 * NI * (ch ? 3 : 2) + DR_VT + 2 * DR_C + (ch ? 0 : 2)) + (ch ? 64 * NI : 4);
-}
+// floats of a stage: the chunk's record and its values
+__host__ __device__ constexpr int dr_stage(int NI) { return dr_record(NI) + DR_C * DR_VT; }
 
-// grid (value tiles, heads, sequences).  CH: kr, qr, er are wk, wq, we of dr_chunk (rows [T][H][Dp]); else kr is qk (rows
-// [T][2 G][Dp]) and ws holds the weights.  v: [T][H][Vp]; out: float rows of H V numbers.
-template <int NI, bool CH>
+// grid (value tiles, heads, sequences).  rec: the records of dr_chunk; v: [T][H][Vp]; out: float rows of H V numbers.
+template <int NI>
 __global__ void __launch_bounds__(DR_THREADS)
-dr_scan_kernel(const float* __restrict__ kr, const float* __restrict__ qr, const float* __restrict__ er,
-               const float* __restrict__ ws, const float* __restrict__ gam, const float* __restrict__ tb,
-               const float* __restrict__ v, float* __restrict__ state, const int* __restrict__ slots,
-               const int* __restrict__ cu_seqlens, float* __restrict__ out, long out_stride, int H, int G, int Dp, int V,
-               int Vp) {
-    constexpr int DS = 64 * NI, D4 = DS / 4, STAGE = dr_stage(NI, CH), ROWS = CH ? 3 : 2;
+dr_scan_kernel(const float* __restrict__ rec, const float* __restrict__ v, float* __restrict__ state,
+               const int* __restrict__ slots, const int* __restrict__ cu_seqlens, float* __restrict__ out, long out_stride, int H,
+               int Dp, int V, int Vp) {
+    constexpr int D4 = 16 * NI, STAGE = dr_stage(NI), RECORD = dr_record(NI);
     extern __shared__ __align__(16) float dr_sm[];
     const int tid = threadIdx.x, lane = tid & 31, l = lane & 15;
     const int b = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * DR_VT;
-    const int kv = h / (H / G), d4 = Dp / 4;
+    const int d4 = Dp / 4;
     const int col0 = (tid >> 5) * 4 + (lane >> 4) * 2;      // this lane's two columns of the tile
     const int my_t = l >> 1, my_col = col0 + (l & 1);       // what the scattered sums leave this lane with
-    // what stands behind the live elements of a row, and behind a short chunk's last token, is zero or finite
-    for (int i = tid; i < DR_STAGES * STAGE; i += DR_THREADS) dr_sm[i] = 0.f;
+    // values that are never fetched (behind a short chunk's last token, behind the last column) meet zeros: finite they must be
+    for (int i = tid; i < DR_STAGES * DR_C * DR_VT; i += DR_THREADS)
+        dr_sm[(i / (DR_C * DR_VT)) * STAGE + RECORD + i % (DR_C * DR_VT)] = 0.f;
     float* st = state + ((long)slots[b] * H + h) * V * Dp;
     dr_f2 S[2][2 * NI];
 #pragma unroll
@@ -397,46 +397,18 @@ dr_scan_kernel(const float* __restrict__ kr, const float* __restrict__ qr, const
     __syncthreads();
     const int first = cu_seqlens[b], n_new = cu_seqlens[b + 1] - first;
     const int n_chunks = (n_new + DR_C - 1) / DR_C;
+    const float* recs = rec + (dr_chunk_index(first, b, 0) * H + h) * RECORD;
+    const int vj = tid / (DR_VT / 4), vi = 4 * (tid % (DR_VT / 4));            // what a thread fetches of the values
+    const float* vsrc = v + ((first + vj) * (long)H + h) * Vp + v0 + vi;
     auto fetch = [&](int chunk) {
         if (chunk < n_chunks) {
             float* sm = dr_sm + (chunk % DR_STAGES) * STAGE;
-            const int at = chunk * DR_C, n = min(DR_C, n_new - at);
-            for (int idx = tid; idx < n * d4; idx += DR_THREADS) {
-                const int j = idx / d4, i = 4 * (idx - j * d4);
-                const long t = first + at + j;
-                if constexpr (CH) {
-                    dr_cp16(sm + j * DS + i, kr + (t * H + h) * Dp + i);
-                    dr_cp16(sm + (DR_C + j) * DS + i, qr + (t * H + h) * Dp + i);
-                    dr_cp16(sm + (2 * DR_C + j) * DS + i, er + (t * H + h) * Dp + i);
-                } else {
-                    dr_cp16(sm + j * DS + i, kr + (t * 2 * G + G + kv) * Dp + i);
-                    dr_cp16(sm + (DR_C + j) * DS + i, kr + (t * 2 * G + kv) * Dp + i);
-                }
-            }
-            float* v_s = sm + ROWS * DR_C * DS;
-            if (tid < n * (DR_VT / 4)) {
-                const int j = tid / (DR_VT / 4), i = 4 * (tid % (DR_VT / 4));
-                if (v0 + i < Vp) dr_cp16(v_s + j * DR_VT + i, v + ((first + at + j) * (long)H + h) * Vp + v0 + i);
-            }
-            float* tb_s = v_s + DR_C * DR_VT;
-            if (tid >= 64 && tid - 64 < n * (2 * DR_C / 4)) {
-                const int j = (tid - 64) / (2 * DR_C / 4), i = 4 * ((tid - 64) % (2 * DR_C / 4));
-                dr_cp16(tb_s + j * 2 * DR_C + i, tb + ((first + at + j) * (long)H + h) * (2 * DR_C) + i);
-            }
-            float* g_s = tb_s + DR_C * 2 * DR_C;
-            const float* gsrc = gam + (dr_chunk_index(first, b, chunk) * H + h) * (CH ? Dp : 1);
-            if constexpr (CH) {
-                for (int i = tid; i < d4; i += DR_THREADS) dr_cp16(g_s + 4 * i, gsrc + 4 * i);
-            } else {
-                if (tid == 0) g_s[0] = gsrc[0];
-                if (tid >= 32 && tid - 32 < n) {
-                    const float* w = ws + ((first + at + tid - 32) * (long)H + h) * 2;
-                    g_s[4 + tid - 32] = w[0];
-                    g_s[4 + DR_C + tid - 32] = w[1];
-                }
-            }
-            // a short chunk: the rows of T and B behind its last token must be zero
-            if (n < DR_C) for (int i = n * 2 * DR_C + tid; i < DR_C * 2 * DR_C; i += DR_THREADS) tb_s[i] = 0.f;
+            const float* src = recs + (long)chunk * H * RECORD;
+#pragma unroll
+            for (int i = 0; i < RECORD / 4; i += DR_THREADS)
+                if (i + tid < RECORD / 4) dr_cp16(sm + 4 * (i + tid), src + 4 * (i + tid));
+            if (vj < min(DR_C, n_new - chunk * DR_C) && v0 + vi < Vp)
+                dr_cp16(sm + RECORD + vj * DR_VT + vi, vsrc + (long)chunk * DR_C * H * Vp);
         }
         dr_cp_commit();
     };
@@ -447,47 +419,45 @@ dr_scan_kernel(const float* __restrict__ kr, const float* __restrict__ qr, const
         __syncthreads();                                   // this chunk is here, and everyone is done with the one before
         fetch(chunk + 2);
         const float* sm = dr_sm + (chunk % DR_STAGES) * STAGE;
-        const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(sm);
+        const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(sm) + l;
         const ulonglong2* q2 = k2 + DR_C * D4;
-        const ulonglong2* e2 = CH ? q2 + DR_C * D4 : k2;
-        const float* v_s = sm + ROWS * DR_C * DS;
-        const float* tb_s = v_s + DR_C * DR_VT;
-        const float* g_s = tb_s + DR_C * 2 * DR_C;
-        float part[16];
-        // R: the chunk's keys on the state
+        const ulonglong2* e2 = q2 + DR_C * D4;
+        const ulonglong2* g2 = e2 + DR_C * D4;
+        const float* tb_s = sm + (3 * DR_C + 1) * 4 * D4 + my_t * 2 * DR_C;      // this lane's row of T, then of B
+        float R[16], O[16];
+        // the chunk's keys and queries on the state
 #pragma unroll
         for (int t = 0; t < DR_C; ++t) {
-            dr_f2 a0 = 0, a1 = 0;
+            dr_f2 r0 = 0, r1 = 0, o0 = 0, o1 = 0;
 #pragma unroll
             for (int i = 0; i < NI; ++i) {
-                const ulonglong2 kk = k2[t * D4 + l + DR_L * i];
-                a0 = dr_fma2(kk.x, S[0][2 * i], a0); a1 = dr_fma2(kk.x, S[1][2 * i], a1);
-                a0 = dr_fma2(kk.y, S[0][2 * i + 1], a0); a1 = dr_fma2(kk.y, S[1][2 * i + 1], a1);
+                const ulonglong2 kk = k2[t * D4 + DR_L * i], qq = q2[t * D4 + DR_L * i];
+                r0 = dr_fma2(kk.x, S[0][2 * i], r0); r1 = dr_fma2(kk.x, S[1][2 * i], r1);
+                o0 = dr_fma2(qq.x, S[0][2 * i], o0); o1 = dr_fma2(qq.x, S[1][2 * i], o1);
+                r0 = dr_fma2(kk.y, S[0][2 * i + 1], r0); r1 = dr_fma2(kk.y, S[1][2 * i + 1], r1);
+                o0 = dr_fma2(qq.y, S[0][2 * i + 1], o0); o1 = dr_fma2(qq.y, S[1][2 * i + 1], o1);
             }
-            part[2 * t] = dr_both(a0); part[2 * t + 1] = dr_both(a1);
+            R[2 * t] = dr_both(r0); R[2 * t + 1] = dr_both(r1);
+            O[2 * t] = dr_both(o0); O[2 * t + 1] = dr_both(o1);
         }
-        float R = dr_scatter16(part, l);
-        if constexpr (!CH) R *= g_s[4 + my_t];
-        const float e = v_s[my_t * DR_VT + my_col] - R;
-        // the queries on the state, while the solution is on its way
+        // the state before the chunk's writes
 #pragma unroll
-        for (int t = 0; t < DR_C; ++t) {
-            dr_f2 a0 = 0, a1 = 0;
+        for (int i = 0; i < NI; ++i) {
+            const ulonglong2 gg = g2[DR_L * i];
 #pragma unroll
-            for (int i = 0; i < NI; ++i) {
-                const ulonglong2 qq = q2[t * D4 + l + DR_L * i];
-                a0 = dr_fma2(qq.x, S[0][2 * i], a0); a1 = dr_fma2(qq.x, S[1][2 * i], a1);
-                a0 = dr_fma2(qq.y, S[0][2 * i + 1], a0); a1 = dr_fma2(qq.y, S[1][2 * i + 1], a1);
+            for (int c = 0; c < 2; ++c) {
+                S[c][2 * i] = dr_mul2(S[c][2 * i], gg.x);
+                S[c][2 * i + 1] = dr_mul2(S[c][2 * i + 1], gg.y);
             }
-            part[2 * t] = dr_both(a0); part[2 * t + 1] = dr_both(a1);
         }
-        float o = dr_scatter16(part, l);
-        if constexpr (!CH) o *= g_s[4 + my_t];
+        const float vv = sm[RECORD + my_t * DR_VT + my_col];
+        dr_scatter16(R, O, l);
+        const float e = vv - R[0];
+        float o = O[0];
         // u = T e: lane (t, column) takes row t
         float u = 0.f;
         {
-            const float4 t0 = *reinterpret_cast<const float4*>(tb_s + my_t * 2 * DR_C);
-            const float4 t1 = *reinterpret_cast<const float4*>(tb_s + my_t * 2 * DR_C + 4);
+            const float4 t0 = *reinterpret_cast<const float4*>(tb_s), t1 = *reinterpret_cast<const float4*>(tb_s + 4);
             const float tr[DR_C] = {t0.x, t0.y, t0.z, t0.w, t1.x, t1.y, t1.z, t1.w};
             const int base = (lane & 16) | (l & 1);
 #pragma unroll
@@ -495,39 +465,20 @@ dr_scan_kernel(const float* __restrict__ kr, const float* __restrict__ qr, const
         }
         // o += B u, and the state: G_0n S + sum_j (G_jn k_j) u_j
         {
-            const float4 t0 = *reinterpret_cast<const float4*>(tb_s + my_t * 2 * DR_C + DR_C);
-            const float4 t1 = *reinterpret_cast<const float4*>(tb_s + my_t * 2 * DR_C + DR_C + 4);
+            const float4 t0 = *reinterpret_cast<const float4*>(tb_s + DR_C), t1 = *reinterpret_cast<const float4*>(tb_s + DR_C + 4);
             const float br[DR_C] = {t0.x, t0.y, t0.z, t0.w, t1.x, t1.y, t1.z, t1.w};
-            const float uw = CH ? u : u * g_s[4 + DR_C + my_t];
-            if constexpr (CH) {
-                const ulonglong2* gg2 = reinterpret_cast<const ulonglong2*>(g_s);
-#pragma unroll
-                for (int i = 0; i < NI; ++i) {
-                    const ulonglong2 gg = gg2[l + DR_L * i];
-#pragma unroll
-                    for (int c = 0; c < 2; ++c) {
-                        S[c][2 * i] = dr_mul2(S[c][2 * i], gg.x);
-                        S[c][2 * i + 1] = dr_mul2(S[c][2 * i + 1], gg.y);
-                    }
-                }
-            } else {
-                const dr_f2 gg = dr_pack2(g_s[0], g_s[0]);
-#pragma unroll
-                for (int i = 0; i < 2 * NI; ++i) { S[0][i] = dr_mul2(S[0][i], gg); S[1][i] = dr_mul2(S[1][i], gg); }
-            }
             const int base = lane & 16;
 #pragma unroll
             for (int j = 0; j < DR_C; ++j) {
-                const float u0 = __shfl_sync(0xffffffffu, uw, base + 2 * j), u1 = __shfl_sync(0xffffffffu, uw, base + 2 * j + 1);
+                const float u0 = __shfl_sync(0xffffffffu, u, base + 2 * j), u1 = __shfl_sync(0xffffffffu, u, base + 2 * j + 1);
                 const dr_f2 p0 = dr_pack2(u0, u0), p1 = dr_pack2(u1, u1);
 #pragma unroll
                 for (int i = 0; i < NI; ++i) {
-                    const ulonglong2 kk = e2[j * D4 + l + DR_L * i];
+                    const ulonglong2 kk = e2[j * D4 + DR_L * i];
                     S[0][2 * i] = dr_fma2(kk.x, p0, S[0][2 * i]); S[0][2 * i + 1] = dr_fma2(kk.y, p0, S[0][2 * i + 1]);
                     S[1][2 * i] = dr_fma2(kk.x, p1, S[1][2 * i]); S[1][2 * i + 1] = dr_fma2(kk.y, p1, S[1][2 * i + 1]);
                 }
-                if constexpr (CH) o = fmaf(br[j], (l & 1) ? u1 : u0, o);
-                else o = fmaf(br[j], __shfl_sync(0xffffffffu, u, base + (l & 1) + 2 * j), o);
+                o = fmaf(br[j], (l & 1) ? u1 : u0, o);
             }
         }
         const int t = chunk * DR_C + my_t;
@@ -765,10 +716,10 @@ static inline int dr_scan_ni(int Dp) {
         e = launch_pdl(k, grid, dim3(DR_THREADS), smem, stream, __VA_ARGS__);                                          \
     } while (0)
 
-// What a chunk contributes apart from the state (see dr_chunk_kernel for the operands; we null: one decay a head).
+// What every chunk contributes apart from the state: rec, float [zlm_delta_chunks][H][zlm_delta_record] (dr_chunk_kernel).
+// g: [T][H][Dp] (channel_decay) or [T][H].
 ZLM_EXPORT int zlm_delta_chunk(const float* qk, const float* g, int channel_decay, const float* beta, const int* cu_seqlens,
-                               float* wk, float* wq, float* we, float* ws, float* gam, float* tb, int n_seqs, int max_new,
-                               int H, int G, int D, cudaStream_t stream) {
+                               float* rec, int n_seqs, int max_new, int H, int G, int D, cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || D <= 0) return ZLM_ERR_BAD_ARG;
     const int Dp = (D + 3) / 4 * 4, ni = dr_scan_ni(Dp), which = channel_decay ? 1 : 0;
@@ -779,34 +730,35 @@ ZLM_EXPORT int zlm_delta_chunk(const float* qk, const float* g, int channel_deca
 #define ZLM_DR_CHUNK(NN)                                                                                               \
     do {                                                                                                               \
         auto* k = which ? dr_chunk_kernel<NN, true> : dr_chunk_kernel<NN, false>;                                      \
-        ZLM_DR_RAISED(k, which, grid, qk, g, beta, cu_seqlens, wk, wq, we, ws, gam, tb, H, G, Dp);                     \
+        ZLM_DR_RAISED(k, which, grid, qk, g, beta, cu_seqlens, rec, H, G, Dp);                                         \
     } while (0)
     ZLM_DR_NI(ZLM_DR_CHUNK)
 #undef ZLM_DR_CHUNK
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 
-// The tokens of a chunk, and the chunks a step of T tokens of n_seqs sequences can have at most (sizes ``gam``).
+// The most chunks a step of T tokens of n_seqs sequences can have, and the floats of a record for keys of D elements (0: too
+// long).
 ZLM_EXPORT int zlm_delta_chunks(int T, int n_seqs) { return T / DR_C + n_seqs + 1; }
-ZLM_EXPORT int zlm_delta_chunk_tokens() { return DR_C; }
+ZLM_EXPORT int zlm_delta_record(int D) {
+    const int ni = dr_scan_ni((D + 3) / 4 * 4);
+    return ni ? dr_record(ni) : 0;
+}
 
-// state: float [slots][H][V][Dp]; out: float rows of H V numbers; the other operands as dr_chunk left them.
-ZLM_EXPORT int zlm_delta_scan(const float* kr, const float* qr, const float* er, const float* ws, const float* gam,
-                              const float* tb, const float* v, int channel_decay, float* state, const int* slots,
-                              const int* cu_seqlens, float* out, long out_stride, int n_seqs, int H, int G, int D, int V,
-                              cudaStream_t stream) {
+// state: float [slots][H][V][Dp]; v: [T][H][Vp]; out: float rows of H V numbers.
+ZLM_EXPORT int zlm_delta_scan(const float* rec, const float* v, float* state, const int* slots, const int* cu_seqlens,
+                              float* out, long out_stride, int n_seqs, int H, int D, int V, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
-    if (H <= 0 || G <= 0 || H % G || D <= 0 || V <= 0) return ZLM_ERR_BAD_ARG;
-    const int Dp = (D + 3) / 4 * 4, Vp = (V + 3) / 4 * 4, ni = dr_scan_ni(Dp), which = channel_decay ? 1 : 0;
+    if (H <= 0 || D <= 0 || V <= 0) return ZLM_ERR_BAD_ARG;
+    const int Dp = (D + 3) / 4 * 4, Vp = (V + 3) / 4 * 4, ni = dr_scan_ni(Dp);
     if (ni == 0 || H > 65535 || n_seqs > 65535) return ZLM_ERR_UNSUPPORTED;
     dim3 grid((V + DR_VT - 1) / DR_VT, H, n_seqs);
-    const size_t smem = (size_t)DR_STAGES * dr_stage(ni, which != 0) * sizeof(float);
-    if (smem > 227 * 1024) return ZLM_ERR_UNSUPPORTED;
+    const size_t smem = (size_t)DR_STAGES * dr_stage(ni) * sizeof(float);
     cudaError_t e = cudaSuccess;
 #define ZLM_DR_SCAN(NN)                                                                                                \
     do {                                                                                                               \
-        auto* k = which ? dr_scan_kernel<NN, true> : dr_scan_kernel<NN, false>;                                        \
-        ZLM_DR_RAISED(k, which, grid, kr, qr, er, ws, gam, tb, v, state, slots, cu_seqlens, out, out_stride, H, G, Dp, V, Vp); \
+        auto* k = dr_scan_kernel<NN>;                                                                                  \
+        ZLM_DR_RAISED(k, 0, grid, rec, v, state, slots, cu_seqlens, out, out_stride, H, Dp, V, Vp);                    \
     } while (0)
     ZLM_DR_NI(ZLM_DR_SCAN)
 #undef ZLM_DR_SCAN

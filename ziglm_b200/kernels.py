@@ -102,11 +102,11 @@ _PROTOTYPES = {
                            c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
         "zlm_delta_chunks": [c_int, c_int],
-        "zlm_delta_chunk_tokens": [],
-        "zlm_delta_chunk": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                            c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
-        "zlm_delta_scan": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                           c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "zlm_delta_record": [c_int],
+        "zlm_delta_chunk": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                            c_void_p],
+        "zlm_delta_scan": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int,
+                           c_void_p],
         "zlm_delta_decode": [c_void_p, c_int, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_long,
                              c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                              c_float, c_void_p, c_long, c_int, c_void_p, c_long, c_void_p],
@@ -685,8 +685,8 @@ def delta_rule(proj: torch.Tensor, taps: torch.Tensor, ring: torch.Tensor, n_hea
     Head h uses q/k head h // (n_heads // n_kv).  a, b float32 rows; out float32 [T, n_heads * value_dim]; state float32
     [slots, n_heads, value_dim, ceil4(dim)]."""
     made = delta_prep(proj, taps, ring, n_heads, n_kv, dim, value_dim, a, b, rate, dt_bias, step)
-    chunks = delta_chunk(made[0], made[2], made[3], n_heads, n_kv, dim, step)
-    delta_scan(made[0], made[1], chunks, n_heads, n_kv, dim, value_dim, state, step, out)
+    records = delta_chunk(made[0], made[2], made[3], n_heads, n_kv, dim, step)
+    delta_scan(records, made[1], n_heads, dim, value_dim, state, step, out)
 
 
 def delta_prep(proj, taps, ring, n_heads, n_kv, dim, value_dim, a, b, rate, dt_bias, step):
@@ -717,35 +717,30 @@ def delta_chunk(qk, g, beta, n_heads, n_kv, dim, step):
     if (qk.shape != (T, 2 * n_kv, dp) or tuple(g.shape[:2]) != (T, n_heads) or (not per_channel and g.shape[2] != 1)
             or beta.shape != (T, n_heads)):
         raise KernelError("delta_chunk: shapes do not match")
-    wk = wq = we = ws = None
-    if per_channel:
-        wk, wq, we = (step.ws.buf(f"delta_w{i}", (T, n_heads, dp), torch.float32) for i in "kqe")
-    else:
-        ws = step.ws.buf("delta_ws", (T, n_heads, 2), torch.float32)
+    size = int(_fn("delta_rule", "zlm_delta_record")(dim))
+    if size <= 0:
+        raise KernelError(f"delta_chunk: keys of {dim} elements are not supported (at most 512)")
     n_chunks = int(_fn("delta_rule", "zlm_delta_chunks")(T, step.n_seqs))
-    gam = step.ws.buf("delta_gam", (n_chunks, n_heads, dp if per_channel else 1), torch.float32)
-    tb = step.ws.buf("delta_tb", (T, n_heads, 2 * int(_fn("delta_rule", "zlm_delta_chunk_tokens")())), torch.float32)
+    records = step.ws.buf("delta_records", (n_chunks, n_heads, size), torch.float32)
     _check(_fn("delta_rule", "zlm_delta_chunk")(
-        qk.data_ptr(), g.data_ptr(), int(per_channel), beta.data_ptr(), step.cu_seqlens.data_ptr(), _ptr(wk), _ptr(wq),
-        _ptr(we), _ptr(ws), gam.data_ptr(), tb.data_ptr(), step.n_seqs, step.max_new, n_heads, n_kv, dim, _stream()),
-        "delta_chunk")
-    return wk, wq, we, ws, gam, tb
+        qk.data_ptr(), g.data_ptr(), int(per_channel), beta.data_ptr(), step.cu_seqlens.data_ptr(), records.data_ptr(),
+        step.n_seqs, step.max_new, n_heads, n_kv, dim, _stream()), "delta_chunk")
+    return records
 
 
-def delta_scan(qk, v, chunks, n_heads, n_kv, dim, value_dim, state, step, out) -> None:
-    """The third kernel of ``delta_rule``: the walk over the chunks with the state.  ``chunks``: what ``delta_chunk`` gave."""
+def delta_scan(records, v, n_heads, dim, value_dim, state, step, out) -> None:
+    """The third kernel of ``delta_rule``: the walk over the chunks with the state."""
     _delta_state(state, n_heads, dim, value_dim)
-    _rows(out, "out"); _cuda(v, "v", torch.float32); _cuda(qk, "qk", torch.float32)
-    T = qk.shape[0]
-    wk, wq, we, ws, gam, tb = chunks
+    _rows(out, "out"); _cuda(v, "v", torch.float32); _cuda(records, "records", torch.float32)
+    T = v.shape[0]
     if (out.dtype != torch.float32 or out.shape != (T, n_heads * value_dim)
-            or v.shape != (T, n_heads, delta_state_size(value_dim)) or tb.shape[0] != T):
+            or v.shape != (T, n_heads, delta_state_size(value_dim)) or records.dim() != 3 or records.shape[1] != n_heads
+            or records.shape[0] < int(_fn("delta_rule", "zlm_delta_chunks")(T, step.n_seqs))
+            or records.shape[2] != int(_fn("delta_rule", "zlm_delta_record")(dim))):
         raise KernelError("delta_scan: shapes or types do not match")
-    per_channel = wk is not None
     _check(_fn("delta_rule", "zlm_delta_scan")(
-        _ptr(wk if per_channel else qk), _ptr(wq), _ptr(we), _ptr(ws), gam.data_ptr(), tb.data_ptr(), v.data_ptr(),
-        int(per_channel), state.data_ptr(), step.slots.data_ptr(), step.cu_seqlens.data_ptr(), out.data_ptr(),
-        _row_stride(out), step.n_seqs, n_heads, n_kv, dim, value_dim, _stream()), "delta_scan")
+        records.data_ptr(), v.data_ptr(), state.data_ptr(), step.slots.data_ptr(), step.cu_seqlens.data_ptr(), out.data_ptr(),
+        _row_stride(out), step.n_seqs, n_heads, dim, value_dim, _stream()), "delta_scan")
 
 
 def delta_rule_decode(proj: torch.Tensor, taps: torch.Tensor, ring: torch.Tensor, n_heads: int, n_kv: int, dim: int,
