@@ -24,7 +24,7 @@
 // an overflow.  dr_chunk makes everything of this that does not depend on S, all chunks and heads side by side: the
 // weighted keys and queries, T = (I + A)^-1 diag(beta) and B.  dr_scan walks the chunks with S in registers, so a chunk is
 // three float products of which none waits for the token before: a column of S is spread over 16 lanes of a warp, a
-// lane holding two columns, the columns of a head over blocks, which need nothing from each other; the sums over the
+// lane holding two or four columns, the columns of a head over blocks, which need nothing from each other; the sums over the
 // lanes are scattered so that lane (t, column) ends with R_t and o_t of its column.  The chunks come through shared memory
 // (cp.async, three stages).  Every sum is float FMA (two at a time, fma.rn.f32x2); nothing that enters the recurrence
 // passes through a 16-bit type behind the projection.
@@ -34,9 +34,10 @@ namespace zlm {
 
 constexpr int DR_C = 8;              // tokens of a chunk
 constexpr int DR_L = 16;             // lanes that share a column of the state in dr_scan
-constexpr int DR_THREADS = 128;      // of dr_chunk (DR_C tokens x DR_L lanes) and of dr_scan
-constexpr int DR_VT = 16;            // value columns of a block of dr_scan: two a lane, two times DR_L lanes a warp
+constexpr int DR_THREADS = 128;      // of dr_chunk: DR_C tokens x DR_L lanes
+constexpr int DR_VT = 16;            // value columns of a block of dr_scan
 constexpr int DR_PREP_WARPS = 4;
+constexpr int DR_SLIDE = 4;          // taps dr_prep keeps in registers
 
 __device__ __forceinline__ float dr_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 __device__ __forceinline__ float dr_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
@@ -122,7 +123,15 @@ dr_prep_kernel(DrIn<T> in, int channel_decay, int tile, float* __restrict__ qk_o
         for (int i = lo; i < hi; ++i) {
             const long t = first + i;
             if (lane == 0) beta_out[t * in.H + h] = dr_sigmoid(in.b[t * in.b_stride + h]);
-            if (channel_decay) {
+            if (channel_decay && VEC && in.a_stride % 4 == 0 && (uintptr_t)in.a % 16 == 0) {
+                for (int c = lane * 4; c < in.D; c += 128) {
+                    const float4 a4 = *reinterpret_cast<const float4*>(in.a + t * in.a_stride + (long)h * in.D + c);
+                    const float4 d4 = *reinterpret_cast<const float4*>(in.dt_bias + h * in.D + c);
+                    *reinterpret_cast<float4*>(g_out + (t * in.H + h) * in.Dp + c) =
+                        make_float4(expf(-rate * dr_softplus(a4.x + d4.x)), expf(-rate * dr_softplus(a4.y + d4.y)),
+                                    expf(-rate * dr_softplus(a4.z + d4.z)), expf(-rate * dr_softplus(a4.w + d4.w)));
+                }
+            } else if (channel_decay) {
                 for (int c = lane; c < in.Dp; c += 32)
                     g_out[(t * in.H + h) * in.Dp + c] = c < in.D
                         ? expf(-rate * dr_softplus(in.a[t * in.a_stride + (long)h * in.D + c] + in.dt_bias[h * in.D + c])) : 0.f;
@@ -139,7 +148,53 @@ dr_prep_kernel(DrIn<T> in, int channel_decay, int tile, float* __restrict__ qk_o
     const int past = in.past_lens[b];
     float* row_s = dr_sm + warp * in.Dp;                  // a q or k head before its norm
     const float q_scale = unit < in.G ? 1.0f / sqrtf((float)in.D) : 1.0f;
-    for (int i = lo; i < hi; ++i) {
+    const bool slid = VEC && in.K <= DR_SLIDE && size <= 128;
+    if constexpr (VEC) {
+        // a lane's four channels, the inputs of the last tokens in registers
+        if (slid) {
+            const int c = lane * 4;
+            const bool on = c < size;
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+            float4 w[DR_SLIDE], win[DR_SLIDE];                // of the token j places back: its tap and its input
+#pragma unroll
+            for (int j = 0; j < DR_SLIDE; ++j) {
+                w[j] = on && j < in.K ? *reinterpret_cast<const float4*>(in.taps + (long)(in.K - 1 - j) * in.C + c0 + c) : zero;
+                win[j] = zero;
+            }
+            auto input = [&](int i) {                         // of the token at index i of the step, or of one before the step
+                if (!on || past + i < 0) return zero;
+                return i >= 0 ? dr_load4<T>(in.proj + (long)(first + i) * in.proj_stride + c0 + c)
+                              : *reinterpret_cast<const float4*>(ring + (long)((past + i) % in.K) * in.C + c0 + c);
+            };
+#pragma unroll
+            for (int j = DR_SLIDE - 1; j > 0; --j)
+                if (j < in.K) win[j - 1] = input(lo - j);
+#pragma unroll 4
+            for (int i = lo; i < hi; ++i) {
+                const long t = first + i;
+#pragma unroll
+                for (int j = DR_SLIDE - 1; j > 0; --j) win[j] = win[j - 1];
+                win[0] = input(i);
+                float4 y = zero;
+#pragma unroll
+                for (int j = DR_SLIDE - 1; j >= 0; --j) {
+                    y.x = fmaf(w[j].x, win[j].x, y.x); y.y = fmaf(w[j].y, win[j].y, y.y);
+                    y.z = fmaf(w[j].z, win[j].z, y.z); y.w = fmaf(w[j].w, win[j].w, y.w);
+                }
+                y.x = dr_silu(y.x); y.y = dr_silu(y.y); y.z = dr_silu(y.z); y.w = dr_silu(y.w);
+                if (is_v) {
+                    if (on) *reinterpret_cast<float4*>(v_out + (t * in.H + (unit - 2 * in.G)) * in.Vp + c) = y;
+                    continue;
+                }
+                const float ss = fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, y.w * y.w)));
+                const float inv = q_scale / sqrtf(warp_sum(ss) + 1e-6f);
+                if (on)
+                    *reinterpret_cast<float4*>(qk_out + (t * 2 * in.G + unit) * in.Dp + c) =
+                        make_float4(y.x * inv, y.y * inv, y.z * inv, y.w * inv);
+            }
+        }
+    }
+    for (int i = slid ? hi : lo; i < hi; ++i) {
         const long t = first + i;
         const T* x = in.proj + t * in.proj_stride;
         float* dst = is_v ? v_out + (t * in.H + (unit - 2 * in.G)) * in.Vp : qk_out + (t * 2 * in.G + unit) * in.Dp;
@@ -342,20 +397,21 @@ __device__ __forceinline__ float dr_both(dr_f2 v) {
     return x + y;
 }
 
-// The sums over 16 lanes of 16 numbers a lane, scattered: lane m is left with the sum of number m in a[0].  Two sets side
-// by side, so that the rounds of one hide those of the other.
-__device__ __forceinline__ void dr_scatter16(float (&a)[16], float (&b)[16], int l) {
+// The sums over 16 lanes of N numbers a lane, scattered: lane l is left with those of numbers l N/16 .. in front.  Two sets
+// side by side, so that the rounds of one hide those of the other.
+template <int N>
+__device__ __forceinline__ void dr_scatter(float (&a)[N], float (&b)[N], int l) {
 #pragma unroll
-    for (int o = 8; o > 0; o >>= 1) {
+    for (int o = 8, half = N / 2; o > 0; o >>= 1, half >>= 1) {
         const bool up = (l & o) != 0;
 #pragma unroll
-        for (int i = 0; i < o; ++i) {
-            const float give = up ? a[i] : a[i + o], keep = up ? a[i + o] : a[i];
+        for (int i = 0; i < half; ++i) {
+            const float give = up ? a[i] : a[i + half], keep = up ? a[i + half] : a[i];
             a[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
         }
 #pragma unroll
-        for (int i = 0; i < o; ++i) {
-            const float give = up ? b[i] : b[i + o], keep = up ? b[i + o] : b[i];
+        for (int i = 0; i < half; ++i) {
+            const float give = up ? b[i] : b[i + half], keep = up ? b[i + half] : b[i];
             b[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
         }
     }
@@ -365,26 +421,30 @@ constexpr int DR_STAGES = 3;
 // floats of a stage: the chunk's record and its values
 __host__ __device__ constexpr int dr_stage(int NI) { return dr_record(NI) + DR_C * DR_VT; }
 
+// A lane holds VC columns: what a lane reads of a chunk's rows from shared memory, which sets the pace, serves all of them.
+// The threads of a block: two times VC columns a warp, DR_VT columns in all.
+__host__ __device__ constexpr int dr_scan_threads(int VC) { return 32 * DR_VT / (2 * VC); }
+
 // grid (value tiles, heads, sequences).  rec: the records of dr_chunk; v: [T][H][Vp]; out: float rows of H V numbers.
-template <int NI>
-__global__ void __launch_bounds__(DR_THREADS)
+template <int NI, int VC>
+__global__ void __launch_bounds__(dr_scan_threads(VC))
 dr_scan_kernel(const float* __restrict__ rec, const float* __restrict__ v, float* __restrict__ state,
                const int* __restrict__ slots, const int* __restrict__ cu_seqlens, float* __restrict__ out, long out_stride, int H,
                int Dp, int V, int Vp) {
-    constexpr int D4 = 16 * NI, STAGE = dr_stage(NI), RECORD = dr_record(NI);
+    constexpr int D4 = 16 * NI, STAGE = dr_stage(NI), RECORD = dr_record(NI), THREADS = dr_scan_threads(VC), X = VC / 2;
     extern __shared__ __align__(16) float dr_sm[];
     const int tid = threadIdx.x, lane = tid & 31, l = lane & 15;
     const int b = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * DR_VT;
     const int d4 = Dp / 4;
-    const int col0 = (tid >> 5) * 4 + (lane >> 4) * 2;      // this lane's two columns of the tile
-    const int my_t = l >> 1, my_col = col0 + (l & 1);       // what the scattered sums leave this lane with
+    const int col0 = ((tid >> 5) * 2 + (lane >> 4)) * VC;   // this lane's columns of the tile
+    const int my_t = l >> 1, my_col = col0 + (l & 1) * X;   // what the scattered sums leave this lane with: X columns of a token
     // values that are never fetched (behind a short chunk's last token, behind the last column) meet zeros: finite they must be
-    for (int i = tid; i < DR_STAGES * DR_C * DR_VT; i += DR_THREADS)
+    for (int i = tid; i < DR_STAGES * DR_C * DR_VT; i += THREADS)
         dr_sm[(i / (DR_C * DR_VT)) * STAGE + RECORD + i % (DR_C * DR_VT)] = 0.f;
     float* st = state + ((long)slots[b] * H + h) * V * Dp;
-    dr_f2 S[2][2 * NI];
+    dr_f2 S[VC][2 * NI];
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
+    for (int c = 0; c < VC; ++c) {
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
             ulonglong2 s = make_ulonglong2(0, 0);
@@ -405,7 +465,7 @@ dr_scan_kernel(const float* __restrict__ rec, const float* __restrict__ v, float
             float* sm = dr_sm + (chunk % DR_STAGES) * STAGE;
             const float* src = recs + (long)chunk * H * RECORD;
 #pragma unroll
-            for (int i = 0; i < RECORD / 4; i += DR_THREADS)
+            for (int i = 0; i < RECORD / 4; i += THREADS)
                 if (i + tid < RECORD / 4) dr_cp16(sm + 4 * (i + tid), src + 4 * (i + tid));
             if (vj < min(DR_C, n_new - chunk * DR_C) && v0 + vi < Vp)
                 dr_cp16(sm + RECORD + vj * DR_VT + vi, vsrc + (long)chunk * DR_C * H * Vp);
@@ -424,44 +484,52 @@ dr_scan_kernel(const float* __restrict__ rec, const float* __restrict__ v, float
         const ulonglong2* e2 = q2 + DR_C * D4;
         const ulonglong2* g2 = e2 + DR_C * D4;
         const float* tb_s = sm + (3 * DR_C + 1) * 4 * D4 + my_t * 2 * DR_C;      // this lane's row of T, then of B
-        float R[16], O[16];
+        float R[DR_C * VC], O[DR_C * VC];
         // the chunk's keys and queries on the state
 #pragma unroll
         for (int t = 0; t < DR_C; ++t) {
-            dr_f2 r0 = 0, r1 = 0, o0 = 0, o1 = 0;
+            dr_f2 r[VC], o[VC];
+#pragma unroll
+            for (int c = 0; c < VC; ++c) r[c] = o[c] = 0;
 #pragma unroll
             for (int i = 0; i < NI; ++i) {
                 const ulonglong2 kk = k2[t * D4 + DR_L * i], qq = q2[t * D4 + DR_L * i];
-                r0 = dr_fma2(kk.x, S[0][2 * i], r0); r1 = dr_fma2(kk.x, S[1][2 * i], r1);
-                o0 = dr_fma2(qq.x, S[0][2 * i], o0); o1 = dr_fma2(qq.x, S[1][2 * i], o1);
-                r0 = dr_fma2(kk.y, S[0][2 * i + 1], r0); r1 = dr_fma2(kk.y, S[1][2 * i + 1], r1);
-                o0 = dr_fma2(qq.y, S[0][2 * i + 1], o0); o1 = dr_fma2(qq.y, S[1][2 * i + 1], o1);
+#pragma unroll
+                for (int c = 0; c < VC; ++c) {
+                    r[c] = dr_fma2(kk.x, S[c][2 * i], r[c]); o[c] = dr_fma2(qq.x, S[c][2 * i], o[c]);
+                    r[c] = dr_fma2(kk.y, S[c][2 * i + 1], r[c]); o[c] = dr_fma2(qq.y, S[c][2 * i + 1], o[c]);
+                }
             }
-            R[2 * t] = dr_both(r0); R[2 * t + 1] = dr_both(r1);
-            O[2 * t] = dr_both(o0); O[2 * t + 1] = dr_both(o1);
+#pragma unroll
+            for (int c = 0; c < VC; ++c) { R[VC * t + c] = dr_both(r[c]); O[VC * t + c] = dr_both(o[c]); }
         }
         // the state before the chunk's writes
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
             const ulonglong2 gg = g2[DR_L * i];
 #pragma unroll
-            for (int c = 0; c < 2; ++c) {
+            for (int c = 0; c < VC; ++c) {
                 S[c][2 * i] = dr_mul2(S[c][2 * i], gg.x);
                 S[c][2 * i + 1] = dr_mul2(S[c][2 * i + 1], gg.y);
             }
         }
-        const float vv = sm[RECORD + my_t * DR_VT + my_col];
-        dr_scatter16(R, O, l);
-        const float e = vv - R[0];
-        float o = O[0];
-        // u = T e: lane (t, column) takes row t
-        float u = 0.f;
+        dr_scatter<DR_C * VC>(R, O, l);
+        float e[X], u[X];
+#pragma unroll
+        for (int x = 0; x < X; ++x) {
+            e[x] = sm[RECORD + my_t * DR_VT + my_col + x] - R[x];
+            u[x] = 0.f;
+        }
+        // u = T e: a lane takes row t for its columns
         {
             const float4 t0 = *reinterpret_cast<const float4*>(tb_s), t1 = *reinterpret_cast<const float4*>(tb_s + 4);
             const float tr[DR_C] = {t0.x, t0.y, t0.z, t0.w, t1.x, t1.y, t1.z, t1.w};
             const int base = (lane & 16) | (l & 1);
 #pragma unroll
-            for (int j = 0; j < DR_C; ++j) u = fmaf(tr[j], __shfl_sync(0xffffffffu, e, base + 2 * j), u);
+            for (int j = 0; j < DR_C; ++j) {
+#pragma unroll
+                for (int x = 0; x < X; ++x) u[x] = fmaf(tr[j], __shfl_sync(0xffffffffu, e[x], base + 2 * j), u[x]);
+            }
         }
         // o += B u, and the state: G_0n S + sum_j (G_jn k_j) u_j
         {
@@ -470,22 +538,34 @@ dr_scan_kernel(const float* __restrict__ rec, const float* __restrict__ v, float
             const int base = lane & 16;
 #pragma unroll
             for (int j = 0; j < DR_C; ++j) {
-                const float u0 = __shfl_sync(0xffffffffu, u, base + 2 * j), u1 = __shfl_sync(0xffffffffu, u, base + 2 * j + 1);
-                const dr_f2 p0 = dr_pack2(u0, u0), p1 = dr_pack2(u1, u1);
+                float uc[VC];
+                dr_f2 p[VC];
+#pragma unroll
+                for (int c = 0; c < VC; ++c) {
+                    uc[c] = __shfl_sync(0xffffffffu, u[c % X], base + 2 * j + c / X);
+                    p[c] = dr_pack2(uc[c], uc[c]);
+                }
 #pragma unroll
                 for (int i = 0; i < NI; ++i) {
                     const ulonglong2 kk = e2[j * D4 + DR_L * i];
-                    S[0][2 * i] = dr_fma2(kk.x, p0, S[0][2 * i]); S[0][2 * i + 1] = dr_fma2(kk.y, p0, S[0][2 * i + 1]);
-                    S[1][2 * i] = dr_fma2(kk.x, p1, S[1][2 * i]); S[1][2 * i + 1] = dr_fma2(kk.y, p1, S[1][2 * i + 1]);
+#pragma unroll
+                    for (int c = 0; c < VC; ++c) {
+                        S[c][2 * i] = dr_fma2(kk.x, p[c], S[c][2 * i]);
+                        S[c][2 * i + 1] = dr_fma2(kk.y, p[c], S[c][2 * i + 1]);
+                    }
                 }
-                o = fmaf(br[j], (l & 1) ? u1 : u0, o);
+#pragma unroll
+                for (int x = 0; x < X; ++x) O[x] = fmaf(br[j], (l & 1) ? uc[X + x] : uc[x], O[x]);
             }
         }
         const int t = chunk * DR_C + my_t;
-        if (t < n_new && v0 + my_col < V) out[(long)(first + t) * out_stride + (long)h * V + v0 + my_col] = o;
+        float* row = out + (long)(first + t) * out_stride + (long)h * V + v0 + my_col;
+#pragma unroll
+        for (int x = 0; x < X; ++x)
+            if (t < n_new && v0 + my_col + x < V) row[x] = O[x];
     }
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
+    for (int c = 0; c < VC; ++c) {
         if (v0 + col0 + c >= V) continue;
 #pragma unroll
         for (int i = 0; i < NI; ++i)
@@ -713,7 +793,7 @@ static inline int dr_scan_ni(int Dp) {
             if (e != cudaSuccess) return (int)e;                                                                       \
             raised[which] = smem;                                                                                      \
         }                                                                                                              \
-        e = launch_pdl(k, grid, dim3(DR_THREADS), smem, stream, __VA_ARGS__);                                          \
+        e = launch_pdl(k, grid, dim3(threads), smem, stream, __VA_ARGS__);                                             \
     } while (0)
 
 // What every chunk contributes apart from the state: rec, float [zlm_delta_chunks][H][zlm_delta_record] (dr_chunk_kernel).
@@ -726,6 +806,7 @@ ZLM_EXPORT int zlm_delta_chunk(const float* qk, const float* g, int channel_deca
     if (ni == 0 || H > 65535 || n_seqs > 65535) return ZLM_ERR_UNSUPPORTED;
     const size_t smem = (size_t)DR_C * 64 * ni * (which ? 3 : 2) * sizeof(float);
     dim3 grid((max_new + DR_C - 1) / DR_C, H, n_seqs);
+    const int threads = DR_THREADS;
     cudaError_t e = cudaSuccess;
 #define ZLM_DR_CHUNK(NN)                                                                                               \
     do {                                                                                                               \
@@ -754,11 +835,15 @@ ZLM_EXPORT int zlm_delta_scan(const float* rec, const float* v, float* state, co
     if (ni == 0 || H > 65535 || n_seqs > 65535) return ZLM_ERR_UNSUPPORTED;
     dim3 grid((V + DR_VT - 1) / DR_VT, H, n_seqs);
     const size_t smem = (size_t)DR_STAGES * dr_stage(ni) * sizeof(float);
+    // a block an SM at most: more warps hide more of each other's waits; else the SM's shared memory sets the pace
+    const bool few = (long)grid.x * grid.y * grid.z <= 148;
     cudaError_t e = cudaSuccess;
 #define ZLM_DR_SCAN(NN)                                                                                                \
     do {                                                                                                               \
-        auto* k = dr_scan_kernel<NN>;                                                                                  \
-        ZLM_DR_RAISED(k, 0, grid, rec, v, state, slots, cu_seqlens, out, out_stride, H, Dp, V, Vp);                    \
+        constexpr int WIDE = NN <= 4 ? 4 : 2;            /* the registers of longer columns */                         \
+        const int which = few ? 0 : 1, threads = dr_scan_threads(few ? 2 : WIDE);                                      \
+        auto* k = few ? dr_scan_kernel<NN, 2> : dr_scan_kernel<NN, WIDE>;                                              \
+        ZLM_DR_RAISED(k, which, grid, rec, v, state, slots, cu_seqlens, out, out_stride, H, Dp, V, Vp);                \
     } while (0)
     ZLM_DR_NI(ZLM_DR_SCAN)
 #undef ZLM_DR_SCAN

@@ -1018,7 +1018,10 @@ static int gemm_tc_run(const void* X, const void* W, const void* bias, int bias_
     // more than 64 tokens and at least two tiles of weight rows: two CTAs per tile of 256 rows x 256 tokens (with 65
     // to 128 tokens half of the tile is empty, which costs less than leaving the K split and the second SM out)
     const bool paired = T > 64 && splits == 0 && N > TC_BM && scale_ssq == nullptr;
-    const int bn = T <= 16 ? 16 : T <= 32 ? 32 : T <= 64 ? 64 : (T <= 128 && !paired) ? 128 : 256;
+    // many tokens and a handful of weight rows: tiles of 64 tokens with the K range split, or a prompt's tiles would
+    // occupy a few SMs
+    const bool narrow = T > 64 && N <= 64 && splits == 0 && !glu && scale_ssq == nullptr && norm_gain == nullptr;
+    const int bn = T <= 16 ? 16 : T <= 32 ? 32 : (T <= 64 || narrow) ? 64 : (T <= 128 && !paired) ? 128 : 256;
     TcArgs a;
     a.bias = bias; a.bias_dtype = bias_dtype; a.Y = Y; a.ldy = ldy; a.T = T; a.N = N; a.K = K;
     a.kb_total = (K + TC_BK - 1) / TC_BK;
