@@ -1193,10 +1193,22 @@ def run_mopilorn(args):
             args_d = (dproj, taps, ring, H, G, D, V, a, b, rate, bias)
             state_bytes, rule_fma = n_seq * H * D * V * 8, 7.0 * n_tok * H * D * V
             if decode:
-                ms = timed(lambda: kernels.delta_rule_decode(*args_d, dst, step, wl[:V].contiguous(), 1e-6, gate, "silu", lout))
+                wn = wl[:V].contiguous()
+                ms = timed(lambda: kernels.delta_rule_decode(*args_d, dst, step, wn, 1e-6, gate, "silu", lout))
+                moved = state_bytes + n_tok * (C * 2 + H * V * 4) + n_seq * K * C * 4
                 report(f"delta_rule_decode ({H} heads of {D}, {kind}; convolution to gated heads), {tag}",
-                       "decayed_linear_attention", ms, state_bytes + n_tok * (C * 2 + H * per * 4 + H * V * 4) + n_seq * K * C * 4, 0,
-                       rule_fma)
+                       "decayed_linear_attention", ms, moved + n_tok * H * per * 4, 0, rule_fma)
+                hrows, w_b = bf(n_tok, d), bf(H, d)
+                if per > 1:
+                    wide = bf(n_tok, C + 256)
+                    kw = dict(a2=(bf(H * D, 128), C), g2=(bf(H * V, 128), C + 128))
+                    small = (H * D + H * V) * 256
+                else:
+                    wide, kw, small = dproj, dict(w_a=bf(H, d)), H * d * 2
+                ms = timed(lambda: kernels.delta_rule_decode(wide, *args_d[1:7], None, None, rate, bias, dst, step, wn, 1e-6,
+                                                             None if per > 1 else gate, "silu", lout, h=hrows, w_b=w_b, **kw))
+                report(f"delta_rule_decode ({H} heads of {D}, {kind}; small products to gated heads), {tag}",
+                       "decayed_linear_attention", ms, moved + small + H * d * 2, 0, rule_fma)
                 continue
             made = kernels.delta_prep(*args_d, step)
             ms = timed(lambda: kernels.delta_prep(*args_d, step))

@@ -153,6 +153,46 @@ def test_single_tokens_of_a_batch_share_the_channels_of_q_and_k():
 
 
 @pytest.mark.parametrize("dn", list(DTYPES))
+@pytest.mark.parametrize("H,G,D,V,d,r,ch", [(3, 3, 20, 28, 96, 8, True), (4, 2, 128, 128, 256, 128, True),
+                                            (4, 1, 40, 24, 520, 0, False), (2, 2, 64, 64, 64, 40, True)])
+def test_single_tokens_with_the_products_before_decays_and_gate_in_the_kernel(H, G, D, V, d, r, ch, dn):
+    """The same step with a, b and the gate made before and with their products left to the kernel."""
+    from ziglm_b200 import kernels
+    dt, dev = DTYPES[dn], "cuda:0"
+    gen = torch.Generator().manual_seed(D)
+    n = lambda *s: (torch.randn(*s, generator=gen) * 0.3).to(dt).to(dev)
+    B, K, C = 3, 4, 2 * G * D + H * V
+    per = H * D if ch else H
+    at = -(-C // 8) * 8
+    proj, h = n(B, at + 2 * r), n(B, d)
+    w_b, w_a, w_a2, w_g2 = n(H, d), n(H, d), n(H * D, r), n(H * V, r)
+    taps, rate, bias = n(K, C).float(), torch.rand(H, generator=gen).to(dev), n(per).float()
+    norm = torch.ones(V, device=dev)
+    outs = []
+    for inside in (False, True):
+        ring = torch.zeros(B, K, C, device=dev)
+        state = torch.linspace(-1, 1, B * H * V * kernels.delta_state_size(D), device=dev).view(B, H, V, -1).contiguous()
+        if D % 4:
+            state[..., D:] = 0
+        out = torch.empty(B, H * V, dtype=dt, device=dev)
+        step = step_of([5] * B, [1] * B, [2, 0, 1])
+        f = lambda w, x: (x.float() @ w.float().t()).contiguous()
+        a1, g1 = proj[:, at:at + r], proj[:, at + r:at + 2 * r]
+        if ch:
+            kw = dict(h=h, w_b=w_b, a2=(w_a2, at), g2=(w_g2, at + r)) if inside else {}
+            rows = (None, None) if inside else (f(w_a2, a1), f(w_b, h))
+            gate, kind = (None if inside else f(w_g2, g1).to(dt)), "sigmoid"
+        else:
+            kw = dict(h=h, w_b=w_b, w_a=w_a) if inside else {}
+            rows = (None, None) if inside else (f(w_a, h), f(w_b, h))
+            gate, kind = n(B, H * V) * 0 + 0.5, "silu"
+        kernels.delta_rule_decode(proj, taps, ring, H, G, D, V, *rows, rate, bias, state, step, norm, 1e-5, gate, kind, out, **kw)
+        outs.append((out.float().cpu(), state.cpu()))
+    close(outs[1][0], outs[0][0], 2e-5 if dn == "float32" else 2e-2, "rows")
+    close(outs[1][1], outs[0][1], 1e-5, "state")
+
+
+@pytest.mark.parametrize("dn", list(DTYPES))
 @pytest.mark.parametrize("C,K,act", [(40, 4, None), (13, 3, "silu"), (128, 1, None), (24, 12, None), (20, 2, "silu")])
 def test_causal_conv_that_keeps_its_inputs(C, K, act, dn):
     from ziglm_b200 import kernels

@@ -576,11 +576,61 @@ dr_scan_kernel(const float* __restrict__ rec, const float* __restrict__ v, float
 }
 
 // ------------------------------------------------------------------------------------- steps of one token a sequence
+// The last products before the decays, the write strength and the gate of low rank, taken by the block that needs them
+// (steps of few sequences: every block reads its head's rows of the weights).  Weights and rows are of the step's type; K
+// counts are multiples of 8 and rows start on 16 bytes.  Null pointers: the product was taken before.
+template <typename T>
+struct DrDots {
+    const T* h;                 // rows the mixer reads, with stride h_stride, width d
+    long h_stride;
+    int d;
+    const T* wb;                // [H][d]
+    const T* wa;                // [H][d]: one decay a head
+    const T* wa2;               // [H * D][ra], read with the columns a_at.. of the projection
+    const T* wg2;               // [H * V][rg], read with the columns g_at.. of the projection
+    int ra, rg;
+    long a_at, g_at;
+};
+
+__device__ __forceinline__ float dr_dot8(const float* __restrict__ w, const float* __restrict__ x) {
+    const float4 a = *reinterpret_cast<const float4*>(w), b = *reinterpret_cast<const float4*>(w + 4);
+    const float4 u = *reinterpret_cast<const float4*>(x), v = *reinterpret_cast<const float4*>(x + 4);
+    return fmaf(a.x, u.x, fmaf(a.y, u.y, fmaf(a.z, u.z, fmaf(a.w, u.w, fmaf(b.x, v.x, fmaf(b.y, v.y, fmaf(b.z, v.z, b.w * v.w)))))));
+}
+__device__ __forceinline__ float dr_dot8(const __nv_bfloat16* __restrict__ w, const __nv_bfloat16* __restrict__ x) {
+    const uint4 a = *reinterpret_cast<const uint4*>(w), b = *reinterpret_cast<const uint4*>(x);
+    const __nv_bfloat162 *pa = reinterpret_cast<const __nv_bfloat162*>(&a), *pb = reinterpret_cast<const __nv_bfloat162*>(&b);
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 u = __bfloat1622float2(pa[i]), v = __bfloat1622float2(pb[i]);
+        s = fmaf(u.x, v.x, s); s = fmaf(u.y, v.y, s);
+    }
+    return s;
+}
+// w . x over n elements by a warp; every lane gets the sum.
+template <typename T>
+__device__ __forceinline__ float dr_warp_dot(const T* __restrict__ w, const T* __restrict__ x, int n, int lane) {
+    float s = 0.f;
+#pragma unroll 4
+    for (int i = lane * 8; i < n; i += 256) s += dr_dot8(w + i, x + i);
+    return warp_sum(s);
+}
+// The same by four neighbouring lanes (part 0..3), for short rows.
+template <typename T>
+__device__ __forceinline__ float dr_quad_dot(const T* __restrict__ w, const T* __restrict__ x, int n, int part) {
+    float s = 0.f;
+#pragma unroll 4
+    for (int i = part * 8; i < n; i += 32) s += dr_dot8(w + i, x + i);
+    s += __shfl_xor_sync(0xffffffffu, s, 1);
+    return s + __shfl_xor_sync(0xffffffffu, s, 2);
+}
+
 // grid (heads, sequences); blockDim a multiple of 32.  norm_w: [V]; gate rows with stride gate_stride ([H * V] numbers,
 // null: none), gate_kind 1 sigmoid, 2 silu; out rows with stride out_stride.
 template <typename T, int L, int NI, bool CH>
 __global__ void __launch_bounds__(NI > 4 ? 512 : 1024)
-dr_decode_kernel(DrIn<T> in, float* __restrict__ state, const float* __restrict__ norm_w, float eps,
+dr_decode_kernel(DrIn<T> in, DrDots<T> dots, float* __restrict__ state, const float* __restrict__ norm_w, float eps,
                  const T* __restrict__ gate, long gate_stride, int gate_kind, T* __restrict__ out, long out_stride) {
     constexpr int DS = 4 * L * NI;
     extern __shared__ __align__(16) float dr_sm[];
@@ -589,6 +639,7 @@ dr_decode_kernel(DrIn<T> in, float* __restrict__ state, const float* __restrict_
     float* g_s = k_s + DS;                                 // [DS] (CH: the decays; else one number)
     float* v_s = g_s + DS;                                 // [V]
     float* o_s = v_s + in.V;                               // [V]
+    float* gate_s = o_s + in.V;                            // [V] where dots.wg2 is given
     __shared__ float scratch[33], scale_s[2], beta_s;
     pdl_launch_dependents();
     const int h = blockIdx.x, b = blockIdx.y;
@@ -621,14 +672,39 @@ dr_decode_kernel(DrIn<T> in, float* __restrict__ state, const float* __restrict_
         v_s[i] = dr_silu(dr_conv1<T>(in, x, ring, 0, pos, c));
         ring_row[c] = to_float(x[c]);
     }
+    // decays and the write strength; the last warps, which have no part in the convolution of short heads, come first
     const float rate = in.rate[h];
-    if constexpr (CH) {
-        for (int i = tid; i < DS; i += blockDim.x)
-            g_s[i] = i < in.D ? expf(-rate * dr_softplus(in.a[(long)b * in.a_stride + (long)h * in.D + i] + in.dt_bias[h * in.D + i])) : 0.f;
-    } else if (tid == 0) {
-        g_s[0] = expf(-rate * dr_softplus(in.a[(long)b * in.a_stride + h] + in.dt_bias[h]));
+    const int warp = tid >> 5, lane = tid & 31, n_warps = blockDim.x >> 5;
+    if (warp == n_warps - 1) {
+        const float z = dots.wb != nullptr ? dr_warp_dot<T>(dots.wb + (long)h * dots.d, dots.h + (long)b * dots.h_stride, dots.d, lane)
+                                           : in.b[(long)b * in.b_stride + h];
+        if (lane == 0) beta_s = dr_sigmoid(z);
     }
-    if (tid == 0) beta_s = dr_sigmoid(in.b[(long)b * in.b_stride + h]);
+    if (!CH && warp == n_warps - 2) {
+        const float z = dots.wa != nullptr ? dr_warp_dot<T>(dots.wa + (long)h * dots.d, dots.h + (long)b * dots.h_stride, dots.d, lane)
+                                           : in.a[(long)b * in.a_stride + h];
+        if (lane == 0) g_s[0] = expf(-rate * dr_softplus(z + in.dt_bias[h]));
+    }
+    if constexpr (CH) {
+        if (dots.wa2 != nullptr) {
+            for (int i0 = 0; i0 < DS; i0 += blockDim.x / 4) {          // the same number of rounds for every thread
+                const int i = i0 + tid / 4, row = min(i, in.D - 1);
+                const float z = dr_quad_dot<T>(dots.wa2 + ((long)h * in.D + row) * dots.ra, x + dots.a_at, dots.ra, tid & 3);
+                if ((tid & 3) == 0 && i < DS)
+                    g_s[i] = i < in.D ? expf(-rate * dr_softplus(z + in.dt_bias[h * in.D + i])) : 0.f;
+            }
+        } else {
+            for (int i = tid; i < DS; i += blockDim.x)
+                g_s[i] = i < in.D ? expf(-rate * dr_softplus(in.a[(long)b * in.a_stride + (long)h * in.D + i] + in.dt_bias[h * in.D + i])) : 0.f;
+        }
+    }
+    if (dots.wg2 != nullptr) {
+        for (int i0 = 0; i0 < in.V; i0 += blockDim.x / 4) {
+            const int i = i0 + tid / 4, row = min(i, in.V - 1);
+            const float z = dr_quad_dot<T>(dots.wg2 + ((long)h * in.V + row) * dots.rg, x + dots.g_at, dots.rg, tid & 3);
+            if ((tid & 3) == 0 && i < in.V) gate_s[i] = z;
+        }
+    }
     __syncthreads();
     if (tid < 64) {
         const float* r = tid < 32 ? q_s : k_s;
@@ -679,8 +755,8 @@ dr_decode_kernel(DrIn<T> in, float* __restrict__ state, const float* __restrict_
     const float inv = 1.0f / sqrtf(ss / (float)in.V + eps);
     for (int i = tid; i < in.V; i += blockDim.x) {
         float y = o_s[i] * inv * norm_w[i];
-        if (gate != nullptr) {
-            const float gv = to_float(gate[(long)b * gate_stride + (long)h * in.V + i]);
+        if (gate_kind != 0) {
+            const float gv = dots.wg2 != nullptr ? gate_s[i] : to_float(gate[(long)b * gate_stride + (long)h * in.V + i]);
             const float sg = dr_sigmoid(gv);
             y *= gate_kind == 2 ? gv * sg : sg;
         }
@@ -851,7 +927,7 @@ ZLM_EXPORT int zlm_delta_scan(const float* rec, const float* v, float* state, co
 }
 
 template <typename T>
-static int dr_decode_launch(const DrIn<T>& in, int channel_decay, int n_seqs, float* state, const float* norm_w, float eps,
+static int dr_decode_launch(const DrIn<T>& in, const DrDots<T>& dots, int channel_decay, int n_seqs, float* state, const float* norm_w, float eps,
                             const void* gate, long gate_stride, int gate_kind, void* out, long out_stride,
                             cudaStream_t stream) {
     int L, NI;
@@ -859,14 +935,14 @@ static int dr_decode_launch(const DrIn<T>& in, int channel_decay, int n_seqs, fl
     int threads = (in.V * L + 31) / 32 * 32;
     threads = threads < 64 ? 64 : (threads > 1024 ? 1024 : threads);
     if (NI > 4 && threads > 512) threads = 512;
-    const size_t smem = ((size_t)3 * 4 * L * NI + 2 * in.V) * sizeof(float);
+    const size_t smem = ((size_t)3 * 4 * L * NI + 3 * in.V) * sizeof(float);
     if (smem > 48 * 1024) return ZLM_ERR_UNSUPPORTED;
     dim3 grid(in.H, n_seqs);
     cudaError_t e = cudaSuccess;
 #define ZLM_DR_DEC(LL, NN)                                                                                             \
     do {                                                                                                               \
         auto* k = channel_decay ? dr_decode_kernel<T, LL, NN, true> : dr_decode_kernel<T, LL, NN, false>;              \
-        e = launch_pdl(k, grid, dim3(threads), smem, stream, in, state, norm_w, eps, (const T*)gate, gate_stride, gate_kind, \
+        e = launch_pdl(k, grid, dim3(threads), smem, stream, in, dots, state, norm_w, eps, (const T*)gate, gate_stride, gate_kind, \
                        (T*)out, out_stride);                                                                           \
     } while (0)
     ZLM_DR_SHAPES(ZLM_DR_DEC)
@@ -874,28 +950,48 @@ static int dr_decode_launch(const DrIn<T>& in, int channel_decay, int n_seqs, fl
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 
+template <typename T>
+static int dr_decode_typed(const void* proj, long proj_stride, const float* taps, float* ring, int H, int G, int D, int V, int K,
+                           const float* a, long a_stride, int channel_decay, const float* b, long b_stride, const float* rate,
+                           const float* dt_bias, const int* slots, const int* past_lens, int n_seqs, float* state,
+                           const float* norm_w, float eps, const void* gate, long gate_stride, int gate_kind, const void* h,
+                           long h_stride, int d, const void* wb, const void* wa, const void* wa2, int ra, long a_at,
+                           const void* wg2, int rg, long g_at, void* out, long out_stride, cudaStream_t stream) {
+    DrIn<T> in;
+    const int s = dr_fill<T>(in, proj, proj_stride, taps, ring, H, G, D, V, K, a, a_stride, b, b_stride, rate, dt_bias, slots,
+                             past_lens, nullptr);
+    if (s) return s;
+    const int per16 = 16 / (int)sizeof(T);
+    if ((wb == nullptr && b == nullptr) || (gate_kind != 0 && gate == nullptr && wg2 == nullptr) ||
+        (channel_decay ? (a == nullptr && wa2 == nullptr) : (a == nullptr && wa == nullptr)) ||
+        ((wb != nullptr || wa != nullptr) && (h == nullptr || d % 8 || h_stride % per16)) ||
+        (wa2 != nullptr && (ra % 8 || a_at % per16 || proj_stride % per16)) ||
+        (wg2 != nullptr && (rg % 8 || g_at % per16 || proj_stride % per16)))
+        return ZLM_ERR_BAD_ARG;
+    for (const void* p : {h, wb, wa, wa2, wg2, wa2 || wg2 ? proj : nullptr})
+        if ((uintptr_t)p % 16) return ZLM_ERR_BAD_ARG;
+    DrDots<T> dots;
+    dots.h = (const T*)h; dots.h_stride = h_stride; dots.d = d; dots.wb = (const T*)wb; dots.wa = (const T*)wa;
+    dots.wa2 = (const T*)wa2; dots.wg2 = (const T*)wg2; dots.ra = ra; dots.rg = rg; dots.a_at = a_at; dots.g_at = g_at;
+    return dr_decode_launch<T>(in, dots, channel_decay, n_seqs, state, norm_w, eps, gate, gate_stride, gate_kind, out, out_stride,
+                               stream);
+}
+
 // One token a sequence (row b of proj belongs to sequence b).  gate: rows of H V numbers of proj's type, or null;
-// gate_kind 1 sigmoid, 2 silu; norm_w: float [V]; out: rows of H V numbers of proj's type.
+// gate_kind 0 none, 1 sigmoid, 2 silu; norm_w: float [V]; out: rows of H V numbers of proj's type.  The products behind b, a
+// and gate may be left to the kernel (DrDots): wb [H][d] and wa [H][d] with the rows h; wa2 [H D][ra] with the columns from
+// a_at on of proj, wg2 [H V][rg] with those from g_at on.
 ZLM_EXPORT int zlm_delta_decode(const void* proj, int dtype, long proj_stride, const float* taps, float* ring, int H, int G,
                                 int D, int V, int K, const float* a, long a_stride, int channel_decay, const float* b,
                                 long b_stride, const float* rate, const float* dt_bias, const int* slots,
                                 const int* past_lens, int n_seqs, float* state, const float* norm_w, float eps,
-                                const void* gate, long gate_stride, int gate_kind, void* out, long out_stride,
-                                cudaStream_t stream) {
+                                const void* gate, long gate_stride, int gate_kind, const void* h, long h_stride, int d,
+                                const void* wb, const void* wa, const void* wa2, int ra, long a_at, const void* wg2, int rg,
+                                long g_at, void* out, long out_stride, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
-    if (dtype == ZLM_F32) {
-        DrIn<float> in;
-        const int s = dr_fill<float>(in, proj, proj_stride, taps, ring, H, G, D, V, K, a, a_stride, b, b_stride, rate, dt_bias,
-                                     slots, past_lens, nullptr);
-        return s ? s : dr_decode_launch<float>(in, channel_decay, n_seqs, state, norm_w, eps, gate, gate_stride, gate_kind, out,
-                                               out_stride, stream);
-    }
-    if (dtype == ZLM_BF16) {
-        DrIn<__nv_bfloat16> in;
-        const int s = dr_fill<__nv_bfloat16>(in, proj, proj_stride, taps, ring, H, G, D, V, K, a, a_stride, b, b_stride, rate,
-                                             dt_bias, slots, past_lens, nullptr);
-        return s ? s : dr_decode_launch<__nv_bfloat16>(in, channel_decay, n_seqs, state, norm_w, eps, gate, gate_stride,
-                                                       gate_kind, out, out_stride, stream);
-    }
-    return ZLM_ERR_UNSUPPORTED;
+    auto run = dtype == ZLM_F32 ? dr_decode_typed<float> : dtype == ZLM_BF16 ? dr_decode_typed<__nv_bfloat16> : nullptr;
+    if (run == nullptr) return ZLM_ERR_UNSUPPORTED;
+    return run(proj, proj_stride, taps, ring, H, G, D, V, K, a, a_stride, channel_decay, b, b_stride, rate, dt_bias, slots,
+               past_lens, n_seqs, state, norm_w, eps, gate, gate_stride, gate_kind, h, h_stride, d, wb, wa, wa2, ra, a_at, wg2, rg,
+               g_at, out, out_stride, stream);
 }

@@ -109,7 +109,8 @@ _PROTOTYPES = {
                            c_void_p],
         "zlm_delta_decode": [c_void_p, c_int, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_long,
                              c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                             c_float, c_void_p, c_long, c_int, c_void_p, c_long, c_void_p],
+                             c_float, c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                             c_long, c_void_p, c_int, c_long, c_void_p, c_long, c_void_p],
     },
     "linear_attention": {
         "zlm_linear_attention_chunk": [],
@@ -744,29 +745,74 @@ def delta_scan(records, v, n_heads, dim, value_dim, state, step, out) -> None:
 
 
 def delta_rule_decode(proj: torch.Tensor, taps: torch.Tensor, ring: torch.Tensor, n_heads: int, n_kv: int, dim: int,
-                      value_dim: int, a: torch.Tensor, b: torch.Tensor, rate: torch.Tensor, dt_bias: torch.Tensor,
-                      state: torch.Tensor, step, norm_weight: torch.Tensor, eps: float, gate: Optional[torch.Tensor],
-                      gate_kind: Optional[str], out: torch.Tensor) -> None:
+                      value_dim: int, a: Optional[torch.Tensor], b: Optional[torch.Tensor], rate: torch.Tensor,
+                      dt_bias: torch.Tensor, state: torch.Tensor, step, norm_weight: torch.Tensor, eps: float,
+                      gate: Optional[torch.Tensor], gate_kind: Optional[str], out: torch.Tensor, h=None, w_b=None, w_a=None,
+                      a2=None, g2=None) -> None:
     """``delta_rule`` for a step of one token a sequence, with what stands behind it in the same kernel: every head's output
     divided by its root mean square (``eps``), times ``norm_weight`` (float32 [value_dim], shared by the heads), times
-    act(gate) (proj's type, [T, n_heads * value_dim]; "sigmoid" or "silu"), into out's rows (proj's type)."""
-    K, per_channel = _delta_args(proj, taps, ring, n_heads, n_kv, dim, value_dim, a, b, rate, dt_bias)
+    act(gate) (proj's type, [T, n_heads * value_dim]; "sigmoid" or "silu"), into out's rows (proj's type).
+
+    The last products before a, b and gate may be left to the kernel, whose blocks then read their head's rows of the weights
+    (all of proj's type): b = w_b h and a = w_a h ([n_heads, d], rows ``h`` [T, d]); a = a2 x and gate = g2 x with ``a2`` and
+    ``g2`` (weight [rows, r], first column of x in proj), r a multiple of 8."""
+    _rows(proj, "proj")
+    T = proj.shape[0]
+    C, K = 2 * n_kv * dim + n_heads * value_dim, taps.shape[0]
+    for t, n in ((taps, "taps"), (ring, "ring"), (rate, "rate"), (dt_bias, "dt_bias")):
+        _cuda(t, n, torch.float32)
+    per_channel = dt_bias.numel() == n_heads * dim
+    if a is not None:
+        per_channel = per_channel and a.shape[1] == n_heads * dim
+    elif w_a is not None:
+        per_channel = False
+    decays = n_heads * dim if per_channel else n_heads
     _delta_state(state, n_heads, dim, value_dim)
     _rows(out, "out"); _cuda(norm_weight, "norm_weight", torch.float32)
-    T = proj.shape[0]
-    if (T != step.n_seqs or out.dtype != proj.dtype or out.shape != (T, n_heads * value_dim)
-            or norm_weight.numel() != value_dim or gate_kind not in HEAD_GATES or (gate is None) != (gate_kind is None)):
-        raise KernelError("delta_rule_decode: one row a sequence, out of proj's type, a weight of one head's length")
+    if (n_heads <= 0 or n_kv <= 0 or n_heads % n_kv or proj.shape[1] < C or taps.shape != (K, C)
+            or tuple(ring.shape[1:]) != (K, C) or rate.numel() != n_heads or dt_bias.numel() != decays
+            or T != step.n_seqs or out.dtype != proj.dtype or out.shape != (T, n_heads * value_dim)
+            or norm_weight.numel() != value_dim or gate_kind not in HEAD_GATES):
+        raise KernelError("delta_rule_decode: shapes or types do not match")
+    for t, width, n in ((a, decays, "a"), (b, n_heads, "b")):
+        if t is not None:
+            _rows(t, n)
+            if t.dtype != torch.float32 or t.shape != (T, width):
+                raise KernelError(f"delta_rule_decode: {n} must be float32 [T, {width}]")
     if gate is not None:
         _rows(gate, "gate")
         if gate.dtype != proj.dtype or gate.shape != out.shape:
             raise KernelError("delta_rule_decode: the gate must have out's type and shape")
+    d = 0
+    if w_b is not None or w_a is not None:
+        _rows(h, "h")
+        d = h.shape[1]
+        for w in (w_b, w_a):
+            if w is not None:
+                _cuda(w, "weight", proj.dtype)
+                if h.dtype != proj.dtype or h.shape[0] != T or w.shape != (n_heads, d):
+                    raise KernelError("delta_rule_decode: w_b and w_a must be [n_heads, d] of h's type")
+    low = []
+    for pair, n_rows in ((a2, n_heads * dim), (g2, n_heads * value_dim)):
+        if pair is None:
+            low.append((None, 0, 0))
+            continue
+        w, at = pair
+        _cuda(w, "weight", proj.dtype)
+        if w.shape[0] != n_rows or at < 0 or at + w.shape[1] > proj.shape[1]:
+            raise KernelError("delta_rule_decode: a product of low rank must be [rows, r] over columns of proj")
+        low.append((w, w.shape[1], int(at)))
+    if ((b is None) == (w_b is None) or [a is None, w_a is None, a2 is None].count(False) != 1
+            or (a2 is not None and not per_channel)
+            or [gate is None, g2 is None].count(False) != (0 if gate_kind is None else 1)):
+        raise KernelError("delta_rule_decode: a, b and gate are each given once, as rows or as the product that makes them")
     _check(_fn("delta_rule", "zlm_delta_decode")(
         proj.data_ptr(), code(proj.dtype), _row_stride(proj), taps.data_ptr(), ring.data_ptr(), n_heads, n_kv, dim, value_dim,
-        K, a.data_ptr(), _row_stride(a), int(per_channel), b.data_ptr(), _row_stride(b), rate.data_ptr(), dt_bias.data_ptr(),
-        step.slots.data_ptr(), step.past_lens.data_ptr(), step.n_seqs, state.data_ptr(), norm_weight.data_ptr(), float(eps),
-        _ptr(gate), _row_stride(gate) if gate is not None else 0, HEAD_GATES[gate_kind], out.data_ptr(), _row_stride(out),
-        _stream()), "delta_rule_decode")
+        K, _ptr(a), _row_stride(a) if a is not None else 0, int(per_channel), _ptr(b), _row_stride(b) if b is not None else 0,
+        rate.data_ptr(), dt_bias.data_ptr(), step.slots.data_ptr(), step.past_lens.data_ptr(), step.n_seqs, state.data_ptr(),
+        norm_weight.data_ptr(), float(eps), _ptr(gate), _row_stride(gate) if gate is not None else 0, HEAD_GATES[gate_kind],
+        _ptr(h) if d else None, _row_stride(h) if d else 0, d, _ptr(w_b), _ptr(w_a), _ptr(low[0][0]), low[0][1], low[0][2],
+        _ptr(low[1][0]), low[1][1], low[1][2], out.data_ptr(), _row_stride(out), _stream()), "delta_rule_decode")
 
 
 def selective_scan(u: torch.Tensor, dt_pre: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, n_states: int,

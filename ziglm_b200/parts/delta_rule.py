@@ -15,7 +15,8 @@ The rank of a product of low rank is an option (``decay_rank``, ``gate_rank``; N
 carries the convolution's last inputs [K, C] and S, both float32 (two ``StateNeed``).  Decays, write strengths, unit
 vectors, the state and the products that enter it are float32 in both precisions; in bfloat16 the projections are, but for
 the last product before a decay or a write strength, whose sums stay float32.
-A step of one token a sequence runs everything between the projections and W_o in one kernel.
+A step of one token a sequence runs everything between the first product and W_o in one kernel (in steps of many sequences
+the small products before a, b and the gate are taken before it).
 """
 from __future__ import annotations
 
@@ -27,6 +28,11 @@ from .. import kernels
 from ..config.spec import MixerSpec
 from .base import FreeDim, KVNeed, LayerIO, ParamDecl, Part, StateNeed, register_mixer
 from .linear import Linear
+
+
+# Sequences up to which a step of one token a sequence leaves the small products before decays, write strengths and the gate
+# to the kernel of the recurrence: its blocks then read their head's rows of the weights once for every sequence.
+FUSED_SEQUENCES = 16
 
 
 def _up8(n: int) -> int:
@@ -157,21 +163,35 @@ class GatedDeltaRule(Part):
         ring, state = io.state
         proj = step.ws.buf("delta_proj", (T, self.proj.out_features), self.dtype)
         self.proj(h, proj)
+        out = step.ws.buf("delta_out", (T, H * V), self.dtype)
+        a_cols = slice(self.a_at, self.a_at + _up8(self.a_rank))
+        g_cols = slice(self.g_at, self.g_at + _up8(self.g_rank))
+        fused = (step.single_token and T <= FUSED_SEQUENCES and h.shape[1] % 8 == 0 and h.stride(0) % 8 == 0
+                 and all(lin is None or lin.weight.dtype == self.dtype for lin in (self.rates, self.a2, self.g2)))
+        args = (proj, self.conv_w, ring, H, self.n_kv, self.dim, V)
+        if fused:
+            low_gate = (self.g2.weight, self.g_at) if self.low_rank_gate else None
+            gate = proj[:, self.g_at:self.g_at + H * V] if self.gate is not None and not self.low_rank_gate else None
+            kernels.delta_rule_decode(
+                *args, None, None, self.rate, self.dt_bias, state, step, self.norm_w, self.eps, gate, self.gate, out, h=h,
+                w_b=self.rates.weight[:H], w_a=self.rates.weight[H:2 * H] if self.decay == "head" else None,
+                a2=(self.a2.weight, self.a_at) if self.decay == "channel" else None, g2=low_gate)
+            self.o(out, residual, accumulate=accumulate)
+            return None
         rates = step.ws.buf("delta_rates", (T, self.rates.out_features), torch.float32)
         self.rates(h, rates)
         if self.decay == "head":
             a = rates[:, H:2 * H]
         else:
             a = step.ws.buf("delta_a", (T, H * self.dim), torch.float32)
-            self.a2(proj[:, self.a_at:self.a_at + _up8(self.a_rank)], a)
+            self.a2(proj[:, a_cols], a)
         gate = None
         if self.low_rank_gate:
             gate = step.ws.buf("delta_gate", (T, H * V), self.dtype)
-            self.g2(proj[:, self.g_at:self.g_at + _up8(self.g_rank)], gate)
+            self.g2(proj[:, g_cols], gate)
         elif self.gate is not None:
             gate = proj[:, self.g_at:self.g_at + H * V]
-        out = step.ws.buf("delta_out", (T, H * V), self.dtype)
-        args = (proj, self.conv_w, ring, H, self.n_kv, self.dim, V, a, rates[:, :H], self.rate, self.dt_bias, state, step)
+        args += (a, rates[:, :H], self.rate, self.dt_bias, state, step)
         if step.single_token:
             kernels.delta_rule_decode(*args, self.norm_w, self.eps, gate, self.gate, out)
         else:
