@@ -161,3 +161,21 @@ def test_the_array_of_block_tables_follows_the_lists():
     table.advance({c: 7})
     check()
     table.check()
+
+
+def test_a_place_with_several_states_has_all_of_them_zeroed_with_its_slot():
+    import torch
+    from ziglm_b200.cache import CacheStorage
+    from ziglm_b200.parts import StateNeed
+    needs = [StateNeed((3,)), None, (StateNeed((2, 4)), StateNeed((5,)))]
+    cache = CacheStorage([None] * 3, [None] * 3, needs, 128, 2, 64, torch.float32, torch.device("cpu"))
+    one, two = cache.io_for(0, []).state, cache.io_for(2, []).state
+    assert one.shape == (2, 3) and cache.io_for(1, []).state is None
+    assert isinstance(two, tuple) and [t.shape for t in two] == [(2, 2, 4), (2, 5)]
+    slot = cache.alloc_slot()
+    for t in (one,) + two:
+        t.fill_(7.0)
+    cache.free_slot(slot)
+    assert cache.alloc_slot() == slot
+    for t in (one,) + two:
+        assert not t[slot].any() and (t[1 - slot] == 7.0).all()
