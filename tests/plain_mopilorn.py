@@ -214,7 +214,7 @@ def gather_streams(x: torch.Tensor, hc: Mapping[str, torch.Tensor]) -> torch.Ten
 
 
 def spread_streams(x: torch.Tensor, y: torch.Tensor, hc: Mapping[str, torch.Tensor]) -> torch.Tensor:
-    """All streams at once from the old ones: x_b <- sum_a mix[a, b] x_a + out[b] y."""
+    """Every new stream is a mixture of the old ones: x_b <- sum_a mix[a, b] x_a + out[b] y."""
     return torch.einsum("ab,atd->btd", hc["mix"].to(x.dtype), x) + hc["out"].to(x.dtype)[:, None, None] * y[None]
 
 

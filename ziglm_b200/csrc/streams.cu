@@ -1,7 +1,7 @@
 // Residual streams (hyper-connections): a token is carried by s copies of the residual, x_1 .. x_s, float rows of
 // s * d numbers.  Around a sublayer with learned numbers in [s], out [s] and mix [s, s] (indexed [from, to]):
 //     u = sum_a in[a] x_a;   h = u / sqrt(mean u^2 + eps) * w;   y = sublayer(h);
-//     x_b <- sum_a mix[a, b] x_a + out[b] y                         (all streams at once from the old ones)
+//     x_b <- sum_a mix[a, b] x_a + out[b] y                         (every x on the right is an old one)
 // stream_norm makes h.  stream_mix forms the new streams in place and, while their elements are in registers, the h of
 // the sublayer that follows: one pass over the streams a sublayer.  y is one branch, or `factor` times the sum of two
 // branches, each divided by its own root mean square over d and multiplied by a weight.

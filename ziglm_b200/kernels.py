@@ -534,7 +534,7 @@ def stream_norm(x: torch.Tensor, streams: int, gather: Optional[torch.Tensor], w
 
 def stream_mix(x: torch.Tensor, streams: int, coef: torch.Tensor, branches, norm_weights=None, norm_eps: float = 0.0,
                factor: float = 1.0, nxt=None) -> None:
-    """New streams in place: x[t, b] <- sum_a mix[a, b] x[t, a] + out[b] y[t], all at once from the old ones.  ``coef``
+    """New streams in place: x[t, b] <- sum_a mix[a, b] x[t, a] + out[b] y[t] (every x on the right is an old one).  ``coef``
     float32 [streams^2 + streams]: mix row by row ([from, to]), then out.  ``branches``: one float32 [T, d] tensor, y, or
     two, and then y = factor * sum_i norm(branch_i) * norm_weights[i] with ``norm_eps``.  ``nxt`` = (gather, weight, eps,
     h): also the rows h [T, d] that ``stream_norm`` would make of the new streams."""
