@@ -19,6 +19,7 @@ from .tikalix import TikalixConfig
 from .vilazen import VilazenConfig
 from .lipadra import LipadraConfig
 from .mopilorn import MopilornConfig
+from .lilulix import LilulixConfig
 from .spec import ModelSpec
 
 _ARCHITECTURES: Dict[str, Any] = {}
@@ -72,3 +73,4 @@ register_architecture(TikalixConfig.ARCHITECTURE, TikalixConfig)
 register_architecture(VilazenConfig.ARCHITECTURE, VilazenConfig)
 register_architecture(LipadraConfig.ARCHITECTURE, LipadraConfig)
 register_architecture(MopilornConfig.ARCHITECTURE, MopilornConfig)
+register_architecture(LilulixConfig.ARCHITECTURE, LilulixConfig)

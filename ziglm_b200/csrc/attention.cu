@@ -199,7 +199,7 @@ rope_norm_store_kernel(T* __restrict__ qkv, long row_stride, int n_heads, int n_
                        int norm_first, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                        const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                        const int* __restrict__ block_table, int bt_stride, T* __restrict__ k_pages,
-                       T* __restrict__ v_pages, int page_size, long page_stride) {
+                       T* __restrict__ v_pages, int page_size, long page_stride, int values_from_keys) {
     __shared__ float cos_s[ROPE_MAX_HALF], sin_s[ROPE_MAX_HALF];
     __shared__ float head_s[RNS_WARPS][ATT_MAX_HD_ROPE];
     pdl_launch_dependents();
@@ -229,7 +229,7 @@ rope_norm_store_kernel(T* __restrict__ qkv, long row_stride, int n_heads, int n_
     }
     const long kv_head_stride = (long)page_size * hd;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int total_heads = n_heads + 2 * n_kv;
+    const int total_heads = n_heads + (values_from_keys ? 1 : 2) * n_kv;
     const int per = (total_heads + gridDim.y - 1) / gridDim.y;
     const int h_lo = blockIdx.y * per, h_hi = min(total_heads, h_lo + per);
     float* hs = head_s[warp];
@@ -243,6 +243,10 @@ rope_norm_store_kernel(T* __restrict__ qkv, long row_stride, int n_heads, int n_
             continue;
         }
         for (int i = lane; i < hd; i += 32) hs[i] = to_float(row[i]);
+        if (values_from_keys && vdst && head >= n_heads) {
+            T* d = vdst + (long)(head - n_heads) * kv_head_stride;
+            for (int i = lane; i < hd; i += 32) d[i] = row[i];
+        }
         __syncwarp();
         float ss = 0.f;
         if (norm_first && norm_dim > 0) {
@@ -297,7 +301,8 @@ rope_norm_store_vec_kernel(__nv_bfloat16* __restrict__ qkv, long row_stride, int
                            int norm_first, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                            const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                            const int* __restrict__ block_table, int bt_stride, __nv_bfloat16* __restrict__ k_pages,
-                           __nv_bfloat16* __restrict__ v_pages, int page_size, long page_stride, int lph) {
+                           __nv_bfloat16* __restrict__ v_pages, int page_size, long page_stride, int values_from_keys,
+                           int lph) {
     __shared__ float cos_s[ROPE_MAX_HALF], sin_s[ROPE_MAX_HALF];
     pdl_launch_dependents();
     const int t = blockIdx.x;
@@ -342,6 +347,9 @@ rope_norm_store_vec_kernel(__nv_bfloat16* __restrict__ qkv, long row_stride, int
         float ss = 0.f;
         if (active) {
             const uint4 lo = *reinterpret_cast<const uint4*>(row + i0);
+            __nv_bfloat16* raw = (values_from_keys && vdst && head >= n_heads)
+                                     ? vdst + (long)(head - n_heads) * kv_head_stride : nullptr;
+            if (raw) *reinterpret_cast<uint4*>(raw + i0) = lo;
             const __nv_bfloat162* lp = reinterpret_cast<const __nv_bfloat162*>(&lo);
 #pragma unroll
             for (int k = 0; k < 4; ++k) {
@@ -350,6 +358,7 @@ rope_norm_store_vec_kernel(__nv_bfloat16* __restrict__ qkv, long row_stride, int
             }
             if (pair) {
                 const uint4 hi = *reinterpret_cast<const uint4*>(row + i0 + half);
+                if (raw) *reinterpret_cast<uint4*>(raw + i0 + half) = hi;
                 const __nv_bfloat162* hp = reinterpret_cast<const __nv_bfloat162*>(&hi);
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
@@ -417,7 +426,7 @@ rope_norm_store_vec_kernel(__nv_bfloat16* __restrict__ qkv, long row_stride, int
             }
         }
     }
-    if (vdst) {
+    if (vdst && !values_from_keys) {
         const int v_units = hd / 8;
         const int n_threads = gridDim.y * blockDim.x;
         for (int idx = blockIdx.y * blockDim.x + threadIdx.x; idx < n_kv * v_units; idx += n_threads) {
@@ -425,6 +434,150 @@ rope_norm_store_vec_kernel(__nv_bfloat16* __restrict__ qkv, long row_stride, int
             *reinterpret_cast<uint4*>(vdst + (long)h * kv_head_stride + i) =
                 *reinterpret_cast<const uint4*>(row0 + (long)(total_qk + h) * hd + i);
         }
+    }
+}
+
+// What stands between the projections and the scores of an attention through a latent, one block per token:
+//   [r | c] in float (`down`, r_off / c_off its columns): c <- c / sqrt(mean c^2 + eps) * w, r <- turned by the token's
+//   position (pairs i, i + rot/2), and [r | c | zeros up to `kept`] is stored as the token's row of the pages;
+//   every query head [dim unturned | rot turned] goes from `q` to `q_out`, its last `rot` elements turned.
+// Everything between the reads and the one rounding of a write is float.  q and q_out may be the same memory.
+template <typename T, typename TQ>
+__global__ void __launch_bounds__(256)
+latent_prep_kernel(const float* __restrict__ down, long down_stride, int c_off, int rank, int r_off, int rot,
+                   const float* __restrict__ w, float eps, const TQ* q, long q_stride, T* q_out, long q_out_stride,
+                   int n_heads, int dim, const float* __restrict__ inv_freq, const int* __restrict__ positions,
+                   const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int bt_stride,
+                   T* __restrict__ pages, int kept, int page_size, long page_stride) {
+    __shared__ float cos_s[ROPE_MAX_HALF], sin_s[ROPE_MAX_HALF];
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    const int pos = positions[t];                       // positions, tables and frequencies are older than the step
+    const int half = rot / 2;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * inv_freq[i], &sin_s[i], &cos_s[i]);
+    __syncthreads();
+    pdl_wait();
+    const float* row = down + (long)t * down_stride;
+    if (blockIdx.y == 0) {
+        const int page = block_table[(long)seq_of_token[t] * bt_stride + pos / page_size];
+        T* dst = pages + (long)page * page_stride + (long)(pos % page_size) * kept;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = row[c_off + i]; ss = fmaf(v, v, ss); }
+        ss = block_sum(ss, scratch);
+        const float inv = 1.0f / sqrtf(ss / (float)rank + eps);
+        for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[rot + i] = from_float<T>((row[c_off + i] * inv) * w[i]);
+        for (int i = threadIdx.x; i < half; i += blockDim.x) {
+            const float a = row[r_off + i], b = row[r_off + half + i], c = cos_s[i], sn = sin_s[i];
+            dst[i] = from_float<T>(a * c - b * sn);
+            dst[half + i] = from_float<T>(b * c + a * sn);
+        }
+        for (int i = rot + rank + threadIdx.x; i < kept; i += blockDim.x) dst[i] = from_float<T>(0.f);
+    }
+    // the query heads, shared out over the blocks of the token
+    const int per = (n_heads + gridDim.y - 1) / gridDim.y;
+    const int h_lo = blockIdx.y * per, h_hi = min(n_heads, h_lo + per);
+    const TQ* qr = q + (long)t * q_stride;
+    T* qw = q_out + (long)t * q_out_stride;
+    const int size = dim + rot;
+    if ((const void*)q != (const void*)q_out)
+        for (int idx = threadIdx.x; idx < (h_hi - h_lo) * dim; idx += blockDim.x) {
+            const long at = (long)(h_lo + idx / dim) * size + idx % dim;
+            qw[at] = from_float<T>(to_float(qr[at]));
+        }
+    for (int idx = threadIdx.x; idx < (h_hi - h_lo) * half; idx += blockDim.x) {
+        const int i = idx % half;
+        const long at = (long)(h_lo + idx / half) * size + dim + i;
+        const float a = to_float(qr[at]), b = to_float(qr[at + half]), c = cos_s[i], sn = sin_s[i];
+        qw[at] = from_float<T>(a * c - b * sn);
+        qw[at + half] = from_float<T>(b * c + a * sn);
+    }
+}
+
+// The same for float queries and bf16 results whose sizes, offsets and strides are multiples of 8: a thread takes eight
+// elements of an unturned part, or eight pairs of a turned one.  Same arithmetic, element by element (the sum of
+// squares in another order).
+__device__ __forceinline__ void lp_load8(const float* p, float (&f)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void lp_store8(__nv_bfloat16* p, const float (&f)[8]) {
+    uint4 o;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) h[k] = __floats2bfloat162_rn(f[2 * k], f[2 * k + 1]);
+    *reinterpret_cast<uint4*>(p) = o;
+}
+__device__ __forceinline__ void lp_turn8(const float* src, __nv_bfloat16* dst, int half, const float* cos8, const float* sin8) {
+    float a[8], b[8], lo[8], hi[8];
+    lp_load8(src, a);
+    lp_load8(src + half, b);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+        lo[k] = a[k] * cos8[k] - b[k] * sin8[k];
+        hi[k] = b[k] * cos8[k] + a[k] * sin8[k];
+    }
+    lp_store8(dst, lo);
+    lp_store8(dst + half, hi);
+}
+
+__global__ void __launch_bounds__(256)
+latent_prep_vec_kernel(const float* __restrict__ down, long down_stride, int c_off, int rank, int r_off, int rot,
+                       const float* __restrict__ w, float eps, const float* __restrict__ q, long q_stride,
+                       __nv_bfloat16* __restrict__ q_out, long q_out_stride, int n_heads, int dim,
+                       const float* __restrict__ inv_freq, const int* __restrict__ positions,
+                       const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int bt_stride,
+                       __nv_bfloat16* __restrict__ pages, int kept, int page_size, long page_stride) {
+    __shared__ __align__(16) float cos_s[ROPE_MAX_HALF], sin_s[ROPE_MAX_HALF];
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    const int pos = positions[t];
+    const int half = rot / 2;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * inv_freq[i], &sin_s[i], &cos_s[i]);
+    __syncthreads();
+    pdl_wait();
+    const float* row = down + (long)t * down_stride;
+    const int per = (n_heads + gridDim.y - 1) / gridDim.y;
+    const int h_lo = blockIdx.y * per, h_hi = min(n_heads, h_lo + per);
+    const float* qr = q + (long)t * q_stride;
+    __nv_bfloat16* qw = q_out + (long)t * q_out_stride;
+    const int size = dim + rot, plain = dim / 8, units = plain + half / 8;
+    for (int idx = threadIdx.x; idx < (h_hi - h_lo) * units; idx += blockDim.x) {
+        const int h = h_lo + idx / units, u = idx % units;
+        if (u < plain) {
+            float a[8];
+            lp_load8(qr + (long)h * size + u * 8, a);
+            lp_store8(qw + (long)h * size + u * 8, a);
+        } else {
+            const int i0 = (u - plain) * 8;
+            const long at = (long)h * size + dim + i0;
+            lp_turn8(qr + at, qw + at, half, cos_s + i0, sin_s + i0);
+        }
+    }
+    if (blockIdx.y == 0) {
+        const int page = block_table[(long)seq_of_token[t] * bt_stride + pos / page_size];
+        __nv_bfloat16* dst = pages + (long)page * page_stride + (long)(pos % page_size) * kept;
+        float ss = 0.f;
+        for (int i = threadIdx.x * 8; i < rank; i += blockDim.x * 8) {
+            float a[8];
+            lp_load8(row + c_off + i, a);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) ss = fmaf(a[k], a[k], ss);
+        }
+        ss = block_sum(ss, scratch);
+        const float inv = 1.0f / sqrtf(ss / (float)rank + eps);
+        for (int i = threadIdx.x * 8; i < rank; i += blockDim.x * 8) {
+            float a[8], g[8];
+            lp_load8(row + c_off + i, a);
+            lp_load8(w + i, g);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) a[k] = (a[k] * inv) * g[k];
+            lp_store8(dst + rot + i, a);
+        }
+        for (int i = threadIdx.x * 8; i < half; i += blockDim.x * 8)
+            lp_turn8(row + r_off + i, dst + i, half, cos_s + i, sin_s + i);
+        for (int i = rot + rank + threadIdx.x; i < kept; i += blockDim.x) dst[i] = __float2bfloat16_rn(0.f);
     }
 }
 
@@ -477,7 +630,8 @@ template <typename T, int VEC, int G, int NREG>
 __global__ void __launch_bounds__(ATT_WARPS * 32)
 attention_general_kernel(const T* __restrict__ q, long q_row_stride, T* __restrict__ out, int n_heads, int n_kv,
                          int hd, float scale, float softcap, int window, int keep_first,
-                         const float* __restrict__ sinks, const int* __restrict__ positions,
+                         const float* __restrict__ sinks, const float* __restrict__ slopes,
+                         const int* __restrict__ positions,
                          const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int bt_stride,
                          const T* __restrict__ k_pages, const T* __restrict__ v_pages, int page_size,
                          long page_stride, float* __restrict__ part_ml, float* __restrict__ part_o, int max_parts) {
@@ -553,6 +707,7 @@ attention_general_kernel(const T* __restrict__ q, long q_row_stride, T* __restri
             for (int g = 0; g < G; ++g) {
                 float sv = sc[g] * scale;
                 if (softcap > 0.f) sv = softcap * tanhf(sv / softcap);       // a soft cap: scores stay inside (-cap, cap)
+                if (slopes != nullptr) sv = fmaf(-slopes[h0 + g], (float)(pos - j), sv);   // less by the distance
                 if (!valid) sv = -INFINITY;
                 const float m_new = fmaxf(m[g], warp_max(sv));   // lane 0 of the block is always valid
                 const float corr = expf(m[g] - m_new);           // exp(-inf) = 0 on the first block
@@ -688,14 +843,14 @@ attention_fold_kernel(T* __restrict__ out, int n_heads, int hd, int window, int 
 
 template <typename T, int VEC, int G>
 static int launch_attention(const void* q, long q_row_stride, void* out, int T_, int n_heads, int n_kv, int hd, float scale,
-                            float softcap, int window, int keep_first, const float* sinks, const int* positions,
-                            const int* seq_of_token, const int* block_table,
+                            float softcap, int window, int keep_first, const float* sinks, const float* slopes,
+                            const int* positions, const int* seq_of_token, const int* block_table,
                             int bt_stride, const void* k_pages, const void* v_pages, int page_size, long page_stride,
                             float* part_ml, float* part_o, int max_parts, cudaStream_t stream) {
     dim3 grid(T_, n_heads / G, part_o ? max_parts : 1);
 #define ZLM_ATT_GO(NREG)                                                                                              \
     attention_general_kernel<T, VEC, G, NREG><<<grid, ATT_WARPS * 32, 0, stream>>>(                                     \
-        (const T*)q, q_row_stride, (T*)out, n_heads, n_kv, hd, scale, softcap, window, keep_first, sinks, positions, seq_of_token, block_table, \
+        (const T*)q, q_row_stride, (T*)out, n_heads, n_kv, hd, scale, softcap, window, keep_first, sinks, slopes, positions, seq_of_token, block_table, \
         bt_stride, (const T*)k_pages, (const T*)v_pages, page_size, page_stride, part_ml, part_o, max_parts)
     if (hd <= 128) ZLM_ATT_GO(4);
     else if (hd <= 256) ZLM_ATT_GO(8);
@@ -710,12 +865,12 @@ static int launch_attention(const void* q, long q_row_stride, void* out, int T_,
 
 template <typename T, int VEC>
 static int pick_group(int group, const void* q, long q_row_stride, void* out, int T_, int n_heads, int n_kv, int hd,
-                      float scale, float softcap, int window, int keep_first, const float* sinks, const int* positions,
-                      const int* seq_of_token, const int* block_table,
+                      float scale, float softcap, int window, int keep_first, const float* sinks, const float* slopes,
+                      const int* positions, const int* seq_of_token, const int* block_table,
                       int bt_stride, const void* k_pages, const void* v_pages, int page_size, long page_stride,
                       float* part_ml, float* part_o, int max_parts, cudaStream_t stream) {
 #define ZLM_ATT(GV)                                                                                                     \
-    launch_attention<T, VEC, GV>(q, q_row_stride, out, T_, n_heads, n_kv, hd, scale, softcap, window, keep_first, sinks, positions, seq_of_token, \
+    launch_attention<T, VEC, GV>(q, q_row_stride, out, T_, n_heads, n_kv, hd, scale, softcap, window, keep_first, sinks, slopes, positions, seq_of_token, \
                                  block_table, bt_stride, k_pages, v_pages, page_size, page_stride, part_ml, part_o,     \
                                  max_parts, stream)
     if (group % 4 == 0 && hd <= 256) return ZLM_ATT(4);
@@ -1035,18 +1190,20 @@ ZLM_EXPORT int zlm_rope_store(void* qkv, int dtype, long row_stride, int T, int 
 // root of (the mean of the squares of its first norm_dim dimensions + norm_eps) before it is written back and
 // stored.  inv_freq == nullptr: no rotation.  k_pages == nullptr: nothing is stored.  norm_first != 0: the norm stands
 // BEFORE the rotation instead, and q_weight / k_weight (float [hd], shared by all query / key heads; nullptr: none)
-// multiply the normed heads.
+// multiply the normed heads.  values_from_keys != 0: the rows are [q heads | k heads | anything else] and a key head as
+// it stands in the row, before its norm and rotation, is stored as the value.
 ZLM_EXPORT int zlm_rope_norm_store(void* qkv, int dtype, long row_stride, int T, int n_heads, int n_kv, int hd, int rot,
                                    const float* inv_freq, float amplitude, int norm_dim, float norm_eps,
                                    int norm_first, const float* q_weight, const float* k_weight,
                                    const int* positions, const int* seq_of_token, const int* block_table, int bt_stride,
-                                   void* k_pages, void* v_pages, int page_size, long page_stride, cudaStream_t stream) {
+                                   void* k_pages, void* v_pages, int page_size, long page_stride, int values_from_keys,
+                                   cudaStream_t stream) {
     if (T <= 0) return 0;
     if (hd <= 0 || rot < 0 || rot > hd || (rot & 1) || n_heads <= 0 || n_kv < 0 || page_size <= 0 || norm_dim < 0 ||
         norm_dim > hd || (k_pages != nullptr && v_pages == nullptr))
         return ZLM_ERR_BAD_ARG;
     if (rot / 2 > ROPE_MAX_HALF || hd > ATT_MAX_HD_ROPE) return ZLM_ERR_UNSUPPORTED;
-    const int total_heads = n_heads + 2 * n_kv;
+    const int total_heads = n_heads + (values_from_keys ? 1 : 2) * n_kv;
     int parts = (296 + T - 1) / T;
     if (parts > (total_heads + RNS_WARPS - 1) / RNS_WARPS) parts = (total_heads + RNS_WARPS - 1) / RNS_WARPS;
     if (parts < 1) parts = 1;
@@ -1056,7 +1213,7 @@ ZLM_EXPORT int zlm_rope_norm_store(void* qkv, int dtype, long row_stride, int T,
         e = launch_pdl(rope_norm_store_kernel<float>, grid, dim3(RNS_WARPS * 32), 0, stream, (float*)qkv, row_stride,
                        n_heads, n_kv, hd, rot, inv_freq, amplitude, norm_dim, norm_eps, norm_first, q_weight, k_weight,
                        positions, seq_of_token, block_table, bt_stride, (float*)k_pages, (float*)v_pages, page_size,
-                       page_stride);
+                       page_stride, values_from_keys);
     else if (dtype == ZLM_BF16 && hd % 8 == 0 && (inv_freq == nullptr || rot % 16 == 0) && row_stride % 8 == 0 &&
              page_stride % 8 == 0 && (uintptr_t)qkv % 16 == 0 && (uintptr_t)k_pages % 16 == 0 &&
              (uintptr_t)v_pages % 16 == 0 && hd / 8 <= 32) {
@@ -1072,14 +1229,52 @@ ZLM_EXPORT int zlm_rope_norm_store(void* qkv, int dtype, long row_stride, int T,
         e = launch_pdl(rope_norm_store_vec_kernel, dim3(T, vparts), dim3(RNS_WARPS * 32), 0, stream, (__nv_bfloat16*)qkv,
                        row_stride, n_heads, n_kv, hd, rot, inv_freq, amplitude, norm_dim, norm_eps, norm_first, q_weight,
                        k_weight, positions, seq_of_token, block_table, bt_stride, (__nv_bfloat16*)k_pages,
-                       (__nv_bfloat16*)v_pages, page_size, page_stride, lph);
+                       (__nv_bfloat16*)v_pages, page_size, page_stride, values_from_keys, lph);
     } else if (dtype == ZLM_BF16)
         e = launch_pdl(rope_norm_store_kernel<__nv_bfloat16>, grid, dim3(RNS_WARPS * 32), 0, stream, (__nv_bfloat16*)qkv,
                        row_stride, n_heads, n_kv, hd, rot, inv_freq, amplitude, norm_dim, norm_eps, norm_first, q_weight,
                        k_weight, positions, seq_of_token, block_table, bt_stride, (__nv_bfloat16*)k_pages,
-                       (__nv_bfloat16*)v_pages, page_size, page_stride);
+                       (__nv_bfloat16*)v_pages, page_size, page_stride, values_from_keys);
     else
         return ZLM_ERR_UNSUPPORTED;
+    return e == cudaSuccess ? launch_status() : (int)e;
+}
+
+// See latent_prep_kernel.  down: float rows; q: rows of q_dtype (float or the pages' type) with n_heads heads of dim + rot
+// elements; q_out: rows of `dtype`, the type of the pages.
+ZLM_EXPORT int zlm_latent_prep(const float* down, long down_stride, int c_off, int rank, int r_off, int rot, const float* w,
+                               float eps, const void* q, int q_dtype, long q_stride, void* q_out, int dtype,
+                               long q_out_stride, int T, int n_heads, int dim, const float* inv_freq, const int* positions,
+                               const int* seq_of_token, const int* block_table, int bt_stride, void* pages, int kept,
+                               int page_size, long page_stride, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (rank <= 0 || rot < 0 || (rot & 1) || n_heads <= 0 || dim < 0 || dim + rot <= 0 || kept < rot + rank ||
+        page_size <= 0 || pages == nullptr || w == nullptr || (rot > 0 && inv_freq == nullptr))
+        return ZLM_ERR_BAD_ARG;
+    if (rot / 2 > ROPE_MAX_HALF) return ZLM_ERR_UNSUPPORTED;
+    int parts = (148 + T - 1) / T;                     // few tokens: the heads of a token are shared out over blocks
+    if (parts > n_heads) parts = n_heads;
+    const dim3 grid(T, parts);
+    const bool no_q = q == q_out && rot == 0;          // nothing changes in the queries
+    const int work = n_heads * (dim + rot) / parts;
+    cudaError_t e;
+#define ZLM_LP(TT, TQ, threads)                                                                                          \
+    e = launch_pdl(latent_prep_kernel<TT, TQ>, grid, dim3(threads), 0, stream, down, down_stride, c_off, rank, r_off, rot, w,     \
+                   eps, (const TQ*)q, q_stride, (TT*)q_out, q_out_stride, n_heads, dim, inv_freq, positions, seq_of_token, \
+                   block_table, bt_stride, (TT*)pages, kept, page_size, page_stride)
+    const int threads = 256;                           // one order of sums, whatever the step
+    if (dtype == ZLM_F32 && q_dtype == ZLM_F32) ZLM_LP(float, float, threads);
+    else if (dtype == ZLM_BF16 && (q_dtype == ZLM_F32 || no_q) && rank % 8 == 0 && rot % 16 == 0 && dim % 8 == 0 && c_off % 4 == 0 &&
+             r_off % 4 == 0 && down_stride % 4 == 0 && q_stride % 4 == 0 && q_out_stride % 8 == 0 && kept % 8 == 0 &&
+             page_stride % 8 == 0 && (((uintptr_t)down | (uintptr_t)q | (uintptr_t)q_out | (uintptr_t)pages | (uintptr_t)w) % 16) == 0)
+        e = launch_pdl(latent_prep_vec_kernel, grid, dim3(work >= 2048 ? 256 : 128), 0, stream, down, down_stride, c_off, rank,
+                       r_off, rot, w, eps, (const float*)q, q_stride, (__nv_bfloat16*)q_out, q_out_stride, no_q ? 0 : n_heads, dim,
+                       inv_freq, positions, seq_of_token, block_table, bt_stride, (__nv_bfloat16*)pages, kept, page_size,
+                       page_stride);
+    else if (dtype == ZLM_BF16 && q_dtype == ZLM_F32) ZLM_LP(__nv_bfloat16, float, threads);
+    else if (dtype == ZLM_BF16 && q_dtype == ZLM_BF16) ZLM_LP(__nv_bfloat16, __nv_bfloat16, threads);
+    else return ZLM_ERR_UNSUPPORTED;
+#undef ZLM_LP
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 
@@ -1095,13 +1290,14 @@ ZLM_EXPORT long zlm_attention_general_scratch(int T, int n_heads, int n_kv, int 
 
 // keep_first (with a window): the first keep_first positions of a sequence stay visible behind the window.  sinks (float,
 // one per query head; may be null): exp(sinks[h]) is added to the softmax's denominator of head h; it has no key and no
-// value and is not scaled.
+// value and is not scaled.  slopes (float, one per query head; may be null): head h's score of a key at distance
+// pos - j is made less by slopes[h] * (pos - j), after the scale and the cap.
 // max_keys: the most keys any token of the step sees.  scratch (float, scratch_floats elements; may be null):
 // when it holds at least zlm_attention_general_scratch(...) floats and that is not 0, the parts of the keys are
 // computed by blocks of their own and folded by a second kernel; the result is bit for bit the same.
 ZLM_EXPORT int zlm_attention_general(const void* q, long q_row_stride, void* out, int dtype, int T, int n_heads,
                                      int n_kv, int hd, float scale, float softcap, int window, int keep_first,
-                                     const float* sinks, const int* positions,
+                                     const float* sinks, const float* slopes, const int* positions,
                                      const int* seq_of_token, const int* block_table, int bt_stride,
                                      const void* k_pages, const void* v_pages, int page_size, long page_stride,
                                      int max_keys, float* scratch, long scratch_floats, cudaStream_t stream) {
@@ -1120,12 +1316,12 @@ ZLM_EXPORT int zlm_attention_general(const void* q, long q_row_stride, void* out
     }
     const int group = n_heads / n_kv;
     if (dtype == ZLM_F32)
-        return pick_group<float, 4>(group, q, q_row_stride, out, T, n_heads, n_kv, hd, scale, softcap, window, keep_first, sinks,
+        return pick_group<float, 4>(group, q, q_row_stride, out, T, n_heads, n_kv, hd, scale, softcap, window, keep_first, sinks, slopes,
                                     positions, seq_of_token, block_table, bt_stride, k_pages, v_pages, page_size, page_stride,
                                     part_ml, part_o, max_parts, stream);
     if (dtype == ZLM_BF16)
         return pick_group<__nv_bfloat16, 8>(group, q, q_row_stride, out, T, n_heads, n_kv, hd, scale, softcap, window, keep_first,
-                                            sinks, positions, seq_of_token, block_table, bt_stride, k_pages, v_pages, page_size,
+                                            sinks, slopes, positions, seq_of_token, block_table, bt_stride, k_pages, v_pages, page_size,
                                             page_stride, part_ml, part_o, max_parts, stream);
     return ZLM_ERR_UNSUPPORTED;
 }

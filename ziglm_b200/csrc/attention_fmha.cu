@@ -70,6 +70,7 @@ struct FmArgs {
     int window;
     int keep_first;      // with a window: the first positions of a sequence that stay visible behind it
     const float* sinks;  // one number per query head in the softmax's denominator (already times log2(e)), or null
+    const float* slopes; // one number per query head by which a score is made less for each position of distance, or null
     const int* block_table;
     int bt_stride;
     const int* cu_seqlens;
@@ -79,10 +80,10 @@ struct FmArgs {
 
 // The softmax of one query row over a step of NP pages: S from tensor memory, P (bf16) back over its first
 // half.  Returns the factor by which the running sum was rescaled; updates m (reference maximum, base 2) and l.
-template <int HD, int NP>
+template <int HD, int NP, bool SLOPES>
 __device__ __forceinline__ float softmax_row(uint32_t t_s, uint32_t t_o, bool full, int lo_vis, int hi_vis, int keep_vis,
                                              float scale, float neg_big, int lt, float& m, float& l, float cap_in2,
-                                             float cap_log2) {
+                                             float cap_log2, float slope, float bias0) {
     constexpr int N = NP * FM_PAGE;
     uint32_t v[N];
 #pragma unroll
@@ -98,6 +99,14 @@ __device__ __forceinline__ float softmax_row(uint32_t t_s, uint32_t t_o, bool fu
             asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(t) : "f"(__uint_as_float(v[i]) * cap_in2));
             v[i] = __float_as_uint(fmaf(-cap_log2, __fdividef(2.0f, t + 1.0f), cap_log2));
         }
+        scale = 1.0f;
+    }
+    if (SLOPES) {
+        // less by the distance: the first key of the step has the bias bias0 <= 0, every further key `slope` more
+        // (both in base 2); the scores then are in base 2 already
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            v[i] = __float_as_uint(fmaf(__uint_as_float(v[i]), scale, fmaf((float)i, slope, bias0)));
         scale = 1.0f;
     }
     float mx8[8];
@@ -160,7 +169,7 @@ __device__ __forceinline__ float softmax_row(uint32_t t_s, uint32_t t_o, bool fu
     return corr;
 }
 
-template <int HD>
+template <int HD, bool SLOPES>
 __global__ void __launch_bounds__(FM_THREADS, 1)
 fmha_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                     const __grid_constant__ CUtensorMap tmap_v, FmArgs a) {
@@ -403,6 +412,7 @@ fmha_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
             m = a.sinks[h] * 1.4426950408889634f;
             l = 1.0f;
         }
+        const float slope = SLOPES ? a.slopes[h] * 1.4426950408889634f : 0.f;
         bool alive = true;
         for (int j = kept_steps > 0 ? 0 : step_lo[t]; j < step_hi[t]; j = (j + 1 == kept_steps ? step_lo[t] : j + 1)) {
             const int lt = local_step(t, j);
@@ -419,10 +429,13 @@ fmha_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
             // (a tcgen05.ld and its wait cost about as much as the arithmetic on 32 scores), the row stays in
             // registers between the maximum and the exponentials, and the stores of P are waited for once.
             float corr;
+            const float bias0 = slope * (float)(key0 - pos);
             if (np == FM_NP)
-                corr = softmax_row<HD, FM_NP>(t_s, t_o, full, lo_vis, hi_vis, keep_vis, scale, neg_big, lt, m, l, a.cap_in2, a.cap_log2);
+                corr = softmax_row<HD, FM_NP, SLOPES>(t_s, t_o, full, lo_vis, hi_vis, keep_vis, scale, neg_big, lt, m, l, a.cap_in2, a.cap_log2,
+                                              slope, bias0);
             else
-                corr = softmax_row<HD, 1>(t_s, t_o, full, lo_vis, hi_vis, keep_vis, scale, neg_big, lt, m, l, a.cap_in2, a.cap_log2);
+                corr = softmax_row<HD, 1, SLOPES>(t_s, t_o, full, lo_vis, hi_vis, keep_vis, scale, neg_big, lt, m, l, a.cap_in2, a.cap_log2,
+                                              slope, bias0);
             (void)corr;
             tmem_st_wait();
             tc_fence_before_sync();
@@ -533,20 +546,20 @@ static int* fm_error_word() {
     return word;
 }
 
-template <int HD>
+template <int HD, bool SLOPES>
 static int fm_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const FmArgs& a, dim3 grid,
                      cudaStream_t stream) {
     static bool done = false;
     if (!done) {
-        cudaError_t e = cudaFuncSetAttribute(fmha_prefill_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        cudaError_t e = cudaFuncSetAttribute(fmha_prefill_kernel<HD, SLOPES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              FmCfg<HD>::SMEM);
         if (e != cudaSuccess) return (int)e;
-        e = cudaFuncSetAttribute(fmha_prefill_kernel<HD>, cudaFuncAttributePreferredSharedMemoryCarveout,
+        e = cudaFuncSetAttribute(fmha_prefill_kernel<HD, SLOPES>, cudaFuncAttributePreferredSharedMemoryCarveout,
                                  cudaSharedmemCarveoutMaxShared);
         if (e != cudaSuccess) return (int)e;
         done = true;
     }
-    cudaError_t e = launch_pdl(fmha_prefill_kernel<HD>, grid, dim3(FM_THREADS), FmCfg<HD>::SMEM, stream, mq, mk, mv, a);
+    cudaError_t e = launch_pdl(fmha_prefill_kernel<HD, SLOPES>, grid, dim3(FM_THREADS), FmCfg<HD>::SMEM, stream, mq, mk, mv, a);
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 
@@ -558,9 +571,11 @@ using namespace zlm;
 // q: bf16 [T, q_row_stride], the query heads first in each row; out: bf16 [T, n_heads * hd].
 // softcap c > 0: the scaled scores become c tanh(score / c); 0: none.  keep_first: with a window, the first positions
 // of a sequence that stay visible behind it.  sinks: float [n_heads] or null; exp(sinks[h]) joins head h's denominator.
+// slopes: positive floats [n_heads] or null; head h's score of a key d positions back is made less by slopes[h] * d.
 ZLM_EXPORT int zlm_attention_prefill_fmha(const void* q, long q_row_stride, long total_tokens, void* out, int B,
                                           int max_new, int n_heads, int n_kv, int hd, float scale, float softcap,
-                                          int window, int keep_first, const float* sinks, const int* cu_seqlens, const int* past_lens, const int* block_table,
+                                          int window, int keep_first, const float* sinks, const float* slopes,
+                                          const int* cu_seqlens, const int* past_lens, const int* block_table,
                                           int bt_stride, const void* k_pages, const void* v_pages, long n_pages,
                                           int page_size, cudaStream_t stream) {
     if (B <= 0 || max_new <= 0) return 0;
@@ -589,12 +604,15 @@ ZLM_EXPORT int zlm_attention_prefill_fmha(const void* q, long q_row_stride, long
     a.window = window;
     a.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
     a.sinks = sinks;
+    a.slopes = slopes;
     a.block_table = block_table;
     a.bt_stride = bt_stride;
     a.cu_seqlens = cu_seqlens;
     a.past_lens = past_lens;
     a.err = fm_error_word();
-    return hd == 128 ? fm_launch<128>(mq, mk, mv, a, grid, stream) : fm_launch<64>(mq, mk, mv, a, grid, stream);
+    if (slopes != nullptr)
+        return hd == 128 ? fm_launch<128, true>(mq, mk, mv, a, grid, stream) : fm_launch<64, true>(mq, mk, mv, a, grid, stream);
+    return hd == 128 ? fm_launch<128, false>(mq, mk, mv, a, grid, stream) : fm_launch<64, false>(mq, mk, mv, a, grid, stream);
 }
 
 ZLM_EXPORT int zlm_attention_fmha_status(int* out) {

@@ -101,11 +101,13 @@ __device__ __forceinline__ void load_q_frags(uint32_t (&qf)[HD / 16][4], const _
 //   gkey0       position in the sequence of that key
 //   lim_lo/hi   last visible position of rows gid / gid+8;  start_lo/hi first visible one
 //   FULL        every key of the step is visible to every row: no masks are evaluated
-template <int HD, int NT, bool FULL>
+//   SLOPES      a score is made less by slope2[row] (base 2) for every position between its key and lim_lo / lim_hi
+template <int HD, int NT, bool FULL, bool SLOPES = false>
 __device__ __forceinline__ void page_step(const uint32_t (&qf)[HD / 16][4], uint32_t k_tile, uint32_t v_tile, int key0,
                                           int gkey0, int lim_lo, int lim_hi, int start_lo, int start_hi,
                                           float scale_log2, float cap_in2, float cap_log2, float (&m)[2],
-                                          float (&l)[2], float (&o)[HD / 8][4], int lane) {
+                                          float (&l)[2], float (&o)[HD / 8][4], int lane,
+                                          const float* slope2 = nullptr) {
     const int gid = lane >> 2, tid4 = lane & 3, mi = lane >> 3, r8 = lane & 7;
     float s[NT][4];
 #pragma unroll
@@ -138,7 +140,12 @@ __device__ __forceinline__ void page_step(const uint32_t (&qf)[HD / 16][4], uint
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const bool hi = i >= 2;
-            if (FULL) {
+            if (SLOPES) {
+                const int key = gkey0 + nt * 8 + 2 * tid4 + (i & 1);
+                const int lim = hi ? lim_hi : lim_lo;
+                const bool vis = FULL || (key <= lim && key >= (hi ? start_hi : start_lo));
+                s[nt][i] = vis ? fmaf(s[nt][i], scale_log2, slope2[hi] * (float)(key - lim)) : -INFINITY;
+            } else if (FULL) {
                 s[nt][i] *= scale_log2;
             } else {
                 const int key = gkey0 + nt * 8 + 2 * tid4 + (i & 1);
@@ -203,6 +210,7 @@ struct AtcCommon {
     int keep_first;      // the split decode kernel only: with a window, the first positions that stay visible behind it
     const int* block_table;
     int bt_stride;
+    const float* slopes; // the split decode kernel only: by how much a head's score is made less per position, or null
     int* err;
     // the flat decode kernel only: out[t, h, d] is multiplied by sigmoid(gate[t * gate_stride + h * hd + d]) before it
     // is rounded (a gate on the heads' outputs); null: none
@@ -242,7 +250,7 @@ __device__ __forceinline__ void produce_pages(const CUtensorMap* tk, const CUten
 }
 
 // ------------------------------------------------------------------- decode
-template <int HD>
+template <int HD, bool SLOPES = false>
 __global__ void __launch_bounds__(ATC_THREADS)
 attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, AtcCommon a,
                    const int* __restrict__ positions, const int* __restrict__ seq_of_token,
@@ -306,14 +314,19 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
         uint32_t qf[HD / 16][4];
         load_q_frags<HD>(qf, gid < group ? qrow + gid * HD : nullptr, gid + 8 < group ? qrow + (gid + 8) * HD : nullptr,
                          tid4);
+        float slope2[2] = {0.f, 0.f};
+        if (SLOPES) {
+            if (gid < group) slope2[0] = a.slopes[kvh * group + gid] * 1.4426950408889634f;
+            if (gid + 8 < group) slope2[1] = a.slopes[kvh * group + gid + 8] * 1.4426950408889634f;
+        }
         int it = 0;
         for (int lp = page_lo; lp < page_hi; ++lp, ++it) {
             const int p = lp < kept_pages ? lp : lp + skip_by;
             const int s = it % C::STAGES;
             if (!mbar_wait(full0 + 8 * s, (it / C::STAGES) & 1, abort_flag, a.err, ERR_ATT_FULL)) break;
             if (p * PAGE >= start && p * PAGE + PAGE - 1 <= pos) {
-                page_step<HD, 2, true>(qf, k0 + s * C::TILE_BYTES, v0 + s * C::TILE_BYTES, warp * 16, p * PAGE + warp * 16,
-                                       pos, pos, start, start, a.scale_log2, a.cap_in2, a.cap_log2, m, l, o, lane);
+                page_step<HD, 2, true, SLOPES>(qf, k0 + s * C::TILE_BYTES, v0 + s * C::TILE_BYTES, warp * 16, p * PAGE + warp * 16,
+                                       pos, pos, start, start, a.scale_log2, a.cap_in2, a.cap_log2, m, l, o, lane, slope2);
             } else {
                 // a page that begins before the window: its kept keys [0, keep) and its keys from the window's first
                 // on, as one range when the two touch and else one after the other
@@ -327,8 +340,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
                 }
                 if (seen) {
                     const int st = joined ? 0 : start;
-                    page_step<HD, 2, false>(qf, k0 + s * C::TILE_BYTES, v0 + s * C::TILE_BYTES, warp * 16, p * PAGE + warp * 16,
-                                            pos, pos, st, st, a.scale_log2, a.cap_in2, a.cap_log2, m, l, o, lane);
+                    page_step<HD, 2, false, SLOPES>(qf, k0 + s * C::TILE_BYTES, v0 + s * C::TILE_BYTES, warp * 16, p * PAGE + warp * 16,
+                                            pos, pos, st, st, a.scale_log2, a.cap_in2, a.cap_log2, m, l, o, lane, slope2);
                 }
             }
             __syncwarp();
@@ -1107,6 +1120,7 @@ static int fill_common(AtcCommon* a, CUtensorMap* mk, CUtensorMap* mv, const voi
     a->keep_first = 0;
     a->block_table = block_table;
     a->bt_stride = bt_stride;
+    a->slopes = nullptr;
     a->err = att_error_word();
     a->gate = nullptr;
     a->gate_stride = 0;
@@ -1120,11 +1134,12 @@ using namespace zlm;
 // Decode-style attention: every token is a tile of its own (its query heads grouped by kv head).
 // part_o: float [T * n_heads * n_splits * hd], part_ml: float [T * n_heads * n_splits * 2] (scratch).
 // keep_first: with a window, the first positions of a sequence that stay visible behind it.  sinks: float [n_heads]
-// or null; exp(sinks[h]) joins head h's denominator.  head_gate: bf16 rows of gate_stride elements with one gate per
+// or null; exp(sinks[h]) joins head h's denominator.  slopes: float [n_heads] or null (not with keep_first); head h's
+// score of a key d positions back is made less by slopes[h] * d.  head_gate: bf16 rows of gate_stride elements with one gate per
 // query head in front, or null; head h of token t leaves multiplied by sigmoid(head_gate[t][h]) * gate_mult.
 ZLM_EXPORT int zlm_attention_decode(const void* q, long q_row_stride, void* out, int T, int n_heads, int n_kv, int hd,
                                     float scale, float softcap, int window, int keep_first, const float* sinks,
-                                    const void* head_gate, long gate_stride, float gate_mult,
+                                    const float* slopes, const void* head_gate, long gate_stride, float gate_mult,
                                     const int* positions, const int* seq_of_token,
                                     const int* block_table, int bt_stride, const void* k_pages, const void* v_pages,
                                     long n_pages, int page_size, int n_splits, float* part_o, float* part_ml,
@@ -1138,14 +1153,17 @@ ZLM_EXPORT int zlm_attention_decode(const void* q, long q_row_stride, void* out,
                          k_pages, v_pages, n_pages, page_size, softcap);
     if (rc) return rc;
     a.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
+    a.slopes = slopes;
+    if (slopes != nullptr && a.keep_first > 0) return ZLM_ERR_UNSUPPORTED;
     dim3 grid(n_splits, n_kv, T);
     using CFG128 = DecodeCfg<128>;
     using CFG64 = DecodeCfg<64>;
     if (hd == 128) {
-        static bool done = false;
-        rc = set_smem(attn_decode_kernel<128>, CFG128::SMEM, &done);
+        static bool done[2] = {false, false};
+        auto* kern = slopes != nullptr ? attn_decode_kernel<128, true> : attn_decode_kernel<128, false>;
+        rc = set_smem(kern, CFG128::SMEM, &done[slopes != nullptr]);
         if (rc) return rc;
-        cudaError_t e = launch_pdl(attn_decode_kernel<128>, grid, dim3(ATC_THREADS), CFG128::SMEM, stream, mk, mv, a,
+        cudaError_t e = launch_pdl(kern, grid, dim3(ATC_THREADS), CFG128::SMEM, stream, mk, mv, a,
                                    positions, seq_of_token, part_o, part_ml);
         if (e == cudaSuccess)
             e = launch_pdl(attn_merge_kernel<128>, dim3(T * n_heads), dim3(128), 0, stream, (const float*)part_o,
@@ -1153,10 +1171,11 @@ ZLM_EXPORT int zlm_attention_decode(const void* q, long q_row_stride, void* out,
                            (const __nv_bfloat16*)head_gate, gate_stride, gate_mult);
         if (e != cudaSuccess) return (int)e;
     } else {
-        static bool done = false;
-        rc = set_smem(attn_decode_kernel<64>, CFG64::SMEM, &done);
+        static bool done[2] = {false, false};
+        auto* kern = slopes != nullptr ? attn_decode_kernel<64, true> : attn_decode_kernel<64, false>;
+        rc = set_smem(kern, CFG64::SMEM, &done[slopes != nullptr]);
         if (rc) return rc;
-        cudaError_t e = launch_pdl(attn_decode_kernel<64>, grid, dim3(ATC_THREADS), CFG64::SMEM, stream, mk, mv, a,
+        cudaError_t e = launch_pdl(kern, grid, dim3(ATC_THREADS), CFG64::SMEM, stream, mk, mv, a,
                                    positions, seq_of_token, part_o, part_ml);
         if (e == cudaSuccess)
             e = launch_pdl(attn_merge_kernel<64>, dim3(T * n_heads), dim3(64), 0, stream, (const float*)part_o,
@@ -1398,6 +1417,7 @@ ZLM_EXPORT int zlm_attention_decode_noalloc(const void* q, long q_row_stride, vo
     a.keep_first = 0;
     a.block_table = block_table;
     a.bt_stride = bt_stride;
+    a.slopes = nullptr;
     a.err = err;
     a.gate = nullptr;
     a.gate_stride = 0;

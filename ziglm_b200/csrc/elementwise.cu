@@ -592,12 +592,111 @@ __global__ void norm_gate_vec2_kernel(const float* __restrict__ x, long x_stride
     }
 }
 
+// x[t, :] <- (x[t, :] + rows[t, :]) + table_row; rows (float32 like x) may be null.
 template <typename TW>
-__global__ void add_row_kernel(float* __restrict__ x, const TW* __restrict__ table_row, long total, int d) {
+__global__ void add_row_kernel(float* __restrict__ x, const float* __restrict__ rows, const TW* __restrict__ table_row,
+                               long total, int d) {
     pdl_launch_dependents();
     pdl_wait();
     const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < total) x[i] += to_float(table_row[i % d]);
+    if (i >= total) return;
+    const float v = rows ? x[i] + rows[i] : x[i];
+    x[i] = v + to_float(table_row[i % d]);
+}
+
+// The same four elements a thread: d is a multiple of 4 and every pointer is aligned for it.
+template <typename TW>
+__global__ void add_row_vec_kernel(float* __restrict__ x, const float* __restrict__ rows,
+                                   const TW* __restrict__ table_row, long total4, int d4) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total4) return;
+    float4 v = reinterpret_cast<const float4*>(x)[i];
+    if (rows) {
+        const float4 r = reinterpret_cast<const float4*>(rows)[i];
+        v.x += r.x; v.y += r.y; v.z += r.z; v.w += r.w;
+    }
+    float w[4];
+    load4<TW>(table_row + 4 * (i % d4), w);
+    v.x += w[0]; v.y += w[1]; v.z += w[2]; v.w += w[3];
+    reinterpret_cast<float4*>(x)[i] = v;
+}
+
+// ------------------------------------------------------ embedding with token pairs
+// A second table adds a row for the pair (token before, token): row (before * mul_prev + token * mul_cur) mod buckets,
+// and row number `buckets` for a sequence's first token.  The token before the first one of a step is a state of its
+// sequence (last[slot]); `past` tells a sequence that starts, whose state counts for nothing.
+struct PairHash {
+    unsigned long long mul_prev, mul_cur, buckets;
+};
+__device__ __forceinline__ int pair_row(const PairHash& h, bool has_before, int before, int token) {
+    if (!has_before) return (int)h.buckets;
+    return (int)(((unsigned long long)before * h.mul_prev + (unsigned long long)token * h.mul_cur) % h.buckets);
+}
+
+// One block per sequence of the step: rows of all its tokens, then the state.
+__global__ void pair_rows_kernel(const int* __restrict__ tokens, const int* __restrict__ cu_seqlens,
+                                 const int* __restrict__ past_lens, const int* __restrict__ slots,
+                                 int* __restrict__ last, int* __restrict__ rows, PairHash h) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int b = blockIdx.x;
+    const int begin = cu_seqlens[b], end = cu_seqlens[b + 1];
+    const bool goes_on = past_lens[b] > 0;
+    int* state = last + slots[b];
+    for (int t = begin + threadIdx.x; t < end; t += blockDim.x) {
+        const bool first = t == begin;
+        rows[t] = pair_row(h, !first || goes_on, first ? *state : tokens[t - 1], tokens[t]);
+    }
+    __syncthreads();                       // the state has been read
+    if (threadIdx.x == 0 && end > begin) *state = tokens[end - 1];
+}
+
+// One block per token: out = table[token] * scale + pairs[row], and a copy of it where `kept` is not null.  rows null:
+// a step of one token a sequence, token t being sequence t's; the row and the state are this block's own work.
+// VEC: d is a multiple of 4 and every pointer is aligned for it.
+template <typename TW, typename TB, bool VEC>
+__global__ void embed_pairs_kernel(const TW* __restrict__ table, const TB* __restrict__ pairs,
+                                   const int* __restrict__ tokens, const int* __restrict__ rows,
+                                   const int* __restrict__ past_lens, const int* __restrict__ slots,
+                                   int* __restrict__ last, PairHash h, float* __restrict__ out, float* __restrict__ kept,
+                                   int d, float scale) {
+    __shared__ int row_s;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int token = tokens[t];
+    if (threadIdx.x == 0) {
+        if (rows != nullptr) row_s = rows[t];
+        else {
+            int* state = last + slots[t];
+            row_s = pair_row(h, past_lens[t] > 0, *state, token);
+            *state = token;
+        }
+    }
+    __syncthreads();
+    const TW* a = table + (long)token * d;
+    const TB* b = pairs + (long)row_s * d;
+    float* o = out + (long)t * d;
+    float* k = kept != nullptr ? kept + (long)t * d : nullptr;
+    if (VEC) {
+        for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) {
+            float u[4], v[4];
+            load4<TW>(a + i, u);
+            load4<TB>(b + i, v);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) u[j] = u[j] * scale + v[j];
+            store4<float>(o + i, u[0], u[1], u[2], u[3]);
+            if (k) store4<float>(k + i, u[0], u[1], u[2], u[3]);
+        }
+    } else {
+        for (int i = threadIdx.x; i < d; i += blockDim.x) {
+            const float v = to_float(a[i]) * scale + to_float(b[i]);
+            o[i] = v;
+            if (k) k[i] = v;
+        }
+    }
 }
 
 __global__ void scale_kernel(float* __restrict__ x, long n, float factor) {
@@ -1003,19 +1102,75 @@ ZLM_EXPORT int zlm_head_norm_gate(const float* x, long x_stride, const float* w,
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 
-ZLM_EXPORT int zlm_add_row(float* x, const void* table_row, int dtype, int T, int d, cudaStream_t stream) {
+// x[t, :] <- (x[t, :] + rows[t, :]) + table_row, all of d elements; rows (float32, or null) has x's shape.
+ZLM_EXPORT int zlm_add_row(float* x, const float* rows, const void* table_row, int dtype, int T, int d,
+                           cudaStream_t stream) {
     if (T <= 0) return 0;
     if (d <= 0) return ZLM_ERR_BAD_ARG;
+    if (dtype != ZLM_F32 && dtype != ZLM_BF16) return ZLM_ERR_UNSUPPORTED;
     const long total = (long)T * d;
-    const unsigned blocks = (unsigned)((total + 255) / 256);
+    const bool vec = d % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)rows % 16 == 0 && (uintptr_t)table_row % 16 == 0;
+    const long n = vec ? total / 4 : total;
+    const unsigned blocks = (unsigned)((n + 255) / 256);
     cudaError_t e;
     if (dtype == ZLM_F32)
-        e = launch_pdl(add_row_kernel<float>, dim3(blocks), dim3(256), 0, stream, x, (const float*)table_row, total, d);
-    else if (dtype == ZLM_BF16)
-        e = launch_pdl(add_row_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, x,
-                       (const __nv_bfloat16*)table_row, total, d);
+        e = vec ? launch_pdl(add_row_vec_kernel<float>, dim3(blocks), dim3(256), 0, stream, x, rows,
+                             (const float*)table_row, n, d / 4)
+                : launch_pdl(add_row_kernel<float>, dim3(blocks), dim3(256), 0, stream, x, rows, (const float*)table_row,
+                             n, d);
     else
-        return ZLM_ERR_UNSUPPORTED;
+        e = vec ? launch_pdl(add_row_vec_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, x, rows,
+                             (const __nv_bfloat16*)table_row, n, d / 4)
+                : launch_pdl(add_row_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, x, rows,
+                             (const __nv_bfloat16*)table_row, n, d);
+    return e == cudaSuccess ? launch_status() : (int)e;
+}
+
+// See embed_pairs_kernel and pair_rows_kernel.  last: int [slots], the last token of every sequence.  rows: int [T]
+// scratch that pair_rows fills; null for a step of one token a sequence (B == T), whose rows the one kernel makes.
+// kept: null, or float [T, d] that receives a copy of out.
+ZLM_EXPORT int zlm_pair_rows(const int* tokens, const int* cu_seqlens, const int* past_lens, const int* slots, int* last,
+                             int* rows, int B, long mul_prev, long mul_cur, long buckets, cudaStream_t stream) {
+    if (B <= 0) return 0;
+    if (mul_prev < 0 || mul_cur < 0 || buckets <= 0 || buckets > 0x7ffffffeL) return ZLM_ERR_BAD_ARG;
+    const PairHash h{(unsigned long long)mul_prev, (unsigned long long)mul_cur, (unsigned long long)buckets};
+    cudaError_t e = launch_pdl(pair_rows_kernel, dim3(B), dim3(256), 0, stream, tokens, cu_seqlens, past_lens, slots, last,
+                               rows, h);
+    return e == cudaSuccess ? launch_status() : (int)e;
+}
+
+namespace zlm {
+template <typename TW, typename TB>
+static cudaError_t launch_embed_pairs(const void* table, const void* pairs, const int* tokens, const int* rows,
+                                      const int* past_lens, const int* slots, int* last, PairHash h, float* out,
+                                      float* kept, int T, int d, float scale, cudaStream_t stream) {
+    const bool vec = d % 4 == 0 && (((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)out | (uintptr_t)kept) % 16) == 0;
+    const int threads = d >= 1024 ? 256 : (d >= 512 ? 128 : 64);
+    return vec ? launch_pdl(embed_pairs_kernel<TW, TB, true>, dim3(T), dim3(threads), 0, stream, (const TW*)table,
+                            (const TB*)pairs, tokens, rows, past_lens, slots, last, h, out, kept, d, scale)
+               : launch_pdl(embed_pairs_kernel<TW, TB, false>, dim3(T), dim3(threads), 0, stream, (const TW*)table,
+                            (const TB*)pairs, tokens, rows, past_lens, slots, last, h, out, kept, d, scale);
+}
+}  // namespace zlm
+
+ZLM_EXPORT int zlm_embed_pairs(const void* table, int table_dtype, const void* pairs, int pairs_dtype, const int* tokens,
+                               const int* rows, const int* past_lens, const int* slots, int* last, long mul_prev,
+                               long mul_cur, long buckets, float* out, float* kept, int T, int d, float scale,
+                               cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (d <= 0 || mul_prev < 0 || mul_cur < 0 || buckets <= 0 || buckets > 0x7ffffffeL) return ZLM_ERR_BAD_ARG;
+    const PairHash h{(unsigned long long)mul_prev, (unsigned long long)mul_cur, (unsigned long long)buckets};
+    const bool tf = table_dtype == ZLM_F32, pf = pairs_dtype == ZLM_F32;
+    if ((!tf && table_dtype != ZLM_BF16) || (!pf && pairs_dtype != ZLM_BF16)) return ZLM_ERR_UNSUPPORTED;
+    cudaError_t e;
+    if (tf && pf)
+        e = launch_embed_pairs<float, float>(table, pairs, tokens, rows, past_lens, slots, last, h, out, kept, T, d, scale, stream);
+    else if (tf)
+        e = launch_embed_pairs<float, __nv_bfloat16>(table, pairs, tokens, rows, past_lens, slots, last, h, out, kept, T, d, scale, stream);
+    else if (pf)
+        e = launch_embed_pairs<__nv_bfloat16, float>(table, pairs, tokens, rows, past_lens, slots, last, h, out, kept, T, d, scale, stream);
+    else
+        e = launch_embed_pairs<__nv_bfloat16, __nv_bfloat16>(table, pairs, tokens, rows, past_lens, slots, last, h, out, kept, T, d, scale, stream);
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 

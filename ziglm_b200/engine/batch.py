@@ -73,6 +73,7 @@ class StepContext:
     host_past_lens: List[int] = field(default_factory=list)
     host_new_lens: List[int] = field(default_factory=list)
     host_slots: List[int] = field(default_factory=list)
+    kept: Dict[str, torch.Tensor] = field(default_factory=dict)     # rows a hook reads later in the step, by name
 
 
 def pack_batch(layout: BatchLayout, host: torch.Tensor, slots: Sequence[int], past_lens: Sequence[int],

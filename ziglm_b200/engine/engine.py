@@ -254,7 +254,7 @@ class Engine:
             block_tables=v["block_tables"], single_token=single, max_new=max_new, max_total=max_total,
             dtype=self.dtype, device=self.device, ws=ws, host_past_lens=past, host_new_lens=new_lens,
             host_slots=slots)
-        step.io = [self.cache.io_for(place, step.block_tables) for place in range(len(self.spec.schedule))]
+        step.io = [self.cache.io_for(place, step.block_tables) for place in range(len(self.cache.reads_from))]
         return step
 
     # ------------------------------------------------------- decode steps as CUDA graphs

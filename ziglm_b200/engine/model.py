@@ -58,6 +58,8 @@ class Model:
         self.embed_hook = hook_class(spec.embed_hook.kind)(spec.embed_hook, dtype, device) if spec.embed_hook else None
         self.logits_hook = hook_class(spec.logits_hook.kind)(spec.logits_hook, dtype, device) if spec.logits_hook else None
         self.place_hooks = {place: hook_class(h.kind)(h, dtype, device) for place, h in spec.place_hooks.items()}
+        # a hook between two places may read the embedded tokens again: they are then kept beside the residual
+        self.keeps_embedding = any("embedding" in getattr(h, "reads_kept", ()) for h in self.place_hooks.values())
         self.embedding: Optional[torch.Tensor] = None
         self.head: Optional[Linear] = None
 
@@ -113,19 +115,45 @@ class Model:
                 reads.append(None)
             state.append(block.state_needs())
             last_place_of[li] = place
+        need = self._embed_hook_state()
+        if need is not None:
+            # the embedding's own state (the token before the step's first) is a place behind the schedule
+            kv.append(None)
+            reads.append(None)
+            state.append(need)
         return kv, reads, state
 
-    # ------------------------------------------------------------------ forward
-    def forward(self, step: StepContext) -> Optional[torch.Tensor]:
-        """Run the step's tokens through the layers; float32 logits [n_want, vocab] or None."""
+    def _embed_hook_state(self) -> Optional[StateNeed]:
+        needs = getattr(self.embed_hook, "state_needs", None)
+        return needs() if needs is not None else None
+
+    def _embed(self, step: StepContext) -> torch.Tensor:
+        """The residual stream of the step's tokens as the first layer finds it."""
         spec = self.spec
         x = step.ws.buf("residual", (step.n_tokens, spec.streams * spec.width), torch.float32)
+        kept = step.ws.buf("kept_embedding", tuple(x.shape), torch.float32) if self.keeps_embedding else None
+        if kept is not None:
+            step.kept["embedding"] = kept
+        if hasattr(self.embed_hook, "embed"):
+            # a hook that is more than a function of the residual looks the tokens up itself
+            io = step.io[len(spec.schedule)] if self._embed_hook_state() is not None else None
+            self.embed_hook.embed(step, io, self.embedding, spec.embedding_scale, x, kept)
+            return x
         if spec.streams > 1:
             kernels.embed_streams(self.embedding, step.tokens, x, spec.streams, spec.embedding_scale)
         else:
             kernels.embed(self.embedding, step.tokens, x, spec.embedding_scale)
         if self.embed_hook is not None:
             self.embed_hook.forward(step, x)
+        if kept is not None:
+            kept.copy_(x)
+        return x
+
+    # ------------------------------------------------------------------ forward
+    def forward(self, step: StepContext) -> Optional[torch.Tensor]:
+        """Run the step's tokens through the layers; float32 logits [n_want, vocab] or None."""
+        spec = self.spec
+        x = self._embed(step)
         carried = None           # the next block's first norm, half done by the block before (steps of few tokens)
         for place, li in enumerate(spec.schedule):
             block = self.blocks[li]

@@ -63,7 +63,10 @@ _PROTOTYPES = {
                          c_void_p],
         "zlm_unary_act": [c_void_p, c_void_p, c_int, c_long, c_int, c_void_p],
         "zlm_sigmoid_mul": [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_void_p],
-        "zlm_add_row": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+        "zlm_add_row": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+        "zlm_pair_rows": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_long, c_long, c_long, c_void_p],
+        "zlm_embed_pairs": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_long, c_long,
+                            c_long, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
         "zlm_convert_rows": [c_void_p, c_int, c_long, c_void_p, c_int, c_long, c_int, c_int, c_void_p],
         "zlm_gate_heads": [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_float, c_void_p],
         "zlm_norm_gate": [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_float,
@@ -142,18 +145,21 @@ _PROTOTYPES = {
                            c_void_p, c_int, c_void_p, c_void_p, c_int, c_long, c_void_p],
         "zlm_rope_norm_store": [c_void_p, c_int, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_int,
                                 c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                                c_int, c_long, c_void_p],
+                                c_int, c_long, c_int, c_void_p],
         "zlm_attention_general": [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int,
-                                  c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_long,
+                                  c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_long,
                                   c_int, c_void_p, c_long, c_void_p],
         "zlm_qk_prep": [c_void_p, c_int, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
                         c_int, c_float, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                         c_void_p, c_int, c_long, c_void_p],
+        "zlm_latent_prep": [c_void_p, c_long, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_long, c_void_p,
+                            c_int, c_long, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                            c_int, c_long, c_void_p],
         "zlm_attention_general_scratch": [c_int, c_int, c_int, c_int, c_int],
     },
     "attention_tc": {
         "zlm_attention_decode": [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int,
-                                 c_void_p, c_void_p, c_long, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int, c_int,
+                                 c_void_p, c_void_p, c_void_p, c_long, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int, c_int,
                                  c_void_p, c_void_p, c_void_p],
         "zlm_attention_decode_flat": [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p,
                                       c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int, c_int, c_void_p,
@@ -167,7 +173,7 @@ _PROTOTYPES = {
     },
     "attention_fmha": {
         "zlm_attention_prefill_fmha": [c_void_p, c_long, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                                       c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                       c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                        c_void_p, c_long, c_int, c_void_p],
         "zlm_attention_fmha_status": [c_void_p],
         "zlm_attention_fmha_wait_selftest": [c_int, c_void_p, c_void_p],
@@ -480,13 +486,45 @@ def head_norm_gate(x: torch.Tensor, weight: Optional[torch.Tensor], gate: Option
         float(mult), _stream()), "head_norm_gate")
 
 
-def add_row(x: torch.Tensor, row: torch.Tensor) -> None:
-    """x[t, :] += row for every t; x is float32 [T, d], row holds d elements."""
+def add_row(x: torch.Tensor, row: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+    """x[t, :] <- (x[t, :] + rows[t, :]) + row for every t; x and ``rows`` (None: left out) are float32 [T, d], ``row``
+    holds d elements."""
     _cuda(x, "x", torch.float32); _cuda(row, "row")
     if x.dim() != 2 or row.numel() != x.shape[1]:
         raise KernelError("add_row: the row must be as wide as x")
-    _check(_fn("elementwise", "zlm_add_row")(x.data_ptr(), row.data_ptr(), code(row.dtype), x.shape[0], x.shape[1],
-                                             _stream()), "add_row")
+    if rows is not None:
+        _cuda(rows, "rows", torch.float32)
+        if rows.shape != x.shape:
+            raise KernelError("add_row: the rows must have x's shape")
+    _check(_fn("elementwise", "zlm_add_row")(x.data_ptr(), _ptr(rows), row.data_ptr(), code(row.dtype), x.shape[0],
+                                             x.shape[1], _stream()), "add_row")
+
+
+def embed_pairs(table: torch.Tensor, pairs: torch.Tensor, last: torch.Tensor, mul_prev: int, mul_cur: int, step,
+                out: torch.Tensor, kept: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+    """out[t, :] = table[token_t] * scale + pairs[r_t] for the step's tokens, float32 [T, d]; r_t =
+    (token before * ``mul_prev`` + token_t * ``mul_cur``) mod (rows of ``pairs`` - 1), and the last row of ``pairs`` for a
+    token at position 0.  ``last`` (int32, one number a slot): the token before a step's first one, which the call reads
+    and replaces by the step's last token of every sequence.  ``kept`` (like ``out``): receives a copy."""
+    _cuda(table, "table"); _cuda(pairs, "pairs"); _cuda(last, "last", torch.int32); _cuda(out, "out", torch.float32)
+    T, d = out.shape
+    if table.shape[1] != d or pairs.shape[1] != d or pairs.shape[0] < 2 or step.tokens.numel() < T:
+        raise KernelError("embed_pairs: shapes do not match")
+    if kept is not None:
+        _cuda(kept, "kept", torch.float32)
+        if kept.shape != out.shape:
+            raise KernelError("embed_pairs: the copy must have the shape of the result")
+    buckets = pairs.shape[0] - 1
+    rows = None
+    if not (step.single_token and T == step.n_seqs):
+        rows = step.ws.buf("pair_rows", (T,), torch.int32)
+        _check(_fn("elementwise", "zlm_pair_rows")(
+            step.tokens.data_ptr(), step.cu_seqlens.data_ptr(), step.past_lens.data_ptr(), step.slots.data_ptr(),
+            last.data_ptr(), rows.data_ptr(), step.n_seqs, int(mul_prev), int(mul_cur), buckets, _stream()), "pair_rows")
+    _check(_fn("elementwise", "zlm_embed_pairs")(
+        table.data_ptr(), code(table.dtype), pairs.data_ptr(), code(pairs.dtype), step.tokens.data_ptr(), _ptr(rows),
+        step.past_lens.data_ptr(), step.slots.data_ptr(), last.data_ptr(), int(mul_prev), int(mul_cur), buckets,
+        out.data_ptr(), _ptr(kept), T, d, float(scale), _stream()), "embed_pairs")
 
 
 def scale_(x: torch.Tensor, factor: float) -> None:
@@ -1119,17 +1157,18 @@ def rope_norm_store(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, r
                     positions: torch.Tensor, seq_of_token: torch.Tensor, block_table: torch.Tensor,
                     k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], page_size: int,
                     norm_first: bool = False, q_weight: Optional[torch.Tensor] = None,
-                    k_weight: Optional[torch.Tensor] = None) -> None:
+                    k_weight: Optional[torch.Tensor] = None, values_from_keys: bool = False) -> None:
     """``rope_store`` with an amplitude on the cosines and sines and a unit RMS norm behind the rotation: every
     q and k head of a row [q heads | k heads | v heads | ...] of qkv is turned, divided by
     sqrt(mean of the squares of its first ``norm_dim`` dimensions + norm_eps) (``norm_dim`` 0: not divided), written
     back and (keys, values) stored in the cache pages.  The row may be wider than the heads.  With ``norm_first`` the
     norm stands before the rotation, and ``q_weight`` / ``k_weight`` (float32 [head_dim], one for all query heads and
-    one for all key heads; None: no weight) multiply the normed heads."""
+    one for all key heads; None: no weight) multiply the normed heads.  With ``values_from_keys`` a row holds no values:
+    it is [q heads | k heads | ...], and a key head as the row holds it, before norm and rotation, is stored as the value."""
     _rows(qkv, "qkv"); _cuda(positions, "positions", torch.int32); _cuda(seq_of_token, "seq_of_token", torch.int32)
     _cuda(block_table, "block_table", torch.int32)
     T = qkv.shape[0]
-    if qkv.shape[1] < (n_heads + 2 * n_kv) * head_dim:
+    if qkv.shape[1] < (n_heads + (1 if values_from_keys else 2) * n_kv) * head_dim:
         raise KernelError("rope_norm_store: the rows are narrower than the heads")
     if inv_freq is not None:
         _cuda(inv_freq, "inv_freq", torch.float32)
@@ -1151,8 +1190,39 @@ def rope_norm_store(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, r
         qkv.data_ptr(), code(qkv.dtype), _row_stride(qkv), T, n_heads, n_kv, head_dim, rotary_dim, _ptr(inv_freq),
         float(amplitude), int(norm_dim), float(norm_eps), int(bool(norm_first)), _ptr(q_weight), _ptr(k_weight),
         positions.data_ptr(), seq_of_token.data_ptr(),
-        block_table.data_ptr(), block_table.stride(0), _ptr(k_pages), _ptr(v_pages), page_size, page_stride, _stream()),
-        "rope_norm_store")
+        block_table.data_ptr(), block_table.stride(0), _ptr(k_pages), _ptr(v_pages), page_size, page_stride,
+        int(bool(values_from_keys)), _stream()), "rope_norm_store")
+
+
+def latent_prep(down: torch.Tensor, c_off: int, rank: int, r_off: int, rotary_dim: int, weight: torch.Tensor, eps: float,
+                q: torch.Tensor, q_out: torch.Tensor, n_heads: int, inv_freq: Optional[torch.Tensor],
+                positions: torch.Tensor, seq_of_token: torch.Tensor, block_table: torch.Tensor, pages: torch.Tensor,
+                page_size: int) -> None:
+    """What stands between the projections and the scores of an attention through a latent.  Of every row of ``down``
+    (float32 [T, ...]) the ``rank`` columns from ``c_off`` on are RMS-normed with ``weight`` (float32) and the
+    ``rotary_dim`` columns from ``r_off`` on turned by the token's position (pairs i, i + rotary_dim/2), and
+    [turned | normed | zeros] becomes the token's row of ``pages`` [n_pages, 1, page_size, size].  Every query head of
+    ``q`` ([T, n_heads * (dim + rotary_dim)], float32 or the pages' type) goes to ``q_out`` (the pages' type; may be ``q``)
+    with its last ``rotary_dim`` elements turned."""
+    _rows(down, "down"); _rows(q, "q"); _rows(q_out, "q_out"); _cuda(weight, "weight", torch.float32)
+    _cuda(positions, "positions", torch.int32); _cuda(seq_of_token, "seq_of_token", torch.int32)
+    _cuda(block_table, "block_table", torch.int32); _cuda(pages, "pages", q_out.dtype)
+    T = q.shape[0]
+    if down.dtype != torch.float32 or down.shape[0] != T or q_out.shape != q.shape or q.shape[1] % n_heads \
+            or weight.numel() != rank or max(c_off + rank, r_off + rotary_dim) > down.shape[1]:
+        raise KernelError("latent_prep: shapes do not match")
+    if pages.dim() != 4 or pages.shape[1] != 1 or pages.shape[2] != page_size or pages.shape[3] < rank + rotary_dim:
+        raise KernelError("latent_prep: cache pages must be [n_pages, 1, page_size, size]")
+    if rotary_dim:
+        _cuda(inv_freq, "inv_freq", torch.float32)
+        if inv_freq.numel() * 2 != rotary_dim or rotary_dim > q.shape[1] // n_heads:
+            raise KernelError("latent_prep: the frequency table must hold rotary_dim/2 entries")
+    _check(_fn("attention", "zlm_latent_prep")(
+        down.data_ptr(), _row_stride(down), c_off, rank, r_off, rotary_dim, weight.data_ptr(), float(eps), q.data_ptr(),
+        code(q.dtype), _row_stride(q), q_out.data_ptr(), code(q_out.dtype), _row_stride(q_out), T, n_heads,
+        q.shape[1] // n_heads - rotary_dim, _ptr(inv_freq), positions.data_ptr(), seq_of_token.data_ptr(),
+        block_table.data_ptr(), block_table.stride(0), pages.data_ptr(), pages.shape[3], page_size, pages.stride(0),
+        _stream()), "latent_prep")
 
 
 def qk_prep(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, rotary_dim: int,
@@ -1258,15 +1328,28 @@ def attention_general_scratch(n_tokens: int, n_heads: int, n_kv: int, head_dim: 
     return int(_fn("attention", "zlm_attention_general_scratch")(n_tokens, n_heads, n_kv, head_dim, max_keys))
 
 
+def _head_numbers(t: Optional[torch.Tensor], n_heads: int, name: str) -> Optional[int]:
+    """Pointer of a float32 tensor of one number per query head (None: no such numbers)."""
+    if t is None:
+        return None
+    _cuda(t, name, torch.float32)
+    if t.numel() != n_heads:
+        raise KernelError(f"attention: one number of {name} per query head is needed")
+    return t.data_ptr()
+
+
 def attention_general(qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, scale: float,
                       window: Optional[int], positions: torch.Tensor, seq_of_token: torch.Tensor,
                       block_table: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                       page_size: int, max_keys: int = 0, scratch: Optional[torch.Tensor] = None,
-                      softcap: float = 0.0, keep_first: int = 0, sinks: Optional[torch.Tensor] = None) -> None:
+                      softcap: float = 0.0, keep_first: int = 0, sinks: Optional[torch.Tensor] = None,
+                      slopes: Optional[torch.Tensor] = None) -> None:
     """out[t, h, :] = softmax(q[t,h] . K[start..pos_t] * scale) @ V over the paged cache; with ``softcap`` c > 0 the
     scaled scores become c * tanh(score / c) before the softmax.  With a window, the first ``keep_first`` positions
     of a sequence stay visible behind it.  ``sinks`` (float32, one per query head): exp(sinks[h]) is added to the
-    softmax's denominator; it has no key and no value and is not scaled.
+    softmax's denominator; it has no key and no value and is not scaled.  ``slopes`` (float32, one positive number per
+    query head): the score of the key at position j (scaled, and capped if it is) is made less by
+    slopes[h] * (pos_t - j).
 
     The queries are the first n_heads*head_dim columns of each row of ``qkv`` (any row stride).
     ``max_keys`` (the most keys a token of the step sees) and ``scratch`` (float32, at least
@@ -1285,13 +1368,10 @@ def attention_general(qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: 
         raise KernelError(f"attention: head size {head_dim} is not supported (a multiple of 8, at most 512)")
     if tuple(k_pages.shape[1:]) != (n_kv, page_size, head_dim) or k_pages.shape != v_pages.shape:
         raise KernelError("attention: cache pages must be [n_pages, n_kv, page_size, head_dim]")
-    if sinks is not None:
-        _cuda(sinks, "sinks", torch.float32)
-        if sinks.numel() != n_heads:
-            raise KernelError("attention: one sink per query head is needed")
     _check(_fn("attention", "zlm_attention_general")(
         qkv.data_ptr(), qkv.stride(0), out.data_ptr(), code(qkv.dtype), T, n_heads, n_kv, head_dim, scale,
-        float(softcap or 0.0), int(window or 0), int(keep_first or 0), _ptr(sinks), positions.data_ptr(), seq_of_token.data_ptr(), block_table.data_ptr(),
+        float(softcap or 0.0), int(window or 0), int(keep_first or 0), _head_numbers(sinks, n_heads, "sinks"),
+        _head_numbers(slopes, n_heads, "slopes"), positions.data_ptr(), seq_of_token.data_ptr(), block_table.data_ptr(),
         block_table.stride(0), k_pages.data_ptr(), v_pages.data_ptr(), page_size, k_pages.stride(0), int(max_keys),
         _ptr(scratch), scratch.numel() if scratch is not None else 0, _stream()),
         "attention_general")
@@ -1311,9 +1391,10 @@ def attention_decode(qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: i
                      block_table: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, page_size: int,
                      n_splits: int, part_o: torch.Tensor, part_ml: torch.Tensor, softcap: float = 0.0,
                      keep_first: int = 0, sinks: Optional[torch.Tensor] = None,
-                     head_gate: Optional[torch.Tensor] = None, head_gate_mult: float = 1.0) -> bool:
-    """Tensor-core attention for steps of one token per sequence (bf16, head size 64 or 128); ``keep_first`` and
-    ``sinks`` as :func:`attention_general` takes them.  ``head_gate`` ([T, n_heads] of the rows' type, a row stride of
+                     head_gate: Optional[torch.Tensor] = None, head_gate_mult: float = 1.0,
+                     slopes: Optional[torch.Tensor] = None) -> bool:
+    """Tensor-core attention for steps of one token per sequence (bf16, head size 64 or 128); ``keep_first``,
+    ``sinks`` and ``slopes`` (not with kept first tokens) as :func:`attention_general` takes them.  ``head_gate`` ([T, n_heads] of the rows' type, a row stride of
     its own): head h of token t leaves multiplied by sigmoid(head_gate[t, h]) * ``head_gate_mult``.
 
     Each token's query heads are grouped by key/value head so that the cache is read once per group; the keys
@@ -1333,17 +1414,14 @@ def attention_decode(qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: i
         raise KernelError("attention_decode: cache pages must be [n_pages, n_kv, page_size, head_dim]")
     if part_o.numel() < T * n_heads * n_splits * head_dim or part_ml.numel() < T * n_heads * n_splits * 2:
         raise KernelError("attention_decode: the scratch is too small for this many splits")
-    if sinks is not None:
-        _cuda(sinks, "sinks", torch.float32)
-        if sinks.numel() != n_heads or not sinks.is_contiguous():
-            raise KernelError("attention_decode: one sink per query head is needed")
     if head_gate is not None:
         _rows(head_gate, "head_gate")
         if head_gate.dtype != qkv.dtype or tuple(head_gate.shape) != (T, n_heads):
             raise KernelError("attention_decode: the gates must be [T, n_heads] of the rows' type")
     status = _fn("attention_tc", "zlm_attention_decode")(
         qkv.data_ptr(), qkv.stride(0), out.data_ptr(), T, n_heads, n_kv, head_dim, scale, float(softcap or 0.0),
-        int(window or 0), int(keep_first or 0) if (window or 0) > 0 else 0, _ptr(sinks), _ptr(head_gate),
+        int(window or 0), int(keep_first or 0) if (window or 0) > 0 else 0, _head_numbers(sinks, n_heads, "sinks"),
+        _head_numbers(slopes, n_heads, "slopes"), _ptr(head_gate),
         _row_stride(head_gate) if head_gate is not None else 0, float(head_gate_mult),
         positions.data_ptr(), seq_of_token.data_ptr(), block_table.data_ptr(), block_table.stride(0),
         k_pages.data_ptr(), v_pages.data_ptr(), k_pages.shape[0], page_size, n_splits, part_o.data_ptr(),
@@ -1472,14 +1550,10 @@ def attention_prefill_fmha(qkv: torch.Tensor, out: torch.Tensor, n_seqs: int, ma
                            head_dim: int, scale: float, window: Optional[int], cu_seqlens: torch.Tensor,
                            past_lens: torch.Tensor, block_table: torch.Tensor, k_pages: torch.Tensor,
                            v_pages: torch.Tensor, page_size: int, softcap: float = 0.0, keep_first: int = 0,
-                           sinks: Optional[torch.Tensor] = None) -> bool:
+                           sinks: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None) -> bool:
     """Prompt attention on the tcgen05 tensor cores (tiles of 128 queries, accumulators in tensor memory); same
-    arguments as :func:`attention_prefill`, and ``keep_first`` / ``sinks`` as :func:`attention_general` takes them.
-    False if refused."""
-    if sinks is not None:
-        _cuda(sinks, "sinks", torch.float32)
-        if sinks.numel() != n_heads or not sinks.is_contiguous():
-            raise KernelError("attention_prefill_fmha: one sink per query head is needed")
+    arguments as :func:`attention_prefill`, and ``keep_first`` / ``sinks`` / ``slopes`` as :func:`attention_general`
+    takes them.  False if refused."""
     _cuda(out, "out", torch.bfloat16); _cuda(k_pages, "k_pages", torch.bfloat16); _cuda(v_pages, "v_pages", torch.bfloat16)
     _cuda(cu_seqlens, "cu_seqlens", torch.int32); _cuda(past_lens, "past_lens", torch.int32)
     _cuda(block_table, "block_table", torch.int32)
@@ -1493,7 +1567,8 @@ def attention_prefill_fmha(qkv: torch.Tensor, out: torch.Tensor, n_seqs: int, ma
         raise KernelError("attention_prefill_fmha: sequence arrays are too short")
     status = _fn("attention_fmha", "zlm_attention_prefill_fmha")(
         qkv.data_ptr(), qkv.stride(0), qkv.shape[0], out.data_ptr(), n_seqs, max_new, n_heads, n_kv, head_dim, scale,
-        float(softcap or 0.0), int(window or 0), int(keep_first or 0) if (window or 0) > 0 else 0, _ptr(sinks), cu_seqlens.data_ptr(),
+        float(softcap or 0.0), int(window or 0), int(keep_first or 0) if (window or 0) > 0 else 0,
+        _head_numbers(sinks, n_heads, "sinks"), _head_numbers(slopes, n_heads, "slopes"), cu_seqlens.data_ptr(),
         past_lens.data_ptr(), block_table.data_ptr(), block_table.stride(0), k_pages.data_ptr(), v_pages.data_ptr(),
         k_pages.shape[0], page_size, _stream())
     if status == -2:
@@ -1552,7 +1627,7 @@ def attention_with_rope(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int
 def attention(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, scale: float,
               window: Optional[int], io, softcap: float = 0.0, gate: Optional[torch.Tensor] = None,
               keep_first: int = 0, sinks: Optional[torch.Tensor] = None, head_gate: Optional[torch.Tensor] = None,
-              head_gate_mult: float = 1.0, chunk: Optional[int] = None) -> bool:
+              head_gate_mult: float = 1.0, chunk: Optional[int] = None, slopes: Optional[torch.Tensor] = None) -> bool:
     """Attention of a step's tokens over the cache of the running layer; picks the kernel.  ``chunk`` (instead of
     ``window``): the positions of a sequence form chunks of that many, counted from its start, and a query sees the
     earlier keys of its own chunk only (the kernels take it as a negative window).  ``softcap`` c > 0:
@@ -1563,7 +1638,8 @@ def attention(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: in
     (the caller multiplies when it was not: in a prompt one pass of ``sigmoid_mul`` over coalesced rows costs less
     than the same work in the prompt kernel's epilogue, where every thread walks a row of its own).  ``head_gate``
     ([T, n_heads], instead of ``gate``): one gate a head, times ``head_gate_mult``; the decode kernel that splits a
-    sequence's keys applies it where it combines the splits, and the result says so likewise."""
+    sequence's keys applies it where it combines the splits, and the result says so likewise.  ``slopes`` (float32, one
+    positive number per query head): a score is made less by slopes[h] for every position between query and key."""
     if gate is not None and head_gate is not None:
         raise KernelError("attention: a gate an element or a gate a head, not both")
     if chunk:
@@ -1575,9 +1651,9 @@ def attention(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: in
     else:
         keep_first = int(keep_first or 0) if window else 0
         span = min(step.max_total, window + keep_first) if window else step.max_total
-    # kept first tokens and sinks: the tcgen05 prompt kernel and the decode kernel that splits a sequence's keys
-    # know both, the other tensor-core kernels neither
-    plain_only = keep_first > 0 or sinks is not None
+    # kept first tokens, sinks and slopes: the tcgen05 prompt kernel and the decode kernel that splits a sequence's
+    # keys know them, the other tensor-core kernels do not
+    plain_only = keep_first > 0 or sinks is not None or slopes is not None
     if plain_only and _tc_attention_ok(qkv.dtype, n_heads, n_kv, head_dim, io.page_size):
         if step.single_token:
             n_splits = decode_splits(step.n_tokens, n_kv, span, io.page_size)
@@ -1586,12 +1662,12 @@ def attention(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: in
             if attention_decode(qkv, out, n_heads, n_kv, head_dim, scale, window, step.positions, step.seq_of_token,
                                 io.block_table, io.k_pages, io.v_pages, io.page_size, n_splits, part_o, part_ml,
                                 softcap=softcap, keep_first=keep_first, sinks=sinks, head_gate=head_gate,
-                                head_gate_mult=head_gate_mult):
+                                head_gate_mult=head_gate_mult, slopes=slopes):
                 return head_gate is not None
         elif step.max_new >= 16 and attention_prefill_fmha(
                 qkv, out, step.n_seqs, step.max_new, n_heads, n_kv, head_dim, scale, window, step.cu_seqlens,
                 step.past_lens, io.block_table, io.k_pages, io.v_pages, io.page_size, softcap=softcap,
-                keep_first=keep_first, sinks=sinks):
+                keep_first=keep_first, sinks=sinks, slopes=slopes):
             return False
     if not plain_only and _tc_attention_ok(qkv.dtype, n_heads, n_kv, head_dim, io.page_size):
         n_blocks = attention_decode_flat_blocks(step.n_tokens, n_heads, n_kv, head_dim) if step.single_token else 0
@@ -1624,7 +1700,7 @@ def attention(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: in
     scratch = step.ws.buf("attn_parts", (need,), torch.float32) if need > 0 else None
     attention_general(qkv, out, n_heads, n_kv, head_dim, scale, window, step.positions, step.seq_of_token,
                       io.block_table, io.k_pages, io.v_pages, io.page_size, max_keys, scratch, softcap=softcap,
-                      keep_first=keep_first, sinks=sinks)
+                      keep_first=keep_first, sinks=sinks, slopes=slopes)
     return False
 
 

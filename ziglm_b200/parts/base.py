@@ -19,7 +19,12 @@ FeedForward     ``forward(step, h, residual)``: adds its output to ``residual``.
 Block           ``forward(step, io, x)``: runs its parts on the residual stream x.
 Hook            ``forward(step, x)``: changes x in place; x is the float32 residual
                 [T, d] after the embedding (``ModelSpec.embed_hook``) or the float32
-                logits [n_want, vocab] (``ModelSpec.logits_hook``).
+                logits [n_want, vocab] (``ModelSpec.logits_hook``).  An embedding hook that
+                is more than a function of x offers ``embed(step, io, table, scale, x, kept)``
+                instead, which fills x from the step's tokens (and ``kept`` with a copy if it
+                is not None), and may ask for state (``state_needs``).  A hook before a place
+                of the schedule names what it reads of ``StepContext.kept`` in ``reads_kept``
+                ("embedding": the residual as the first layer found it).
 
 A norm that rides on its neighbours
 -----------------------------------

@@ -363,7 +363,7 @@ class SharedNormBlock(Part):
     """One norm whose rows the mixer and the feed-forward both read: with h = norm(x), x += mixer(h) + ff(h).
 
     The two sublayers add into the float32 residual one after the other; neither reads what the other wrote, so the
-    sum is the arrangement's.  A layer whose spec has no feed-forward ends after the mixer.  ``spec.ffn_norm`` is not
+    sum is the arrangement's.  In steps of few tokens the norm rides on the products around it, where the parts can.  A layer whose spec has no feed-forward ends after the mixer.  ``spec.ffn_norm`` is not
     used (it is None)."""
 
     def __init__(self, spec: LayerSpec, dtype: torch.dtype, device: torch.device):
@@ -410,15 +410,24 @@ class SharedNormBlock(Part):
         return self.mixer.state_needs()
 
     def accepts_normed_input(self) -> bool:
-        """The block before may hand this block's norm over as finished rows (``h_in``); a norm half done by a
-        product is not taken, since two sublayers would have to complete it."""
-        return False
+        """Whether ``forward`` may be handed this block's norm half done (``h_in``): both sublayers' first products then
+        complete it."""
+        return bool(self.mixer_norm.fusable and self.mixer.takes_normed_input
+                    and (self.ffn is None or self.ffn.takes_normed_input))
 
     def forward(self, step, io: LayerIO, x: torch.Tensor, h_in=None, next_norm=None):
-        h = h_in if isinstance(h_in, torch.Tensor) else self.mixer_norm.forward(step, x)
+        """``h_in``: this block's norm, half done by the block before (else the norm kernel runs).  ``next_norm``: the
+        norm of the block after; the result is its half-done form if this block's last product did it, else None."""
+        h = h_in if h_in is not None else self.mixer_norm.forward(step, x)
+        if self.ffn is None:
+            if self.mixer.fuses_next_norm and next_norm is not None:
+                return self.mixer.forward(step, io, h, x, next_norm=next_norm)
+            self.mixer.forward(step, io, h, x)
+            return None
         self.mixer.forward(step, io, h, x)
-        if self.ffn is not None:
-            self.ffn.forward(step, h, x)
+        if self.ffn.fuses_next_norm and next_norm is not None:
+            return self.ffn.forward(step, h, x, next_norm=next_norm)
+        self.ffn.forward(step, h, x)
         return None
 
 

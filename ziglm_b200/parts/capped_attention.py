@@ -1,7 +1,7 @@
 """Grouped-query attention with the options of newer decoders, each of which may be left out.
 
 For the rows h the mixer reads, H query heads, G key/value heads, query/key size D and value size V:
-    q = W_q h + b_q,  k = W_k h + b_k,  v = W_v h + b_v
+    q = W_q h + b_q,  k = W_k h + b_k,  v = W_v h + b_v       (``values`` "keys": no W_v; v = k as projected, before its norm)
     q, k, v <- conv(q), conv(k), conv(v)        a causal convolution a channel over the last taps tokens  (``conv``: taps;
                                                 no bias, zeros before the start; the inputs are a state of the sequence)
     q, k <- q / rms(q) * w_q, k / rms(k) * w_k  q (all heads as one vector) and k likewise  (``qk_norm`` "whole")
@@ -14,6 +14,7 @@ For the rows h the mixer reads, H query heads, G key/value heads, query/key size
     v <- (1 - l) v + l v_first                  v_first: the values of the same tokens in the first layer that takes
                                                 part (``value_mix`` "mix"; that layer itself says "first"); l learned
     s_ij = (q_i . k_j) * scale;  s <- c tanh(s / c)                               (``softcap`` c; None: left out)
+    s_ij <- s_ij - slope_h (i - j)              slope_h = 2^(-B (h + 1) / H)      (``distance_bias`` B; None: left out)
     j visible to i:  j <= i and (i - j < window or j < keep_first)                (``MixerSpec.window``, ``keep_first``)
                      or j <= i and floor(i / c) = floor(j / c)                    (``chunk`` c instead of a window)
     p = softmax over the visible j, with exp(sink_h) also in the denominator       (``sink``: a learned number a head;
@@ -100,6 +101,16 @@ class CappedAttention(Part):
         self.conv = int(o.get("conv") or 0)
         if self.conv < 0:
             raise ValueError(f"capped_attention: a convolution of {self.conv} taps")
+        if o.get("values") not in (None, "keys"):
+            raise ValueError(f"capped_attention: values {o.get('values')!r} are not known (keys)")
+        self.values_from_keys = o.get("values") == "keys"
+        if self.values_from_keys and (self.value_dim != self.dim or self.conv or o.get("value_mix") is not None
+                                      or self.norm_kind == "whole"):
+            raise ValueError("capped_attention: values that are the keys have the keys' size and go with no convolution, "
+                             "no norm of the whole q and k and no mixed values")
+        self.distance_bias = None if o.get("distance_bias") is None else float(o["distance_bias"])
+        if self.distance_bias is not None and (not self.distance_bias > 0.0 or self.keep_first):
+            raise ValueError("capped_attention: the exponent of a distance bias is positive and goes with no kept first tokens")
         self.value_mix = o.get("value_mix")
         if self.value_mix not in (None, "first", "mix"):
             raise ValueError(f"capped_attention: value_mix {self.value_mix!r} is not known (first, mix)")
@@ -117,6 +128,7 @@ class CappedAttention(Part):
         self.q_norm_w: Optional[torch.Tensor] = None
         self.k_norm_w: Optional[torch.Tensor] = None
         self.sinks: Optional[torch.Tensor] = None
+        self.slopes: Optional[torch.Tensor] = None
         self.mix = 0.0
 
     @staticmethod
@@ -135,10 +147,14 @@ class CappedAttention(Part):
         H, G, D, d = spec.n_heads, spec.n_kv_heads, spec.head_dim, spec.width
         o = spec.options
         V = int(o.get("value_dim", D))
-        p = {"q.weight": ParamDecl((H * D, d)), "k.weight": ParamDecl((G * D, d)), "v.weight": ParamDecl((G * V, d)),
-             "o.weight": ParamDecl((d, H * V))}
+        own_values = o.get("values") != "keys"
+        p = {"q.weight": ParamDecl((H * D, d)), "k.weight": ParamDecl((G * D, d)), "o.weight": ParamDecl((d, H * V))}
+        if own_values:
+            p["v.weight"] = ParamDecl((G * V, d))
         if spec.bias:
-            p.update({"q.bias": ParamDecl((H * D,)), "k.bias": ParamDecl((G * D,)), "v.bias": ParamDecl((G * V,))})
+            p.update({"q.bias": ParamDecl((H * D,)), "k.bias": ParamDecl((G * D,))})
+            if own_values:
+                p["v.bias"] = ParamDecl((G * V,))
         if o.get("gate") == "sigmoid":
             p["g.weight"] = ParamDecl((H * V, d))
         elif o.get("gate") == "sigmoid_head":
@@ -161,7 +177,9 @@ class CappedAttention(Part):
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         H, G, D, V, P = self.n_heads, self.n_kv, self.dim, self.value_dim, self.kept
         order = self.position.head_order(D) if hasattr(self.position, "head_order") else None
-        parts = [("q", H, D, order), ("k", G, D, order), ("v", G, V, None)]
+        if self.values_from_keys and order is not None:
+            raise ValueError("capped_attention: values that are the keys cannot follow a position encoding that reorders heads")
+        parts = [("q", H, D, order), ("k", G, D, order)] + ([] if self.values_from_keys else [("v", G, V, None)])
         ws = [tensors[f"{n}.weight"] for n, _, _, _ in parts] + ([tensors["g.weight"]] if self.gated else [])
         wide = torch.float32 if any(w.dtype == torch.float32 for w in ws) else ws[0].dtype
         blocks = [_pad_heads(_order_heads(tensors[f"{n}.weight"].to(wide), heads, size, ordr), heads, size, P)
@@ -200,8 +218,12 @@ class CappedAttention(Part):
         if self.has_sink:
             self.sinks = (tensors["sink"].float().contiguous() if self.sink_learned
                           else torch.zeros(H, dtype=torch.float32, device=w_o.device))
+        if self.distance_bias is not None:
+            self.slopes = torch.tensor([2.0 ** (-self.distance_bias * (h + 1) / H) for h in range(H)], dtype=torch.float32,
+                                       device=w_o.device)
         if self.value_mix == "mix":
             self.mix = float(tensors["vmix"].float().item())
+        self.takes_normed_input = self.proj.takes_normed()
 
     def kernel_libraries(self) -> Tuple[str, ...]:
         libs = ("attention", "elementwise") + (("recurrent",) if self.conv else ())
@@ -223,12 +245,23 @@ class CappedAttention(Part):
         the decode kernel that turns the heads and writes the cache itself can do."""
         return (self.norm_kind is None and self.value_mix is None and not self.softcap and not self.gated
                 and not self.has_sink and self.chunk is None and self.keep_first == 0
+                and not self.values_from_keys and self.distance_bias is None
                 and float(getattr(self.position, "amplitude", 1.0)) == 1.0)
 
-    def forward(self, step, io: LayerIO, h: torch.Tensor, residual: torch.Tensor, accumulate: bool = True):
+    fuses_next_norm = True
+
+    def _close(self, step, out: torch.Tensor, residual: torch.Tensor, accumulate: bool, next_norm):
+        if not accumulate:
+            self.o(out, residual)
+            return None
+        return self.o.accumulate_with_norm(step, out, residual, next_norm, "attn_next")
+
+    def forward(self, step, io: LayerIO, h, residual: torch.Tensor, accumulate: bool = True, next_norm=None):
+        """``h``: the normalised rows or a half-done norm (:class:`NormedInput`).  With ``next_norm`` the output projection
+        may do the first half of that norm; the result is then its :class:`NormedInput`."""
         T = residual.shape[0]
         H, G, P = self.n_heads, self.n_kv, self.kept
-        heads_width = (H + 2 * G) * P
+        heads_width = (H + (1 if self.values_from_keys else 2) * G) * P
         proj = step.ws.buf("cattn_proj", (T, heads_width + self.gate_cols), self.dtype)
         self.proj(h, proj)
         gate = proj[:, heads_width:] if self.gate == "sigmoid" else None
@@ -243,8 +276,7 @@ class CappedAttention(Part):
         out = step.ws.buf("attn_out", (T, H * P), self.dtype)
         if self.conv and self._plain() and kernels.attention_with_rope(step, proj, out, H, G, P, self.scale, self.window, io,
                                                                        inv_freq, rot, io.writes_cache):
-            self.o(out, residual, accumulate=accumulate)
-            return None
+            return self._close(step, out, residual, accumulate, next_norm)
         k_pages, v_pages = (io.k_pages, io.v_pages) if io.writes_cache else (None, None)
         if self.norm_kind == "whole" or self.value_mix is not None:
             if amplitude != 1.0:
@@ -264,18 +296,18 @@ class CappedAttention(Part):
             kernels.rope_norm_store(proj, H, G, P, rot, inv_freq, amplitude, self.dim if head_norm else 0,
                                     (self.norm_eps or 0.0) if head_norm else 0.0, step.positions, step.seq_of_token,
                                     io.block_table, k_pages, v_pages, io.page_size, norm_first=first,
-                                    q_weight=self.q_norm_w if first else None, k_weight=self.k_norm_w if first else None)
+                                    q_weight=self.q_norm_w if first else None, k_weight=self.k_norm_w if first else None,
+                                    values_from_keys=self.values_from_keys)
         # the flat decode kernel multiplies by an element gate's sigmoid as it stores, the decode kernel that splits a
         # sequence's keys by a head's gate where it combines the splits; behind the others a kernel does
         gated = kernels.attention(step, proj, out, H, G, P, self.scale, self.window, io, softcap=self.softcap, gate=gate,
                                   keep_first=self.keep_first, sinks=self.sinks, head_gate=head_gate,
-                                  head_gate_mult=self.out_scale, chunk=self.chunk)
+                                  head_gate_mult=self.out_scale, chunk=self.chunk, slopes=self.slopes)
         if self.gate == "sigmoid" and not gated:
             kernels.sigmoid_mul(out, gate, out)
         elif self.gate == "sigmoid_head" and not gated:
             kernels.gate_heads(out, head_gate, out, H, self.out_scale)
-        self.o(out, residual, accumulate=accumulate)
-        return None
+        return self._close(step, out, residual, accumulate, next_norm)
 
 
 register_mixer("capped_attention", CappedAttention)

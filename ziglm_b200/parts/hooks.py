@@ -2,7 +2,11 @@
 
 ``add_row``   x[t, :] += table[row, :] for every token of the step: a learned vector added to the residual
               stream at a fixed place (the start of a pass through a repeated run of layers).  Options:
-              ``rows`` and ``width`` (the table's shape), ``row``.
+              ``rows`` and ``width`` (the table's shape), ``row``; ``add_embedding``: the residual as the first layer
+              found it is added before the row, x[t, :] <- (x[t, :] + embedded[t, :]) + table[row, :].
+``token_pairs``  the embedding of a token plus a row of a second table that its pair with the token before chooses: row
+              (before * mul_prev + token * mul_cur) mod buckets, and the last row, number ``buckets``, for a sequence's first
+              token.  The last token of a sequence is a state of it.  Options: ``buckets``, ``width``, ``mul_prev``, ``mul_cur``.
 ``scale``     logits *= factor.  Option: ``factor``.
 ``soft_cap``  logits <- cap tanh(logits / cap), in float32.  Option: ``cap``.
 ``rmsnorm``   x <- x / sqrt(mean(x^2) + eps) * (w + offset) over every row, in place and in float32: a norm of the
@@ -17,7 +21,7 @@ import torch
 
 from .. import kernels
 from ..config.spec import HookSpec
-from .base import ParamDecl, Part, register_hook
+from .base import LayerIO, ParamDecl, Part, StateNeed, register_hook
 
 
 class AddRow(Part):
@@ -26,6 +30,7 @@ class AddRow(Part):
         self.row_index = int(spec.options["row"])
         if not 0 <= self.row_index < int(spec.options["rows"]):
             raise ValueError(f"add_row: row {self.row_index} is outside the table of {spec.options['rows']} rows")
+        self.reads_kept = ("embedding",) if spec.options.get("add_embedding") else ()
         self.row: Optional[torch.Tensor] = None
 
     @classmethod
@@ -39,7 +44,34 @@ class AddRow(Part):
         return ("elementwise",)
 
     def forward(self, step, x: torch.Tensor) -> None:
-        kernels.add_row(x, self.row)
+        kernels.add_row(x, self.row, rows=step.kept["embedding"] if self.reads_kept else None)
+
+
+class TokenPairs(Part):
+    def __init__(self, spec: HookSpec, dtype: torch.dtype, device: torch.device):
+        super().__init__(spec, dtype, device)
+        o = spec.options
+        self.mul_prev, self.mul_cur = int(o["mul_prev"]), int(o["mul_cur"])
+        if int(o["buckets"]) < 1 or min(self.mul_prev, self.mul_cur) < 0:
+            raise ValueError("token_pairs: at least one bucket and factors that are not negative are needed")
+        self.table: Optional[torch.Tensor] = None
+
+    @classmethod
+    def declare(cls, spec: HookSpec) -> Dict[str, ParamDecl]:
+        return {"table": ParamDecl((int(spec.options["buckets"]) + 1, int(spec.options["width"])))}
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.table = tensors["table"].contiguous()
+
+    def kernel_libraries(self) -> Tuple[str, ...]:
+        return ("elementwise",)
+
+    def state_needs(self) -> StateNeed:
+        return StateNeed((1,), torch.int32)
+
+    def embed(self, step, io: LayerIO, table: torch.Tensor, scale: float, x: torch.Tensor,
+              kept: Optional[torch.Tensor]) -> None:
+        kernels.embed_pairs(table, self.table, io.state, self.mul_prev, self.mul_cur, step, x, kept, scale)
 
 
 class Scale(Part):
@@ -94,6 +126,7 @@ class NormRows(Part):
 
 
 register_hook("add_row", AddRow)
+register_hook("token_pairs", TokenPairs)
 register_hook("rmsnorm", NormRows)
 register_hook("scale", Scale)
 register_hook("soft_cap", SoftCap)

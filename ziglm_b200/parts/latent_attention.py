@@ -7,7 +7,8 @@ latent sizes Rq, R:
     [c | r] = W_dkv h             c <- norm(c)             R and Rr elements a position (r is not normed)
     k_j = W_uk c_j,  v_j = W_uv c_j                        [H, D], [H, V]   (j: a position)
     s_ij = (q_i[:D] . k_j + rot(q_i[D:], i) . rot(r_j, j)) * scale,  j <= i and i - j < window
-    p = softmax_j(s);  o_i = sum_j p_ij v_j
+    p = softmax_j(s), with exp(sink_h) also in the denominator  (``sink``: a learned number a head; left out: a plain softmax)
+    o_i = sum_j p_ij v_j
     out = W_o (o * sigmoid(W_g h))                                          (``gate`` None: out = W_o o)
 Only c and the rotated r are kept per position: one vector of Rr + R elements that is key and value at once
 (``KVNeed(values_are_keys=True)``).  The products with W_uk and W_uv are moved to the other side of the
@@ -16,10 +17,12 @@ attention, head by head:
     l_i  = sum_j p_ij [rot(r_j) | c_j],                                      o_i  = W_uv[h] l_i[Rr:],
 so the attention itself is the library's attention of H query heads over one key/value head of size Rr + R
 whose keys and values are the same pages, and the two per-head products are block-diagonal products (the first also
-moves the rotated part of a query to the front of its head, in the order that makes the encoding's pairs the halves
-the rotation kernel turns; the second skips the first Rr elements).  The projections of h that are normed or gated
-(W_dq, W_dkv, W_g) are one matrix product with a float32 result: the norms of the latents and the gate's sigmoid
-read it in float32.
+moves the rotated part of a query to the front of its head; the second skips the first Rr elements).  The projections
+of h (W_dq or W_q, W_dkv, W_g) are one matrix product with a float32 result: the norms of the latents, the rotations
+and the gate's sigmoid read it in float32.  One kernel (``kernels.latent_prep``) stands between the projections and the
+first per-head product: it norms c, turns r and the queries' rotated parts, and writes the token's row of the cache.
+The rows of W_q and W_dkv that are rotated are taken in the order that makes the encoding's pairs the halves the kernel
+turns.
 """
 from __future__ import annotations
 
@@ -50,9 +53,8 @@ class LatentAttention(Part):
         if self.gate not in (None, "sigmoid"):
             raise ValueError(f"latent_attention: output gate {self.gate!r} is not known (sigmoid)")
         self.window = None if spec.window is None else int(spec.window)
-        # the attention kernels take head sizes that are multiples of 8: a latent of another size is kept with
-        # zeros behind it (they add nothing to a score and their part of the result is not read)
-        self.kept = -(-(self.rot_dim + self.kv_rank) // 8) * 8
+        self.has_sink = bool(o.get("sink"))
+        self.kept = self.kept_size(self.rot_dim + self.kv_rank, dtype)
         if self.kept > 512:
             raise ValueError(f"latent_attention: a key/value latent of {self.kv_rank} elements beside {self.rot_dim} "
                              "rotated ones is not supported (at most 512 together)")
@@ -63,15 +65,28 @@ class LatentAttention(Part):
         if not self.rot_dim and table is not None:
             raise ValueError("latent_attention: a rotation needs a rotated part of the keys (rot_dim)")
         eps = float(o["norm_eps"])
-        norm_kind = o.get("norm", "rmsnorm")
-        self.q_norm = (norm_class(norm_kind)(NormSpec(norm_kind, self.q_rank, eps), dtype, device)
+        self.norm_eps = eps
+        self.q_norm = (norm_class("rmsnorm")(NormSpec("rmsnorm", self.q_rank, eps), dtype, device)
                        if self.q_rank is not None else None)
-        self.kv_norm = norm_class(norm_kind)(NormSpec(norm_kind, self.kv_rank, eps), dtype, device)
-        self.down: Optional[Linear] = None       # [W_dq; W_dkv; W_g], whichever exist
-        self.uq: Optional[Linear] = None         # W_uq, or W_q when there is no query latent
+        self.kv_norm_w: Optional[torch.Tensor] = None
+        self.sinks: Optional[torch.Tensor] = None
+        self.down: Optional[Linear] = None       # [W_dq or W_q; W_dkv; W_g], the last where there is a gate
+        self.uq: Optional[Linear] = None         # W_uq where there is a query latent
         self.o: Optional[Linear] = None
         self.uk_t: Optional[torch.Tensor] = None  # [H, kept, D + Rr]: per head, a query into the latent's space
         self.uv: Optional[torch.Tensor] = None    # [H, V, kept]
+
+    @staticmethod
+    def kept_size(size: int, dtype: torch.dtype) -> int:
+        """The size a position's vector is kept with: a multiple of 8; in bfloat16 the next size the tensor-core attention
+        kernels take (64, 128) when that is at most a third more.  What lies behind the vector is zero: it adds nothing to
+        a score and its part of the result is not read."""
+        kept = -(-size // 8) * 8
+        if dtype == torch.bfloat16:
+            for fast in (64, 128):
+                if kept <= fast and fast * 3 <= kept * 4:
+                    return fast
+        return kept
 
     @classmethod
     def declare(cls, spec: MixerSpec) -> Dict[str, ParamDecl]:
@@ -88,6 +103,8 @@ class LatentAttention(Part):
             p["q.weight"] = ParamDecl((H * (D + Rr), d))
         if o.get("gate", "sigmoid") == "sigmoid":
             p["g.weight"] = ParamDecl((H * V, d))
+        if o.get("sink"):
+            p["sink"] = ParamDecl((H,))
         return p
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -95,23 +112,28 @@ class LatentAttention(Part):
         order = self.position.head_order(Rr) if Rr and hasattr(self.position, "head_order") else None
         order = list(order) if order is not None else list(range(Rr))
         dkv = tensors["dkv.weight"]
-        if Rr:
+        wq = tensors["uq.weight"] if self.q_rank is not None else tensors["q.weight"]
+        if order != list(range(Rr)):
             # the rotated rows in the order that makes the encoding's pairs the halves the kernel turns
-            idx = torch.tensor(list(range(R)) + [R + i for i in order], dtype=torch.long, device=dkv.device)
-            dkv = dkv.index_select(0, idx)
-        ws = ([tensors["dq.weight"]] if self.q_rank is not None else []) + [dkv]
+            dkv = dkv.index_select(0, torch.tensor(list(range(R)) + [R + i for i in order], dtype=torch.long, device=dkv.device))
+            head = torch.tensor(list(range(D)) + [D + i for i in order], dtype=torch.long, device=wq.device)
+            wq = wq.view(H, D + Rr, -1).index_select(1, head).reshape(H * (D + Rr), -1)
+        ws = [tensors["dq.weight"] if self.q_rank is not None else wq, dkv]
         ws += [tensors["g.weight"]] if self.gate else []
         wide = torch.float32 if any(w.dtype == torch.float32 for w in ws) else ws[0].dtype
         self.down = Linear(torch.cat([w.to(wide) for w in ws], dim=0))
-        self.uq = Linear(tensors["uq.weight"] if self.q_rank is not None else tensors["q.weight"])
+        self.uq = Linear(wq) if self.q_rank is not None else None
         self.o = Linear(tensors["o.weight"])
         if self.q_norm is not None:
             self.q_norm.bind({"weight": tensors["dq_norm.weight"]})
-        self.kv_norm.bind({"weight": tensors["dkv_norm.weight"]})
+        self.kv_norm_w = tensors["dkv_norm.weight"].float().contiguous()
+        if self.has_sink:
+            self.sinks = tensors["sink"].float().contiguous()
+        self.takes_normed_input = self.down.takes_normed()
         uk = tensors["uk.weight"].view(H, D, R)
         into = uk.new_zeros(H, K, D + Rr)                    # row r of a head: what element r of q' is made of
-        for r, src in enumerate(order):
-            into[:, r, D + src] = 1.0                        # the rotated part moves to the front, exactly
+        for r in range(Rr):
+            into[:, r, D + r] = 1.0                          # the rotated part moves to the front, exactly
         into[:, Rr:Rr + R, :D] = uk.transpose(1, 2)
         uv = tensors["uv.weight"].view(H, V, R)
         out_of = uv.new_zeros(H, V, K)
@@ -121,7 +143,8 @@ class LatentAttention(Part):
 
     def kernel_libraries(self) -> Tuple[str, ...]:
         libs = ("elementwise", "block_linear", "attention")
-        libs += kernels.fast_attention_libraries(self.dtype, self.kept, min(self.n_heads, self.HEADS_AT_ONCE), 1)
+        libs += kernels.fast_attention_libraries(self.dtype, self.kept, min(self.n_heads, self.HEADS_AT_ONCE), 1,
+                                                 sinks=self.has_sink)
         for lin in (self.down, self.uq, self.o):
             if lin is not None:
                 libs += lin.libraries(self.dtype)
@@ -133,32 +156,33 @@ class LatentAttention(Part):
     def state_needs(self) -> Optional[StateNeed]:
         return None
 
-    def forward(self, step, io: LayerIO, h: torch.Tensor, residual: torch.Tensor, accumulate: bool = True):
+    fuses_next_norm = True
+
+    def forward(self, step, io: LayerIO, h, residual: torch.Tensor, accumulate: bool = True, next_norm=None):
+        """``h``: the normalised rows or a half-done norm (:class:`NormedInput`).  With ``next_norm`` the output projection
+        may do the first half of that norm; the result is then its :class:`NormedInput`."""
         T = residual.shape[0]
         H, D, V, Rn, Rr, K = self.n_heads, self.dim, self.value_dim, self.kv_rank, self.rot_dim, self.kept
-        Rq = self.q_rank or 0
-        proj = step.ws.buf("lat_proj", (T, Rq + Rn + Rr + (H * V if self.gate else 0)), torch.float32)
+        first = self.q_rank if self.q_rank is not None else H * (D + Rr)
+        proj = step.ws.buf("lat_proj", (T, first + Rn + Rr + (H * V if self.gate else 0)), torch.float32)
         self.down(h, proj)
-        q = step.ws.buf("lat_q", (T, H * (D + Rr)), self.dtype)
         if self.q_norm is not None:
-            cq = step.ws.buf("lat_cq", (T, Rq), self.dtype)
-            self.q_norm.forward_rows(proj[:, :Rq], cq)
+            cq = step.ws.buf("lat_cq", (T, first), self.dtype)
+            self.q_norm.forward_rows(proj[:, :first], cq)
+            q = step.ws.buf("lat_q", (T, H * (D + Rr)), self.dtype)
             self.uq(cq, q)
+            turned = q
         else:
-            self.uq(h, q)
-        # a row of ``qc``: the H queries in the latent's space, then the token's key/value head: [rotated | latent]
-        qc = step.ws.buf("lat_qc", (T, (H + 1) * K), self.dtype)
-        self.kv_norm.forward_rows(proj[:, Rq:Rq + Rn], qc[:, H * K + Rr:H * K + Rr + Rn])
-        if Rr:
-            kernels.convert_rows(proj[:, Rq + Rn:Rq + Rn + Rr], qc[:, H * K:H * K + Rr])
-        if K != Rr + Rn:
-            qc[:, H * K + Rr + Rn:].zero_()
-        kernels.block_linear(q, self.uk_t, qc[:, :H * K])
+            q = proj[:, :first]
+            turned = q if self.dtype == torch.float32 else step.ws.buf("lat_q", (T, first), self.dtype)
         table = self.position.rotary_table()
-        kernels.rope_store(qc, H, 1, K, Rr, table[0] if table is not None else None, step.positions, step.seq_of_token,
-                           io.block_table, io.k_pages, None, io.page_size, keys_only=True)
+        kernels.latent_prep(proj, first, Rn, first + Rn, Rr, self.kv_norm_w, self.norm_eps, q, turned, H,
+                            table[0] if table is not None else None, step.positions, step.seq_of_token, io.block_table,
+                            io.k_pages, io.page_size)
+        qc = step.ws.buf("lat_qc", (T, H * K), self.dtype)      # the H queries in the latent's space
+        kernels.block_linear(turned, self.uk_t, qc)
         heads = step.ws.buf("lat_heads", (T, H * V), self.dtype)
-        gate = proj[:, Rq + Rn + Rr:] if self.gate else None
+        gate = proj[:, first + Rn + Rr:] if self.gate else None
         # all heads read the one key/value head; the tensor-core kernels take up to 16 query heads a key/value head,
         # so more heads go through them 16 at a time (the queries are a column slice of the rows, the latent pages
         # are the same)
@@ -167,14 +191,17 @@ class LatentAttention(Part):
         for h0 in range(0, H, n):
             h1 = min(H, h0 + n)
             mixed = step.ws.buf("lat_mixed", (T, (h1 - h0) * K), self.dtype)
-            kernels.attention(step, qc[:, h0 * K:h1 * K], mixed, h1 - h0, 1, K, self.scale, self.window, io)
+            kernels.attention(step, qc[:, h0 * K:h1 * K], mixed, h1 - h0, 1, K, self.scale, self.window, io,
+                              sinks=self.sinks[h0:h1] if self.has_sink else None)
             if self.gate:
                 kernels.block_linear(mixed, self.uv[h0:h1], heads[:, h0 * V:h1 * V], epilogue="sigmoid_gate",
                                      gate=gate[:, h0 * V:h1 * V])
             else:
                 kernels.block_linear(mixed, self.uv[h0:h1], heads[:, h0 * V:h1 * V])
-        self.o(heads, residual, accumulate=accumulate)
-        return None
+        if not accumulate:
+            self.o(heads, residual)
+            return None
+        return self.o.accumulate_with_norm(step, heads, residual, next_norm, "attn_next")
 
     HEADS_AT_ONCE = 16
 

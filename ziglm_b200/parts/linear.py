@@ -32,6 +32,10 @@ class Linear:
             return ("gemm_generic",) + kernels.fast_gemm_libraries()
         return ("gemm_generic",)
 
+    def takes_normed(self) -> bool:
+        """Whether this product can complete a norm that the product before it has begun (:class:`NormedInput`)."""
+        return (self.weight.dtype == torch.bfloat16 and self.in_features % 8 == 0 and self.weight.data_ptr() % 16 == 0)
+
     def __call__(self, x, out: torch.Tensor, accumulate: bool = False) -> torch.Tensor:
         """``x``: the input rows, or a :class:`NormedInput` whose norm this product completes."""
         if isinstance(x, NormedInput):

@@ -63,6 +63,7 @@ class GatedMLP(Part):
         else:
             self.gate_up = Linear(torch.cat([g.to(wide), u.to(wide)], dim=0), bias)
         self.down = Linear(tensors["down.weight"], tensors["down.bias"] if self.spec.bias else None)
+        self.takes_normed_input = self.gate_up.takes_normed()
 
     def kernel_libraries(self) -> Tuple[str, ...]:
         libs = ("elementwise",)
