@@ -13,6 +13,7 @@
     python bench.py --case vilazen [--shape 1b|8b] [--layers L]    the Vilazen design beside Llama at equal width, its kernels alone
     python bench.py --case lipadra [--shape 1b|8b] [--layers L]    the Lipadra design beside Tumatar and Llama at equal width, its kernels alone
     python bench.py --case mopilorn [--shape 1b|8b] [--layers L]   the Mopilorn design beside Vilazen and Llama at equal width, its kernels alone
+    python bench.py --case lilulix [--shape 1b|8b] [--layers L]    the Lilulix design beside Vilazen and Llama at equal width, its kernels alone
 
 A "step" is one decode step of a batch of 8 sequences at a context of 4096
 tokens.  ``value`` is decoded tokens a second, timed on the device with CUDA
@@ -1233,6 +1234,178 @@ def run_mopilorn(args):
     return 0
 
 
+def run_lilulix(args):
+    """The Lilulix design beside the Vilazen design (the library's closest: a shared norm, latent attention, attention with
+    sinks) and the Llama shape, all of the same width and with random weights: a prompt of ``--prompt-tokens`` and decode
+    steps of ``--batch`` sequences at ``--context``, ``--layers`` layer runs of each (default 4; of Lilulix half as many
+    layers, passed through twice), and every kernel the design adds or changes, alone, against its own roofline (the larger
+    of bytes / measured copy bandwidth and FLOPs / measured bf16 peak), each beside the library's like kernel timed in the
+    same run on operands of the same size."""
+    import torch
+    from types import SimpleNamespace
+    from ziglm_b200 import kernels
+    from ziglm_b200.config.shapes import shape
+    from ziglm_b200.engine.workspace import Workspace
+    from ziglm_b200.parts.base import LayerIO
+    torch.cuda.set_device(0)
+    pk = peaks()
+    size = "8b" if args.shape == "8b" else "1b"
+    layers = args.layers or 4
+    T, batch, context = args.prompt_tokens, args.batch, args.context
+    max_seq = max(context, T) + 64
+    gen = torch.Generator().manual_seed(7)
+    out = {"case": "lilulix", "width_of": "llama-" + size, "dtype": "bf16", "layer_runs": layers, "prompt_tokens": T,
+           "batch": batch, "context": context, "data": "synthetic", "l2": "a 256 MiB buffer is rewritten before every timed call",
+           "peaks": pk["source"], "models": {}}
+    with ClockSampler() as clocks:
+        for name in ("lilulix-" + size, "vilazen-" + size, "llama-" + size):
+            cfg = shape(name)
+            if name.startswith("lilulix"):
+                half = max(1, layers // 2)
+                cfg["layers"], cfg["loop"] = cfg["layers"][:half], {"start": 0, "stop": half, "times": 2}
+                vocab = cfg["vocab"]
+            elif "layers" in cfg:
+                cfg["layers"] = cfg["layers"][:layers]
+                vocab = cfg["vocab"]
+            else:
+                cfg["num_hidden_layers"] = layers
+                cfg["max_position_embeddings"] = max(cfg["max_position_embeddings"], max_seq)
+                vocab = cfg["vocab_size"]
+            eng = _engine_for(cfg, "bfloat16", batch, max_seq)
+            ids = lambda n: torch.randint(0, vocab, (n,), generator=gen).tolist()
+            pre = _time_prompt(eng, ids(T), args.warmup, args.steps)
+            slots = [eng.alloc_slot() for _ in range(batch)]
+            eng.step([(s, ids(3)) for s in slots])
+            for _ in range(2):
+                eng.step([(s, [1]) for s in slots])
+            eng.graph_launched_kernels()
+            eng.step([(s, [1]) for s in slots])
+            launches = eng.graph_launched_kernels()
+            for s in slots:
+                eng.free_slot(s)
+            dec = _time_decode_at(eng, batch, context, args.warmup, args.steps, ids)
+            out["models"][name] = {"prefill_ms": round(pre, 3), "prefill_tok_s": round(T / pre * 1e3, 1),
+                                   "decode_ms": round(dec, 4), "decode_tok_s": round(batch / dec * 1e3, 1),
+                                   "launches_per_decode_step": launches}
+            del eng
+            torch.cuda.empty_cache()
+    out["clocks"] = clocks.summary()
+    # ---- the kernels, alone
+    cfg = shape("lilulix-" + size)
+    d, buckets = cfg["width"], cfg["embedding"]["bigram"]["buckets"]
+    lat, att, ff = cfg["layers"][0]["mixer"], cfg["layers"][1]["mixer"], cfg["layers"][0]["mlp"]["ff"]
+    H, G, hd, scale = att["heads"], att["kv_heads"], att["dim"], att["scale"]
+    LH, LD, LR, LC, LV = lat["heads"], lat["dim"], lat["rot_dim"], lat["kv_rank"], lat["vdim"]
+    dev = torch.device("cuda:0")
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=dev)
+    bf = lambda *sh: (torch.randn(*sh, device=dev) * 0.05).to(torch.bfloat16)
+    f32 = lambda *sh: torch.randn(*sh, device=dev) * 0.05
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    hbm, peak = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    rows = []
+
+    def report(what, like, ms, nbytes, flops):
+        floor = max(nbytes / hbm, flops / peak) * 1e3
+        rows.append({"kernel": what, "like": like, "ms": round(ms, 4), "roofline_ms": round(floor, 4),
+                     "frac_of_roofline": round(floor / ms, 4)})
+
+    def timed(fn):
+        return _timed(fn, args.warmup, args.steps, flush)
+
+    kernels.require(("elementwise", "attention", "attention_tc", "attention_fmha", "block_linear", "gemm_generic", "gemm_tc"))
+    page = 64
+    inv_freq = torch.rand(hd // 2, device=dev)
+    lat_freq = torch.rand(LR // 2, device=dev)
+    zero, slopes = torch.zeros(H, device=dev), torch.tensor([2.0 ** (-8.0 * (h + 1) / H) for h in range(H)], device=dev)
+    table, pairs_table = bf(cfg["vocab"], d), bf(buckets + 1, d)
+    for n_tok, tag in ((T, f"prompt of {T}"), (batch, f"decode batch {batch}")):
+        decode = n_tok != T
+        past = context - 1 if decode else 0
+        n_seq = n_tok if decode else 1
+        per_seq = -(-(past + (1 if decode else T)) // page)
+        k_pages, v_pages = bf(n_seq * per_seq, G, page, hd), bf(n_seq * per_seq, G, page, hd)
+        blocks = torch.arange(n_seq * per_seq, dtype=torch.int32, device=dev).view(n_seq, per_seq)
+        new = [1] * n_seq if decode else [T]
+        cu = [0]
+        for n in new:
+            cu.append(cu[-1] + n)
+        step = SimpleNamespace(
+            n_tokens=n_tok, n_seqs=n_seq, single_token=decode, max_new=max(new), max_total=past + max(new),
+            tokens=torch.randint(0, cfg["vocab"], (n_tok,), dtype=torch.int32, device=dev),
+            positions=i32([past + i for n in new for i in range(n)]), seq_of_token=i32([b for b, n in enumerate(new) for _ in range(n)]),
+            cu_seqlens=i32(cu), past_lens=i32([past] * n_seq), total_lens=i32([past + n for n in new]),
+            slots=i32(list(range(n_seq))), ws=Workspace(dev))
+        io = LayerIO(k_pages=k_pages, v_pages=v_pages, block_table=blocks, page_size=page)
+        # the embedding, and what a pass begins with
+        x, kept, last = f32(n_tok, d), f32(n_tok, d), torch.zeros(n_seq, 1, dtype=torch.int32, device=dev)
+        ms = timed(lambda: kernels.embed(table, step.tokens, x))
+        report(f"embed, {tag}", "-", ms, n_tok * d * 6, 0)
+        ms = timed(lambda: kernels.embed_pairs(table, pairs_table, last, 40503, 65599, step, x, kept))
+        report(f"embed_pairs with a copy kept, {tag}", "embed", ms, n_tok * d * 12, 0)
+        row = bf(d)
+        ms = timed(lambda: kernels.add_row(x, row))
+        report(f"add_row, {tag}", "-", ms, n_tok * d * 8, 0)
+        ms = timed(lambda: kernels.add_row(x, row, rows=kept))
+        report(f"add_row with the kept embedding, {tag}", "add_row", ms, n_tok * d * 12, 0)
+        # norm of heads with values that are the keys, beside the library's rotation + cache write
+        qkv, qk = bf(n_tok, (H + 2 * G) * hd), bf(n_tok, (H + G) * hd)
+        wq, wk = f32(hd) + 1, f32(hd) + 1
+        ms = timed(lambda: kernels.rope_store(qkv, H, G, hd, hd, inv_freq, step.positions, step.seq_of_token, blocks, k_pages,
+                                              v_pages, page))
+        report(f"rope_store (rotation + cache write), {tag}", "-", ms, n_tok * (H + G) * hd * 4 + n_tok * G * hd * 2 * 3, 0)
+        ms = timed(lambda: kernels.rope_norm_store(qk, H, G, hd, 0, None, 1.0, hd, 1e-6, step.positions, step.seq_of_token, blocks,
+                                                   k_pages, v_pages, page, norm_first=True, q_weight=wq, k_weight=wk,
+                                                   values_from_keys=True))
+        report(f"rope_norm_store (norm of heads + cache write, values from keys), {tag}", "rope_store", ms,
+               n_tok * (H + G) * hd * 4 + n_tok * G * hd * 2 * 2, 0)
+        # attention: every key, with sinks, with sinks and the bias
+        att_out = torch.empty(n_tok, H * hd, dtype=torch.bfloat16, device=dev)
+        if decode:
+            att_bytes, att_flops = n_seq * context * G * hd * 2 * 2 + n_tok * H * hd * 4, 4.0 * n_tok * H * hd * context
+        else:
+            att_bytes, att_flops = n_tok * (H + 2 * G) * hd * 2 + n_tok * H * hd * 2, 4.0 * H * hd * (T * (T + 1) // 2)
+        for sk, sl, what, like in ((None, None, "attention, every key", "-"),
+                                   (zero, None, "attention with sinks", "attention, every key"),
+                                   (zero, slopes, "attention with sinks and a distance bias", "attention, every key")):
+            ms = timed(lambda: kernels.attention(step, qkv, att_out, H, G, hd, scale, None, io, sinks=sk, slopes=sl))
+            report(f"{what}, {tag}", like, ms, att_bytes, att_flops)
+        del k_pages, v_pages
+        # the latent's preparation and its attention over one shared head
+        K = LC + LR
+        lat_pages = bf(n_seq * per_seq, 1, page, K)
+        lio = LayerIO(k_pages=lat_pages, v_pages=lat_pages, block_table=blocks, page_size=page)
+        first = LH * (LD + LR)
+        proj, turned = f32(n_tok, first + LC + LR + LH * LV), bf(n_tok, first)
+        wl = f32(LC) + 1
+        ms = timed(lambda: kernels.latent_prep(proj, first, LC, first + LC, LR, wl, 1e-6, proj[:, :first], turned, LH, lat_freq,
+                                               step.positions, step.seq_of_token, blocks, lat_pages, page))
+        report(f"latent_prep (latent norm + rotations + cache write), {tag}", "rope_store", ms,
+               n_tok * (first * 6 + K * 6), 0)
+        qc, mixed = bf(n_tok, LH * K), torch.empty(n_tok, min(LH, 16) * K, dtype=torch.bfloat16, device=dev)
+        n = min(LH, 16)
+        lsinks = f32(n) * 20
+        if decode:
+            lb, lf = n_seq * context * K * 2 + n_tok * n * K * 4, 4.0 * n_tok * n * K * context
+        else:
+            lb, lf = n_tok * (n + 1) * K * 2 + n_tok * n * K * 2, 4.0 * n * K * (T * (T + 1) // 2)
+        for sk, what, like in ((None, "attention over one shared latent head", "-"),
+                               (lsinks, "attention over one shared latent head with learned sinks", "the same without")):
+            ms = timed(lambda: kernels.attention(step, qc[:, :n * K], mixed, n, 1, K, 128 ** -0.5, None, lio, sinks=sk))
+            report(f"{what} ({n} query heads), {tag}", like, ms, lb, lf)
+        del lat_pages
+        # the feed-forward's first product with the tanh form of gelu
+        h, wg, act = bf(n_tok, d), bf(2 * ff, d), torch.empty(n_tok, ff, dtype=torch.bfloat16, device=dev)
+        gb, gf = n_tok * d * 2 + 2 * ff * d * 2 + n_tok * ff * 2, 4.0 * n_tok * d * ff
+        ms = timed(lambda: kernels.gemm_tc(h, wg, act, glu="silu"))
+        report(f"gemm_tc gated silu, {tag}", "-", ms, gb, gf)
+        ms = timed(lambda: kernels.gemm_tc(h, wg, act, glu="gelu_tanh"))
+        report(f"gemm_tc gated tanh gelu, {tag}", "gemm_tc gated silu", ms, gb, gf)
+    out["kernels"] = rows
+    out["wait_errors"] = wait_errors(kernels)
+    print(json.dumps(out))
+    return 0
+
+
 def run_workload(args):
     """The two workloads beside the headline one, through ``Engine.generate`` (host token ids in, ids out):
 
@@ -1452,14 +1625,14 @@ def main():
                     help="run fewer layers than the configuration has (both numbers are reported)")
     ap.add_argument("--case", default="full",
                     choices=["full", "prefill", "decode", "workload-1b", "workload-13b", "float32", "reference-kernels",
-                             "tumatar", "tikalix", "vilazen", "lipadra", "mopilorn"],
+                             "tumatar", "tikalix", "vilazen", "lipadra", "mopilorn", "lilulix"],
                     help="full: the whole measurement; prefill / decode: that phase alone (for profilers and sweeps); "
                          "workload-1b / workload-13b: the two other workloads through Engine.generate; float32: the "
                          "8B shape in true 32-bit; reference-kernels: the reference's CUDA kernels alone, if built; tumatar: the "
                          "Tumatar design beside the Llama shape of the same width (--shape 1b or 8b), and its kernels alone; tikalix: "
                          "the same for the Tikalix design; vilazen: the same for the Vilazen design; lipadra: the Lipadra design "
                          "beside the Tumatar design and the Llama shape of the same width, and its kernels alone; mopilorn: the "
-                         "Mopilorn design beside the Vilazen design and the Llama shape likewise")
+                         "Mopilorn design beside the Vilazen design and the Llama shape likewise; lilulix: the same for the Lilulix design")
     ap.add_argument("--shape", default="8b", choices=sorted(SHAPES), help="--case prefill/decode: layer sizes")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="--case prefill/decode")
     ap.add_argument("--repeats", type=int, default=2, help="workload cases: timed repetitions after one warm-up")
@@ -1491,6 +1664,8 @@ def main():
         return run_lipadra(args)
     if args.case == "mopilorn":
         return run_mopilorn(args)
+    if args.case == "lilulix":
+        return run_lilulix(args)
     if args.case != "full":
         return run_case(args)
     return run_ours(args)

@@ -46,6 +46,10 @@ LAYER_TYPES = ("latent_attention", "attention")
 # Constants the design fixes.
 BIAS_EXPONENT = 8.0         # attention: head h of H loses 2^(-BIAS_EXPONENT (h + 1) / H) of its score a position
 
+# A choice of this library, not of the design: how much larger than it is a cached latent may be kept in bfloat16 if
+# that lets the tensor-core attention kernels take it.
+PAD_LATENT = 4.0 / 3.0
+
 
 @dataclass(frozen=True)
 class LilulixConfig:
@@ -160,7 +164,8 @@ class LilulixConfig:
                              scale=float(m["scale"]),
                              position=PositionSpec(kind="rope", rotary_dim=m["rot_dim"], theta=float(m["rot"]["base"])),
                              options={"value_dim": m["vdim"], "kv_rank": m["kv_rank"], "q_rank": None,
-                                      "rot_dim": m["rot_dim"], "gate": "sigmoid", "sink": True, "norm_eps": eps})
+                                      "rot_dim": m["rot_dim"], "gate": "sigmoid", "sink": True, "norm_eps": eps,
+                                      "pad_to_fast": PAD_LATENT})
         for p in ("q", "k", "o"):
             names[f"mixer.{p}.weight"] = f"mix.{p}"
         for p in ("q", "k"):

@@ -171,6 +171,25 @@ SHAPES["mopilorn-1b"] = _mopilorn(2048, 128256, 8, 32, 8, 64, 8192)
 SHAPES["mopilorn-8b"] = _mopilorn(4096, 128256, 16, 32, 8, 128, 14336)
 
 
+def _lilulix(width: int, vocab: int, pairs: int, heads: int, kv_heads: int, dim: int, ff: int) -> Dict[str, Any]:
+    """A Lilulix stack of ``pairs`` times (latent attention, biased attention over its own keys), the first pair passed
+    through twice, with the attention heads of the Llama shape of that width, a key/value latent of 96 beside 32 rotated
+    dimensions (what the tensor-core attention takes) and a table of as many token pairs as the vocabulary has tokens."""
+    lat = {"heads": width // 128, "dim": 96, "rot_dim": 32, "vdim": 128, "kv_rank": 96, "scale": 128 ** -0.5,
+           "rot": {"dims": 32, "base": 500000.0}}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+    mlp = {"kind": "dense", "ff": ff}
+    two = ({"type": "latent_attention", "mixer": lat, "mlp": mlp}, {"type": "attention", "mixer": att, "mlp": mlp})
+    return {"architecture": "Lilulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": vocab, "mul_prev": 40503, "mul_cur": 65599}},
+            "loop": {"start": 0, "stop": 2, "times": 2},
+            "layers": [copy.deepcopy(x) for _ in range(pairs) for x in two]}
+
+
+SHAPES["lilulix-1b"] = _lilulix(2048, 128256, 7, 32, 8, 64, 8192)
+SHAPES["lilulix-8b"] = _lilulix(4096, 128256, 15, 32, 8, 128, 14336)
+
+
 def shape(name: str) -> Dict[str, Any]:
     """A copy of the named config.json dictionary."""
     try:

@@ -210,7 +210,8 @@ struct AtcCommon {
     int keep_first;      // the split decode kernel only: with a window, the first positions that stay visible behind it
     const int* block_table;
     int bt_stride;
-    const float* slopes; // the split decode kernel only: by how much a head's score is made less per position, or null
+    const float* slopes; // the decode kernels only: by how much a head's score is made less per position, or null
+    const float* sinks;  // the flat decode kernel only: one number a head in the softmax's denominator, or null
     int* err;
     // the flat decode kernel only: out[t, h, d] is multiplied by sigmoid(gate[t * gate_stride + h * hd + d]) before it
     // is rounded (a gate on the heads' outputs); null: none
@@ -396,6 +397,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
 // sinks (float, one per head, or null): exp(sinks[h]) joins the denominator of head h.
 // head_gate (or null): head h of token t is multiplied by sigmoid(head_gate[t * gate_stride + h]) * gate_mult
 // before it is rounded.
+constexpr int MERGE_SPLITS = 256;       // splits whose weights the merge keeps in shared memory
 template <int HD>
 __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                   __nv_bfloat16* __restrict__ out, int n_splits, const float* __restrict__ sinks = nullptr,
@@ -409,6 +411,37 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
     if (head_gate != nullptr) {
         const float g = __bfloat162float(head_gate[(row / n_heads) * gate_stride + row % n_heads]);
         factor = (1.0f / (1.0f + expf(-g))) * gate_mult;
+    }
+    if (n_splits <= MERGE_SPLITS) {
+        // the splits' weights once for the block, side by side, then a column of sums a thread with eight loads in flight
+        __shared__ float w_s[MERGE_SPLITS];
+        __shared__ float scratch[33];
+        const float2* ml = reinterpret_cast<const float2*>(part_ml) + row * n_splits;
+        float big = sink;
+        for (int s = threadIdx.x; s < n_splits; s += blockDim.x) big = fmaxf(big, ml[s].x);
+        big = block_max(big, scratch);
+        float den = 0.f;
+        for (int s = threadIdx.x; s < n_splits; s += blockDim.x) {
+            const float2 v = ml[s];
+            const float wgt = v.x == -INFINITY ? 0.f : exp2f(v.x - big);
+            w_s[s] = wgt;
+            den = fmaf(v.y, wgt, den);
+        }
+        den = block_sum(den, scratch);                       // its barriers also publish the weights
+        if (sinks != nullptr) den += exp2f(sink - big);
+        for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+            const float* po = part_o + row * n_splits * HD + d;
+            float acc = 0.f;
+            for (int s0 = 0; s0 < n_splits; s0 += 8) {
+                float v[8];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) v[u] = s0 + u < n_splits ? po[(long)(s0 + u) * HD] : 0.f;
+#pragma unroll
+                for (int u = 0; u < 8; ++u) acc = fmaf(v[u], s0 + u < n_splits ? w_s[s0 + u] : 0.f, acc);
+            }
+            out[row * HD + d] = __float2bfloat16_rn((acc / den) * factor);
+        }
+        return;
     }
     float big = sink;
     for (int s = 0; s < n_splits; ++s) big = fmaxf(big, part_ml[(row * n_splits + s) * 2]);
@@ -492,7 +525,43 @@ struct FlatRope {
     const float* inv_freq;     // [rot / 2]
     __nv_bfloat16* k_pages;
     __nv_bfloat16* v_pages;
+    // instead of a rotation, an RMS norm of every query head and of the new key over its first norm_dim elements
+    // (0: none) with weights that all heads of a kind share (float [HD], zero behind norm_dim)
+    int norm_dim;
+    float norm_eps;
+    const float* q_w;
+    const float* k_w;
+    int values_from_keys;      // the rows are [q heads | k heads]; the new value is the key before its norm
 };
+
+// Norm the fragments of 16 query rows in registers: a row's elements lie in the four threads of its quad.
+template <int HD>
+__device__ __forceinline__ void norm_q_frags(uint32_t (&qf)[HD / 16][4], const float* __restrict__ w, int norm_dim,
+                                             float eps, int tid4) {
+    float ss[2] = {0.f, 0.f};
+#pragma unroll
+    for (int ks = 0; ks < HD / 16; ++ks)
+#pragma unroll
+        for (int slot = 0; slot < 4; ++slot) {
+            const float2 x = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&qf[ks][slot]));
+            ss[slot & 1] = fmaf(x.x, x.x, fmaf(x.y, x.y, ss[slot & 1]));
+        }
+    float inv[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        ss[h] += __shfl_xor_sync(0xffffffffu, ss[h], 1);
+        ss[h] += __shfl_xor_sync(0xffffffffu, ss[h], 2);
+        inv[h] = 1.0f / sqrtf(ss[h] / (float)norm_dim + eps);
+    }
+#pragma unroll
+    for (int ks = 0; ks < HD / 16; ++ks)
+#pragma unroll
+        for (int slot = 0; slot < 4; ++slot) {
+            const float2 g = *reinterpret_cast<const float2*>(w + ks * 16 + 2 * tid4 + (slot >= 2 ? 8 : 0));
+            const float2 x = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&qf[ks][slot]));
+            qf[ks][slot] = pack_bf16((x.x * inv[slot & 1]) * g.x, (x.y * inv[slot & 1]) * g.y);
+        }
+}
 
 // Rotate the fragments of 16 query rows in registers: column c of a fragment pairs with c + rot/2,
 // which lies HP = rot/32 fragments further in the same thread and the same register.
@@ -524,7 +593,9 @@ __device__ __forceinline__ void rotate_q_frags(uint32_t (&qf)[HD / 16][4], const
     }
 }
 
-template <int HD>
+// MORE: the kernel also knows sinks, slopes and the norm of the heads (a form of its own, so that the plain one keeps its
+// registers).
+template <int HD, bool MORE>
 __global__ void __launch_bounds__(ATC_THREADS, 2)
 attn_decode_flat_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
                         AtcCommon a, FlatRope rope, const int* __restrict__ positions,
@@ -696,6 +767,21 @@ attn_decode_flat_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
                          tid4);
         if (half > 0) rotate_q_frags<HD>(qf, cs_s, sn_s, half, tid4);
         float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+        float slope2[2] = {0.f, 0.f};
+        if (MORE) {
+            if (rope.norm_dim > 0) norm_q_frags<HD>(qf, rope.q_w, rope.norm_dim, rope.norm_eps, tid4);
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const int r = gid + 8 * h;
+                if (r >= group) continue;
+                if (a.slopes != nullptr) slope2[h] = a.slopes[kvh * group + r] * 1.4426950408889634f;
+                if (a.sinks != nullptr && j == 0 && warp == 0) {
+                    // the number that belongs to no key counts once: where the item's first page is, in one warp
+                    m[h] = a.sinks[kvh * group + r] * 1.4426950408889634f;
+                    l[h] = tid4 == 0 ? 1.0f : 0.f;
+                }
+            }
+        }
         float o[HD / 8][4];
 #pragma unroll
         for (int n = 0; n < HD / 8; ++n)
@@ -712,7 +798,16 @@ attn_decode_flat_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
                 if (landed) {
                     const int r = pos % PAGE;
                     const __nv_bfloat16* knew = a.q + (long)t * a.q_row_stride + (long)(a.n_heads + kvh) * HD;
-                    const __nv_bfloat16* vnew = knew + (long)a.n_kv * HD;
+                    const __nv_bfloat16* vnew = (MORE && rope.values_from_keys) ? knew : knew + (long)a.n_kv * HD;
+                    float kinv = 1.0f;
+                    if (MORE && rope.norm_dim > 0) {
+                        float ss = 0.f;
+                        for (int d = lane; d < HD; d += 32) {
+                            const float x = __bfloat162float(knew[d]);
+                            ss = fmaf(x, x, ss);
+                        }
+                        kinv = 1.0f / sqrtf(warp_sum(ss) / (float)rope.norm_dim + rope.norm_eps);
+                    }
                     const long crow = ((long)a.block_table[(long)seq_of_token[t] * a.bt_stride + p] * a.n_kv + kvh) * PAGE + r;
                     __nv_bfloat16* kdst = rope.k_pages + crow * HD;
                     __nv_bfloat16* vdst = rope.v_pages + crow * HD;
@@ -724,6 +819,8 @@ attn_decode_flat_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
                             const int ii = d < half ? d : d - half;
                             const float x = __bfloat162float(knew[ii]), y = __bfloat162float(knew[ii + half]);
                             kv = __float2bfloat16_rn(d < half ? x * cs_s[ii] - y * sn_s[ii] : x * sn_s[ii] + y * cs_s[ii]);
+                        } else if (MORE && rope.norm_dim > 0) {
+                            kv = __float2bfloat16_rn((__bfloat162float(knew[d]) * kinv) * rope.k_w[d]);
                         } else {
                             kv = knew[d];
                         }
@@ -739,11 +836,11 @@ attn_decode_flat_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
             }
             if (!landed) break;
             if (p * PAGE >= start && p * PAGE + PAGE - 1 <= pos)
-                page_step<HD, 2, true>(qf, k0 + s * C::TILE_BYTES, v0 + s * C::TILE_BYTES, warp * 16, p * PAGE + warp * 16,
-                                       pos, pos, start, start, a.scale_log2, a.cap_in2, a.cap_log2, m, l, o, lane);
+                page_step<HD, 2, true, MORE>(qf, k0 + s * C::TILE_BYTES, v0 + s * C::TILE_BYTES, warp * 16, p * PAGE + warp * 16,
+                                       pos, pos, start, start, a.scale_log2, a.cap_in2, a.cap_log2, m, l, o, lane, slope2);
             else
-                page_step<HD, 2, false>(qf, k0 + s * C::TILE_BYTES, v0 + s * C::TILE_BYTES, warp * 16, p * PAGE + warp * 16,
-                                        pos, pos, start, start, a.scale_log2, a.cap_in2, a.cap_log2, m, l, o, lane);
+                page_step<HD, 2, false, MORE>(qf, k0 + s * C::TILE_BYTES, v0 + s * C::TILE_BYTES, warp * 16, p * PAGE + warp * 16,
+                                        pos, pos, start, start, a.scale_log2, a.cap_in2, a.cap_log2, m, l, o, lane, slope2);
             __syncwarp();
             if (lane == 0) mbar_arrive(empty0 + 8 * s);
         }
@@ -1121,6 +1218,7 @@ static int fill_common(AtcCommon* a, CUtensorMap* mk, CUtensorMap* mv, const voi
     a->block_table = block_table;
     a->bt_stride = bt_stride;
     a->slopes = nullptr;
+    a->sinks = nullptr;
     a->err = att_error_word();
     a->gate = nullptr;
     a->gate_stride = 0;
@@ -1188,9 +1286,12 @@ ZLM_EXPORT int zlm_attention_decode(const void* q, long q_row_stride, void* out,
 
 // Decode attention with the pages of the whole step divided evenly over one resident wave of blocks.
 //   n_blocks  0: two blocks (or what fits) per SM; else that many blocks
+//   norm_dim, norm_eps, q_w, k_w, values_from_keys   see FlatRope (norm_dim 0: no norm); a norm goes with rope_fused and
+//             without a rotation
+//   sinks, slopes   float [n_heads] or null, as zlm_attention_decode takes them
 //   scratch   floats for zlm_attention_decode_flat_scratch(...) of the same arguments
 namespace zlm {
-template <int HD>
+template <int HD, bool MORE>
 static int flat_blocks(int group, int T, int* smem_out) {
     const FlatSizes z = flat_sizes<HD>(group, T);
     if (smem_out) *smem_out = z.smem;
@@ -1201,11 +1302,11 @@ static int flat_blocks(int group, int T, int* smem_out) {
     if (max_dynamic == 0) {
         // the kernel's static shared memory counts against the same 227 KB
         cudaFuncAttributes fa;
-        if (cudaFuncGetAttributes(&fa, attn_decode_flat_kernel<HD>) != cudaSuccess) { cudaGetLastError(); return 0; }
+        if (cudaFuncGetAttributes(&fa, attn_decode_flat_kernel<HD, MORE>) != cudaSuccess) { cudaGetLastError(); return 0; }
         const int room = 227 * 1024 - (int)fa.sharedSizeBytes;
-        if (cudaFuncSetAttribute(attn_decode_flat_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, room) !=
+        if (cudaFuncSetAttribute(attn_decode_flat_kernel<HD, MORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, room) !=
                 cudaSuccess ||
-            cudaFuncSetAttribute(attn_decode_flat_kernel<HD>, cudaFuncAttributePreferredSharedMemoryCarveout,
+            cudaFuncSetAttribute(attn_decode_flat_kernel<HD, MORE>, cudaFuncAttributePreferredSharedMemoryCarveout,
                                  cudaSharedmemCarveoutMaxShared) != cudaSuccess) {
             cudaGetLastError();
             return 0;
@@ -1213,7 +1314,7 @@ static int flat_blocks(int group, int T, int* smem_out) {
         max_dynamic = room;
     }
     if (z.smem > max_dynamic) return 0;
-    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attn_decode_flat_kernel<HD>, ATC_THREADS, z.smem) !=
+    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attn_decode_flat_kernel<HD, MORE>, ATC_THREADS, z.smem) !=
         cudaSuccess) return 0;
     return sms * min(per_sm, 2);
 }
@@ -1221,8 +1322,8 @@ static int flat_blocks(int group, int T, int* smem_out) {
 
 ZLM_EXPORT int zlm_attention_decode_flat_blocks(int T, int n_heads, int n_kv, int hd) {
     if (T <= 0 || T > FLAT_MAX_TOKENS || n_heads <= 0 || n_kv <= 0 || n_heads % n_kv || n_heads / n_kv > 16) return 0;
-    if (hd == 128) return flat_blocks<128>(n_heads / n_kv, T, nullptr);
-    if (hd == 64) return flat_blocks<64>(n_heads / n_kv, T, nullptr);
+    if (hd == 128) return flat_blocks<128, false>(n_heads / n_kv, T, nullptr);
+    if (hd == 64) return flat_blocks<64, false>(n_heads / n_kv, T, nullptr);
     return 0;
 }
 
@@ -1240,16 +1341,28 @@ ZLM_EXPORT int zlm_attention_decode_flat(const void* q, long q_row_stride, void*
                                          const void* k_pages, const void* v_pages, long n_pages, int page_size,
                                          int n_blocks, int* counters, float* scratch, long scratch_floats,
                                          int rope_fused, int rope_store, int rot, const float* inv_freq,
+                                         int norm_dim, float norm_eps, const float* q_w, const float* k_w,
+                                         int values_from_keys, const float* sinks, const float* slopes,
                                          const void* gate, long gate_stride, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (T > FLAT_MAX_TOKENS) return ZLM_ERR_UNSUPPORTED;
     if (n_kv > 0 && n_heads / n_kv > 16) return ZLM_ERR_UNSUPPORTED;
+    if (norm_dim < 0 || norm_dim > hd || (norm_dim > 0 && (!q_w || !k_w || !rope_fused || rot > 0)) ||
+        (values_from_keys && !rope_fused))
+        return ZLM_ERR_UNSUPPORTED;
+    if (((uintptr_t)q_w % 8) || ((uintptr_t)k_w % 8)) return ZLM_ERR_UNSUPPORTED;
+    const bool more = norm_dim > 0 || values_from_keys || sinks != nullptr || slopes != nullptr;
     if (rope_fused && (rot < 0 || rot > hd || rot % 32 || (rot > 0 && !inv_freq))) return ZLM_ERR_UNSUPPORTED;
     FlatRope rope;
     rope.fused = rope_fused ? 1 : 0;
     rope.store = rope_fused && rope_store ? 1 : 0;
     rope.rot = rope_fused ? rot : 0;
     rope.inv_freq = inv_freq;
+    rope.norm_dim = norm_dim;
+    rope.norm_eps = norm_eps;
+    rope.q_w = q_w;
+    rope.k_w = k_w;
+    rope.values_from_keys = values_from_keys;
     rope.k_pages = (__nv_bfloat16*)const_cast<void*>(k_pages);
     rope.v_pages = (__nv_bfloat16*)const_cast<void*>(v_pages);
     AtcCommon a;
@@ -1259,20 +1372,20 @@ ZLM_EXPORT int zlm_attention_decode_flat(const void* q, long q_row_stride, void*
     if (rc) return rc;
     a.gate = (const __nv_bfloat16*)gate;          // bf16 [T, gate_stride]: the heads' outputs times its sigmoid
     a.gate_stride = gate_stride;
+    a.sinks = sinks;
+    a.slopes = slopes;
     const int group = n_heads / n_kv;
     int smem = 0;
-    const int resident = hd == 128 ? flat_blocks<128>(group, T, &smem) : flat_blocks<64>(group, T, &smem);
+    const int resident = more ? (hd == 128 ? flat_blocks<128, true>(group, T, &smem) : flat_blocks<64, true>(group, T, &smem))
+                              : (hd == 128 ? flat_blocks<128, false>(group, T, &smem) : flat_blocks<64, false>(group, T, &smem));
     if (resident <= 0) return ZLM_ERR_UNSUPPORTED;
     if (n_blocks <= 0) n_blocks = resident;
     if (!counters || !scratch || zlm_attention_decode_flat_scratch(T, n_heads, n_kv, hd, n_blocks) > scratch_floats)
         return ZLM_ERR_BAD_ARG;
-    cudaError_t e;
-    if (hd == 128)
-        e = launch_pdl(attn_decode_flat_kernel<128>, dim3(n_blocks), dim3(ATC_THREADS), (size_t)smem, stream, mk, mv, a,
-                       rope, positions, seq_of_token, T, counters, scratch, (__nv_bfloat16*)out);
-    else
-        e = launch_pdl(attn_decode_flat_kernel<64>, dim3(n_blocks), dim3(ATC_THREADS), (size_t)smem, stream, mk, mv, a,
-                       rope, positions, seq_of_token, T, counters, scratch, (__nv_bfloat16*)out);
+    auto* kern = more ? (hd == 128 ? attn_decode_flat_kernel<128, true> : attn_decode_flat_kernel<64, true>)
+                      : (hd == 128 ? attn_decode_flat_kernel<128, false> : attn_decode_flat_kernel<64, false>);
+    cudaError_t e = launch_pdl(kern, dim3(n_blocks), dim3(ATC_THREADS), (size_t)smem, stream, mk, mv, a, rope, positions,
+                               seq_of_token, T, counters, scratch, (__nv_bfloat16*)out);
     if (e != cudaSuccess) return (int)e;
     return launch_status();
 }
@@ -1418,6 +1531,7 @@ ZLM_EXPORT int zlm_attention_decode_noalloc(const void* q, long q_row_stride, vo
     a.block_table = block_table;
     a.bt_stride = bt_stride;
     a.slopes = nullptr;
+    a.sinks = nullptr;
     a.err = err;
     a.gate = nullptr;
     a.gate_stride = 0;

@@ -227,7 +227,6 @@ block_linear_rows_kernel(const TX* __restrict__ x, long x_stride, const TX* __re
                          const float* __restrict__ gate, long gate_stride) {
     constexpr int V = BlVec<TX>::N;
     pdl_launch_dependents();
-    pdl_wait();
     const int lane = threadIdx.x & 31;
     const long col = (long)blockIdx.x * SL_WARPS + (threadIdx.x >> 5);
     if (col >= (long)B * N) return;
@@ -235,9 +234,17 @@ block_linear_rows_kernel(const TX* __restrict__ x, long x_stride, const TX* __re
     const TX* wr = w + col * K;
     const TX* xb = x + (long)b * K;
     float acc[SL_ROWS] = {};
+    float w0[V];                                   // weights are older than the step: the first are requested before the wait
+    if (lane * V < K) bl_load16<TX>(wr + lane * V, w0);
+    pdl_wait();
     for (int k = lane * V; k < K; k += 32 * V) {
         float wv[V];
-        bl_load16<TX>(wr + k, wv);
+        if (k == lane * V) {
+#pragma unroll
+            for (int i = 0; i < V; ++i) wv[i] = w0[i];
+        } else {
+            bl_load16<TX>(wr + k, wv);
+        }
 #pragma unroll
         for (int t = 0; t < SL_ROWS; ++t) {
             if (t < T) {
@@ -248,13 +255,15 @@ block_linear_rows_kernel(const TX* __restrict__ x, long x_stride, const TX* __re
             }
         }
     }
+    float mine = 0.f;                              // lane t finishes row t
 #pragma unroll
     for (int t = 0; t < SL_ROWS; ++t) {
         if (t < T) {
             const float v = warp_sum(acc[t]);
-            if (lane == 0) bl_store<TO>(out, out_stride, t, col, v, bias, epi, gate, gate_stride);
+            if (lane == t) mine = v;
         }
     }
+    if (lane < T) bl_store<TO>(out, out_stride, lane, col, mine, bias, epi, gate, gate_stride);
 }
 
 }  // namespace zlm

@@ -635,49 +635,45 @@ __device__ __forceinline__ int pair_row(const PairHash& h, bool has_before, int 
     return (int)(((unsigned long long)before * h.mul_prev + (unsigned long long)token * h.mul_cur) % h.buckets);
 }
 
-// One block per sequence of the step: rows of all its tokens, then the state.
-__global__ void pair_rows_kernel(const int* __restrict__ tokens, const int* __restrict__ cu_seqlens,
-                                 const int* __restrict__ past_lens, const int* __restrict__ slots,
-                                 int* __restrict__ last, int* __restrict__ rows, PairHash h) {
+// The state behind a step of several tokens a sequence: launched behind the kernel that reads the old one.
+__global__ void pair_state_kernel(const int* __restrict__ tokens, const int* __restrict__ cu_seqlens,
+                                  const int* __restrict__ slots, int* __restrict__ last, int n_seqs) {
     pdl_launch_dependents();
     pdl_wait();
-    const int b = blockIdx.x;
-    const int begin = cu_seqlens[b], end = cu_seqlens[b + 1];
-    const bool goes_on = past_lens[b] > 0;
-    int* state = last + slots[b];
-    for (int t = begin + threadIdx.x; t < end; t += blockDim.x) {
-        const bool first = t == begin;
-        rows[t] = pair_row(h, !first || goes_on, first ? *state : tokens[t - 1], tokens[t]);
-    }
-    __syncthreads();                       // the state has been read
-    if (threadIdx.x == 0 && end > begin) *state = tokens[end - 1];
+    const int b = blockIdx.x * blockDim.x + threadIdx.x;
+    if (b < n_seqs && cu_seqlens[b + 1] > cu_seqlens[b]) last[slots[b]] = tokens[cu_seqlens[b + 1] - 1];
 }
 
-// One block per token: out = table[token] * scale + pairs[row], and a copy of it where `kept` is not null.  rows null:
-// a step of one token a sequence, token t being sequence t's; the row and the state are this block's own work.
+// One block per token: out = table[token] * scale + pairs[row], and a copy of it where `kept` is not null.
+// seq_of_token null: a step of one token a sequence, token t being sequence t's; the state is this block's own to replace.
 // VEC: d is a multiple of 4 and every pointer is aligned for it.
 template <typename TW, typename TB, bool VEC>
 __global__ void embed_pairs_kernel(const TW* __restrict__ table, const TB* __restrict__ pairs,
-                                   const int* __restrict__ tokens, const int* __restrict__ rows,
-                                   const int* __restrict__ past_lens, const int* __restrict__ slots,
-                                   int* __restrict__ last, PairHash h, float* __restrict__ out, float* __restrict__ kept,
-                                   int d, float scale) {
-    __shared__ int row_s;
+                                   const int* __restrict__ tokens, const int* __restrict__ seq_of_token,
+                                   const int* __restrict__ cu_seqlens, const int* __restrict__ past_lens,
+                                   const int* __restrict__ slots, int* __restrict__ last, PairHash h,
+                                   float* __restrict__ out, float* __restrict__ kept, int d, float scale) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
     const int token = tokens[t];
-    if (threadIdx.x == 0) {
-        if (rows != nullptr) row_s = rows[t];
-        else {
-            int* state = last + slots[t];
-            row_s = pair_row(h, past_lens[t] > 0, *state, token);
-            *state = token;
-        }
+    const int seq = seq_of_token != nullptr ? seq_of_token[t] : t;
+    const bool first = seq_of_token == nullptr || t == cu_seqlens[seq];
+    bool has_before = true;
+    int before = 0;
+    if (first) {
+        has_before = past_lens[seq] > 0;
+        before = last[slots[seq]];
+    } else {
+        before = tokens[t - 1];
     }
-    __syncthreads();
+    const int row = pair_row(h, has_before, before, token);
+    if (seq_of_token == nullptr) {
+        __syncthreads();                   // every thread has read the state
+        if (threadIdx.x == 0) last[slots[seq]] = token;
+    }
     const TW* a = table + (long)token * d;
-    const TB* b = pairs + (long)row_s * d;
+    const TB* b = pairs + (long)row * d;
     float* o = out + (long)t * d;
     float* k = kept != nullptr ? kept + (long)t * d : nullptr;
     if (VEC) {
@@ -1126,51 +1122,45 @@ ZLM_EXPORT int zlm_add_row(float* x, const float* rows, const void* table_row, i
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 
-// See embed_pairs_kernel and pair_rows_kernel.  last: int [slots], the last token of every sequence.  rows: int [T]
-// scratch that pair_rows fills; null for a step of one token a sequence (B == T), whose rows the one kernel makes.
-// kept: null, or float [T, d] that receives a copy of out.
-ZLM_EXPORT int zlm_pair_rows(const int* tokens, const int* cu_seqlens, const int* past_lens, const int* slots, int* last,
-                             int* rows, int B, long mul_prev, long mul_cur, long buckets, cudaStream_t stream) {
-    if (B <= 0) return 0;
-    if (mul_prev < 0 || mul_cur < 0 || buckets <= 0 || buckets > 0x7ffffffeL) return ZLM_ERR_BAD_ARG;
-    const PairHash h{(unsigned long long)mul_prev, (unsigned long long)mul_cur, (unsigned long long)buckets};
-    cudaError_t e = launch_pdl(pair_rows_kernel, dim3(B), dim3(256), 0, stream, tokens, cu_seqlens, past_lens, slots, last,
-                               rows, h);
-    return e == cudaSuccess ? launch_status() : (int)e;
-}
-
 namespace zlm {
 template <typename TW, typename TB>
-static cudaError_t launch_embed_pairs(const void* table, const void* pairs, const int* tokens, const int* rows,
-                                      const int* past_lens, const int* slots, int* last, PairHash h, float* out,
-                                      float* kept, int T, int d, float scale, cudaStream_t stream) {
+static cudaError_t launch_embed_pairs(const void* table, const void* pairs, const int* tokens, const int* seq_of_token,
+                                      const int* cu_seqlens, const int* past_lens, const int* slots, int* last,
+                                      PairHash h, float* out, float* kept, int T, int d, float scale,
+                                      cudaStream_t stream) {
     const bool vec = d % 4 == 0 && (((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)out | (uintptr_t)kept) % 16) == 0;
     const int threads = d >= 1024 ? 256 : (d >= 512 ? 128 : 64);
     return vec ? launch_pdl(embed_pairs_kernel<TW, TB, true>, dim3(T), dim3(threads), 0, stream, (const TW*)table,
-                            (const TB*)pairs, tokens, rows, past_lens, slots, last, h, out, kept, d, scale)
+                            (const TB*)pairs, tokens, seq_of_token, cu_seqlens, past_lens, slots, last, h, out, kept, d, scale)
                : launch_pdl(embed_pairs_kernel<TW, TB, false>, dim3(T), dim3(threads), 0, stream, (const TW*)table,
-                            (const TB*)pairs, tokens, rows, past_lens, slots, last, h, out, kept, d, scale);
+                            (const TB*)pairs, tokens, seq_of_token, cu_seqlens, past_lens, slots, last, h, out, kept, d, scale);
 }
 }  // namespace zlm
 
+// See embed_pairs_kernel.  last: int [slots], the last token of every sequence.  single != 0: a step of one token a
+// sequence (T == n_seqs), one launch; else the state is replaced by a second one.  kept: null, or float [T, d] that
+// receives a copy of out.
 ZLM_EXPORT int zlm_embed_pairs(const void* table, int table_dtype, const void* pairs, int pairs_dtype, const int* tokens,
-                               const int* rows, const int* past_lens, const int* slots, int* last, long mul_prev,
-                               long mul_cur, long buckets, float* out, float* kept, int T, int d, float scale,
-                               cudaStream_t stream) {
+                               const int* seq_of_token, const int* cu_seqlens, const int* past_lens, const int* slots,
+                               int* last, int n_seqs, int single, long mul_prev, long mul_cur, long buckets, float* out,
+                               float* kept, int T, int d, float scale, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (d <= 0 || mul_prev < 0 || mul_cur < 0 || buckets <= 0 || buckets > 0x7ffffffeL) return ZLM_ERR_BAD_ARG;
+    if (d <= 0 || n_seqs <= 0 || mul_prev < 0 || mul_cur < 0 || buckets <= 0 || buckets > 0x7ffffffeL || (single && T != n_seqs))
+        return ZLM_ERR_BAD_ARG;
     const PairHash h{(unsigned long long)mul_prev, (unsigned long long)mul_cur, (unsigned long long)buckets};
     const bool tf = table_dtype == ZLM_F32, pf = pairs_dtype == ZLM_F32;
     if ((!tf && table_dtype != ZLM_BF16) || (!pf && pairs_dtype != ZLM_BF16)) return ZLM_ERR_UNSUPPORTED;
+    const int* seq = single ? nullptr : seq_of_token;
     cudaError_t e;
-    if (tf && pf)
-        e = launch_embed_pairs<float, float>(table, pairs, tokens, rows, past_lens, slots, last, h, out, kept, T, d, scale, stream);
-    else if (tf)
-        e = launch_embed_pairs<float, __nv_bfloat16>(table, pairs, tokens, rows, past_lens, slots, last, h, out, kept, T, d, scale, stream);
-    else if (pf)
-        e = launch_embed_pairs<__nv_bfloat16, float>(table, pairs, tokens, rows, past_lens, slots, last, h, out, kept, T, d, scale, stream);
-    else
-        e = launch_embed_pairs<__nv_bfloat16, __nv_bfloat16>(table, pairs, tokens, rows, past_lens, slots, last, h, out, kept, T, d, scale, stream);
+#define ZLM_EP(TW, TB) e = launch_embed_pairs<TW, TB>(table, pairs, tokens, seq, cu_seqlens, past_lens, slots, last, h, out, kept, T, d, scale, stream)
+    if (tf && pf) ZLM_EP(float, float);
+    else if (tf) ZLM_EP(float, __nv_bfloat16);
+    else if (pf) ZLM_EP(__nv_bfloat16, float);
+    else ZLM_EP(__nv_bfloat16, __nv_bfloat16);
+#undef ZLM_EP
+    if (e == cudaSuccess && !single)
+        e = launch_pdl(pair_state_kernel, dim3((n_seqs + 127) / 128), dim3(128), 0, stream, tokens, cu_seqlens, slots, last,
+                       n_seqs);
     return e == cudaSuccess ? launch_status() : (int)e;
 }
 

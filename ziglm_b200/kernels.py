@@ -7,6 +7,7 @@ with a tensor that is not on a CUDA device is an error.
 """
 from __future__ import annotations
 
+import contextlib
 import ctypes
 from ctypes import c_float, c_int, c_long, c_void_p
 from typing import Optional, Tuple
@@ -64,9 +65,8 @@ _PROTOTYPES = {
         "zlm_unary_act": [c_void_p, c_void_p, c_int, c_long, c_int, c_void_p],
         "zlm_sigmoid_mul": [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_void_p],
         "zlm_add_row": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
-        "zlm_pair_rows": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_long, c_long, c_long, c_void_p],
-        "zlm_embed_pairs": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_long, c_long,
-                            c_long, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
+        "zlm_embed_pairs": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                            c_int, c_long, c_long, c_long, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
         "zlm_convert_rows": [c_void_p, c_int, c_long, c_void_p, c_int, c_long, c_int, c_int, c_void_p],
         "zlm_gate_heads": [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_float, c_void_p],
         "zlm_norm_gate": [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_float,
@@ -163,7 +163,8 @@ _PROTOTYPES = {
                                  c_void_p, c_void_p, c_void_p],
         "zlm_attention_decode_flat": [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p,
                                       c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int, c_int, c_void_p,
-                                      c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_void_p, c_long, c_void_p],
+                                      c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p,
+                                      c_int, c_void_p, c_void_p, c_void_p, c_long, c_void_p],
         "zlm_attention_decode_flat_blocks": [c_int, c_int, c_int, c_int],
         "zlm_attention_decode_flat_scratch": [c_int, c_int, c_int, c_int, c_int],
         "zlm_attention_prefill": [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int,
@@ -251,6 +252,26 @@ def _stream() -> int:
     if _raw_stream is not None and _current_device is not None:
         return _raw_stream(_current_device())
     return torch.cuda.current_stream().cuda_stream
+
+
+_side_streams = {}
+
+
+@contextlib.contextmanager
+def beside():
+    """Launches inside the block go to a second stream of the device, behind everything launched so far; the context's
+    value is called to make what is launched afterwards wait for them.  Inside a graph capture both become branches of
+    the graph."""
+    main = torch.cuda.current_stream()
+    side = _side_streams.get(main.device)
+    if side is None:
+        side = _side_streams[main.device] = torch.cuda.Stream(main.device)
+    fork, done = torch.cuda.Event(), torch.cuda.Event()
+    fork.record(main)
+    side.wait_event(fork)
+    with torch.cuda.stream(side):
+        yield lambda: main.wait_event(done)
+        done.record(side)
 
 
 def _cuda(t: torch.Tensor, name: str, dtype: Optional[torch.dtype] = None) -> None:
@@ -514,17 +535,15 @@ def embed_pairs(table: torch.Tensor, pairs: torch.Tensor, last: torch.Tensor, mu
         _cuda(kept, "kept", torch.float32)
         if kept.shape != out.shape:
             raise KernelError("embed_pairs: the copy must have the shape of the result")
-    buckets = pairs.shape[0] - 1
-    rows = None
-    if not (step.single_token and T == step.n_seqs):
-        rows = step.ws.buf("pair_rows", (T,), torch.int32)
-        _check(_fn("elementwise", "zlm_pair_rows")(
-            step.tokens.data_ptr(), step.cu_seqlens.data_ptr(), step.past_lens.data_ptr(), step.slots.data_ptr(),
-            last.data_ptr(), rows.data_ptr(), step.n_seqs, int(mul_prev), int(mul_cur), buckets, _stream()), "pair_rows")
+    single = bool(step.single_token and T == step.n_seqs)
     _check(_fn("elementwise", "zlm_embed_pairs")(
-        table.data_ptr(), code(table.dtype), pairs.data_ptr(), code(pairs.dtype), step.tokens.data_ptr(), _ptr(rows),
-        step.past_lens.data_ptr(), step.slots.data_ptr(), last.data_ptr(), int(mul_prev), int(mul_cur), buckets,
-        out.data_ptr(), _ptr(kept), T, d, float(scale), _stream()), "embed_pairs")
+        table.data_ptr(), code(table.dtype), pairs.data_ptr(), code(pairs.dtype), step.tokens.data_ptr(),
+        step.seq_of_token.data_ptr(), step.cu_seqlens.data_ptr(), step.past_lens.data_ptr(), step.slots.data_ptr(),
+        last.data_ptr(), step.n_seqs, int(single), int(mul_prev), int(mul_cur), pairs.shape[0] - 1, out.data_ptr(), _ptr(kept),
+        T, d, float(scale), _stream()), "embed_pairs")
+    if not single:
+        global _launches
+        _launches += 1          # the state is replaced by a second launch
 
 
 def scale_(x: torch.Tensor, factor: float) -> None:
@@ -1459,7 +1478,10 @@ def attention_decode_flat(qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_
                           block_table: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, page_size: int,
                           n_blocks: int, counters: torch.Tensor, scratch: torch.Tensor,
                           rope: Optional[Tuple[Optional[torch.Tensor], int, bool]] = None, softcap: float = 0.0,
-                          gate: Optional[torch.Tensor] = None) -> bool:
+                          gate: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
+                          slopes: Optional[torch.Tensor] = None,
+                          norm: Optional[Tuple[int, float, torch.Tensor, torch.Tensor]] = None,
+                          values_from_keys: bool = False) -> bool:
     """Tensor-core attention for steps of one token per sequence, with the pages of all sequences of the
     step divided evenly over ``n_blocks`` blocks (one resident wave), whatever the sequences' lengths.  One
     launch: the block that finishes a sequence's last piece merges the pieces.
@@ -1475,7 +1497,11 @@ def attention_decode_flat(qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_
     (rotated) and values go into the cache pages.  rotary_dim must be a multiple of 32.
 
     ``gate`` (bf16 [T, n_heads * head_dim], may be a column slice): the output is multiplied by its sigmoid before
-    it is rounded.
+    it is rounded.  ``sinks`` and ``slopes`` as :func:`attention_general` takes them.
+
+    ``norm`` = (norm_dim, eps, q weight, k weight) with ``rope`` = (None, 0, store): instead of a rotation every query head
+    and the new key are RMS-normed over their first norm_dim elements (weights float32 [head_dim], zero behind norm_dim).
+    ``values_from_keys``: the rows are [q heads | k heads] and the new value is the key before that norm.
     """
     _cuda(out, "out", torch.bfloat16); _cuda(k_pages, "k_pages", torch.bfloat16); _cuda(v_pages, "v_pages", torch.bfloat16)
     _cuda(positions, "positions", torch.int32); _cuda(seq_of_token, "seq_of_token", torch.int32)
@@ -1502,14 +1528,25 @@ def attention_decode_flat(qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_
             _cuda(inv_freq, "inv_freq", torch.float32)
             if inv_freq.numel() * 2 != rot:
                 raise KernelError("attention_decode_flat: the frequency table must hold rotary_dim/2 entries")
-        if qkv.shape[1] < (n_heads + (2 * n_kv if store else 0)) * head_dim:
+        if qkv.shape[1] < (n_heads + ((1 if values_from_keys else 2) * n_kv if store else 0)) * head_dim:
             raise KernelError("attention_decode_flat: the rows must hold the key and value heads to be stored")
+    norm_dim, norm_eps, q_w, k_w = 0, 0.0, None, None
+    if norm is not None:
+        norm_dim, norm_eps, q_w, k_w = norm
+        for w in (q_w, k_w):
+            _cuda(w, "norm weight", torch.float32)
+            if w.numel() != head_dim:
+                raise KernelError("attention_decode_flat: a norm weight holds one number for each element of a head")
+    if (norm is not None or values_from_keys) and rope is None:
+        raise KernelError("attention_decode_flat: the norm of the heads is part of the fused form")
     status = _fn("attention_tc", "zlm_attention_decode_flat")(
         qkv.data_ptr(), qkv.stride(0), out.data_ptr(), T, n_heads, n_kv, head_dim, scale, float(softcap or 0.0),
         int(window or 0),
         positions.data_ptr(), seq_of_token.data_ptr(), block_table.data_ptr(), block_table.stride(0),
         k_pages.data_ptr(), v_pages.data_ptr(), k_pages.shape[0], page_size, n_blocks, counters.data_ptr(),
-        scratch.data_ptr(), scratch.numel(), fused, int(bool(store)), int(rot), _ptr(inv_freq),
+        scratch.data_ptr(), scratch.numel(), fused, int(bool(store)), int(rot), _ptr(inv_freq), int(norm_dim),
+        float(norm_eps), _ptr(q_w), _ptr(k_w), int(bool(values_from_keys)), _head_numbers(sinks, n_heads, "sinks"),
+        _head_numbers(slopes, n_heads, "slopes"),
         *_gate_args(gate, T, n_heads * head_dim), _stream())
     if status == -2:
         return False
@@ -1604,24 +1641,37 @@ def decode_splits(n_tokens: int, n_kv: int, max_total: int, page_size: int = 64)
     return max(1, min(want, pages, 64))
 
 
-def attention_with_rope(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: int, head_dim: int,
-                        scale: float, window: Optional[int], io, inv_freq: Optional[torch.Tensor], rotary_dim: int,
-                        store: bool) -> bool:
-    """Decode steps on the tensor-core path: rotation, cache write and attention in one kernel.  False when
-    the step is not of that kind; the caller then runs ``rope_store`` and ``attention``."""
-    if not (step.single_token and _tc_attention_ok(qkv.dtype, n_heads, n_kv, head_dim, io.page_size)):
-        return False
-    if inv_freq is not None and rotary_dim % 32:
-        return False
+FLAT_PIECES = 8         # pieces of a (sequence, key/value head) that the flat decode kernel merges in one round of loads
+
+
+def _flat_room(step, n_heads: int, n_kv: int, head_dim: int):
+    """(blocks, counters, scratch) of the flat decode kernel for a step of one token a sequence; None: sizes it refuses."""
     n_blocks = attention_decode_flat_blocks(step.n_tokens, n_heads, n_kv, head_dim)
     if n_blocks <= 0:
-        return False
+        return None
     need = attention_decode_flat_scratch(step.n_tokens, n_heads, n_kv, head_dim, n_blocks)
-    scratch = step.ws.buf("attn_flat_scratch", (need,), torch.float32)
-    counters = step.ws.buf("attn_flat_counters", (step.n_tokens * n_kv,), torch.int32, zeros=True)
+    return (n_blocks, step.ws.buf("attn_flat_counters", (step.n_tokens * n_kv,), torch.int32, zeros=True),
+            step.ws.buf("attn_flat_scratch", (need,), torch.float32))
+
+
+def attention_with_rope(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: int, head_dim: int,
+                        scale: float, window: Optional[int], io, inv_freq: Optional[torch.Tensor], rotary_dim: int,
+                        store: bool, norm=None, values_from_keys: bool = False, sinks: Optional[torch.Tensor] = None,
+                        slopes: Optional[torch.Tensor] = None, softcap: float = 0.0) -> bool:
+    """Decode steps on the tensor-core path: rotation (or, without one, the ``norm`` of the heads that
+    :func:`attention_decode_flat` takes), cache write and attention in one kernel.  False when the step is not of that
+    kind; the caller then runs ``rope_store`` (or ``rope_norm_store``) and ``attention``."""
+    if not (step.single_token and _tc_attention_ok(qkv.dtype, n_heads, n_kv, head_dim, io.page_size)):
+        return False
+    if inv_freq is not None and (rotary_dim % 32 or norm is not None):
+        return False
+    room = _flat_room(step, n_heads, n_kv, head_dim)
+    if room is None:
+        return False
     return attention_decode_flat(qkv, out, n_heads, n_kv, head_dim, scale, window, step.positions, step.seq_of_token,
-                                 io.block_table, io.k_pages, io.v_pages, io.page_size, n_blocks, counters, scratch,
-                                 rope=(inv_freq, rotary_dim, store))
+                                 io.block_table, io.k_pages, io.v_pages, io.page_size, *room,
+                                 rope=(inv_freq, rotary_dim, store), norm=norm, values_from_keys=values_from_keys,
+                                 sinks=sinks, slopes=slopes, softcap=softcap)
 
 
 def attention(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, scale: float,
@@ -1652,10 +1702,19 @@ def attention(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: in
         keep_first = int(keep_first or 0) if window else 0
         span = min(step.max_total, window + keep_first) if window else step.max_total
     # kept first tokens, sinks and slopes: the tcgen05 prompt kernel and the decode kernel that splits a sequence's
-    # keys know them, the other tensor-core kernels do not
+    # keys know them; the flat decode kernel knows sinks and slopes, and is one launch instead of two (a gate a head
+    # rides on the other's second); the prompt kernel of few rows knows none
     plain_only = keep_first > 0 or sinks is not None or slopes is not None
     if plain_only and _tc_attention_ok(qkv.dtype, n_heads, n_kv, head_dim, io.page_size):
         if step.single_token:
+            room = _flat_room(step, n_heads, n_kv, head_dim) if keep_first == 0 and head_gate is None else None
+            # a block of the flat kernel merges a sequence's pieces alone: with many pieces (few sequences and key/value
+            # heads) the second kernel of the other, which merges rows side by side, is faster (43 against 50 us at eight
+            # sequences of 4,096 tokens on one key/value head)
+            if room is not None and step.n_tokens * n_kv * FLAT_PIECES >= room[0] and attention_decode_flat(
+                    qkv, out, n_heads, n_kv, head_dim, scale, window, step.positions, step.seq_of_token, io.block_table,
+                    io.k_pages, io.v_pages, io.page_size, *room, softcap=softcap, gate=gate, sinks=sinks, slopes=slopes):
+                return gate is not None
             n_splits = decode_splits(step.n_tokens, n_kv, span, io.page_size)
             part_o = step.ws.buf("attn_part_o", (step.n_tokens * n_heads * n_splits * head_dim,), torch.float32)
             part_ml = step.ws.buf("attn_part_ml", (step.n_tokens * n_heads * n_splits * 2,), torch.float32)
@@ -1670,15 +1729,11 @@ def attention(step, qkv: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: in
                 keep_first=keep_first, sinks=sinks, slopes=slopes):
             return False
     if not plain_only and _tc_attention_ok(qkv.dtype, n_heads, n_kv, head_dim, io.page_size):
-        n_blocks = attention_decode_flat_blocks(step.n_tokens, n_heads, n_kv, head_dim) if step.single_token else 0
-        if n_blocks > 0:
-            need = attention_decode_flat_scratch(step.n_tokens, n_heads, n_kv, head_dim, n_blocks)
-            scratch = step.ws.buf("attn_flat_scratch", (need,), torch.float32)
-            counters = step.ws.buf("attn_flat_counters", (step.n_tokens * n_kv,), torch.int32, zeros=True)
-            if attention_decode_flat(qkv, out, n_heads, n_kv, head_dim, scale, window, step.positions,
-                                     step.seq_of_token, io.block_table, io.k_pages, io.v_pages, io.page_size,
-                                     n_blocks, counters, scratch, softcap=softcap, gate=gate):
-                return gate is not None
+        room = _flat_room(step, n_heads, n_kv, head_dim) if step.single_token else None
+        if room is not None and attention_decode_flat(
+                qkv, out, n_heads, n_kv, head_dim, scale, window, step.positions, step.seq_of_token, io.block_table,
+                io.k_pages, io.v_pages, io.page_size, *room, softcap=softcap, gate=gate):
+            return gate is not None
         if step.single_token:
             n_splits = decode_splits(step.n_tokens, n_kv, span, io.page_size)
             part_o = step.ws.buf("attn_part_o", (step.n_tokens * n_heads * n_splits * head_dim,), torch.float32)

@@ -38,6 +38,12 @@ part may accept its input normalised that way:
                       of ``h`` and completes the norm in its first product.
 ``fusable``           (norms) the norm is gain * x / sqrt(mean x^2 + eps) and nothing else.
 Parts without these attributes are never asked; a block falls back to the norm kernel.
+
+A feed-forward beside its mixer
+-------------------------------
+``in_two_steps``      (feed-forwards) ``forward`` is ``second_step(step, first_step(step, h), residual, next_norm)``,
+                      and the first step does not touch the residual: a block whose mixer and feed-forward read the
+                      same rows may run it on a stream of its own while the mixer runs.
 """
 from __future__ import annotations
 
@@ -110,6 +116,7 @@ class Part:
     fuses_next_norm = False
     takes_normed_input = False
     fusable = False
+    in_two_steps = False
     can_overwrite = False      # mixers and feed-forwards: ``forward(..., accumulate=False)`` writes instead of adding
 
     def __init__(self, spec: Any, dtype: torch.dtype, device: torch.device):

@@ -363,7 +363,8 @@ class SharedNormBlock(Part):
     """One norm whose rows the mixer and the feed-forward both read: with h = norm(x), x += mixer(h) + ff(h).
 
     The two sublayers add into the float32 residual one after the other; neither reads what the other wrote, so the
-    sum is the arrangement's.  In steps of few tokens the norm rides on the products around it, where the parts can.  A layer whose spec has no feed-forward ends after the mixer.  ``spec.ffn_norm`` is not
+    sum is the arrangement's.  In steps of few tokens the norm rides on the products around it, where the parts can, and the
+    feed-forward's first product runs beside the mixer.  A layer whose spec has no feed-forward ends after the mixer.  ``spec.ffn_norm`` is not
     used (it is None)."""
 
     def __init__(self, spec: LayerSpec, dtype: torch.dtype, device: torch.device):
@@ -424,11 +425,21 @@ class SharedNormBlock(Part):
                 return self.mixer.forward(step, io, h, x, next_norm=next_norm)
             self.mixer.forward(step, io, h, x)
             return None
+        if self.ffn.in_two_steps and x.shape[0] <= self.BESIDE_ROWS:
+            # few rows: the mixer is a chain of small kernels that wait for one another, the feed-forward's first product
+            # streams weights; it does so on a stream of its own meanwhile
+            with kernels.beside() as join:
+                act = self.ffn.first_step(step, h)
+            self.mixer.forward(step, io, h, x)
+            join()
+            return self.ffn.second_step(step, act, x, next_norm if self.ffn.fuses_next_norm else None)
         self.mixer.forward(step, io, h, x)
         if self.ffn.fuses_next_norm and next_norm is not None:
             return self.ffn.forward(step, h, x, next_norm=next_norm)
         self.ffn.forward(step, h, x)
         return None
+
+    BESIDE_ROWS = 64
 
 
 register_block("shared_norm", SharedNormBlock)

@@ -248,6 +248,12 @@ class CappedAttention(Part):
                 and not self.values_from_keys and self.distance_bias is None
                 and float(getattr(self.position, "amplitude", 1.0)) == 1.0)
 
+    def _normed_flat(self) -> bool:
+        """A weighted norm of the heads and no rotation stand before the scores: what the decode kernel that writes the
+        cache itself does as well."""
+        return (self.norm_kind == "head_first" and self.position.rotary_table() is None and not self.conv
+                and self.value_mix is None and not self.gated and self.chunk is None and self.keep_first == 0)
+
     fuses_next_norm = True
 
     def _close(self, step, out: torch.Tensor, residual: torch.Tensor, accumulate: bool, next_norm):
@@ -276,6 +282,11 @@ class CappedAttention(Part):
         out = step.ws.buf("attn_out", (T, H * P), self.dtype)
         if self.conv and self._plain() and kernels.attention_with_rope(step, proj, out, H, G, P, self.scale, self.window, io,
                                                                        inv_freq, rot, io.writes_cache):
+            return self._close(step, out, residual, accumulate, next_norm)
+        if self._normed_flat() and kernels.attention_with_rope(
+                step, proj, out, H, G, P, self.scale, self.window, io, None, 0, io.writes_cache,
+                norm=(self.dim, self.norm_eps, self.q_norm_w, self.k_norm_w), values_from_keys=self.values_from_keys,
+                sinks=self.sinks, slopes=self.slopes, softcap=self.softcap):
             return self._close(step, out, residual, accumulate, next_norm)
         k_pages, v_pages = (io.k_pages, io.v_pages) if io.writes_cache else (None, None)
         if self.norm_kind == "whole" or self.value_mix is not None:

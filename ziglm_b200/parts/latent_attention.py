@@ -54,7 +54,7 @@ class LatentAttention(Part):
             raise ValueError(f"latent_attention: output gate {self.gate!r} is not known (sigmoid)")
         self.window = None if spec.window is None else int(spec.window)
         self.has_sink = bool(o.get("sink"))
-        self.kept = self.kept_size(self.rot_dim + self.kv_rank, dtype)
+        self.kept = self.kept_size(self.rot_dim + self.kv_rank, dtype, float(o.get("pad_to_fast", 1.0)))
         if self.kept > 512:
             raise ValueError(f"latent_attention: a key/value latent of {self.kv_rank} elements beside {self.rot_dim} "
                              "rotated ones is not supported (at most 512 together)")
@@ -77,14 +77,14 @@ class LatentAttention(Part):
         self.uv: Optional[torch.Tensor] = None    # [H, V, kept]
 
     @staticmethod
-    def kept_size(size: int, dtype: torch.dtype) -> int:
+    def kept_size(size: int, dtype: torch.dtype, most: float = 1.0) -> int:
         """The size a position's vector is kept with: a multiple of 8; in bfloat16 the next size the tensor-core attention
-        kernels take (64, 128) when that is at most a third more.  What lies behind the vector is zero: it adds nothing to
-        a score and its part of the result is not read."""
+        kernels take (64, 128) when that is at most ``most`` times as much (the option ``pad_to_fast``).  What lies behind
+        the vector is zero: it adds nothing to a score and its part of the result is not read."""
         kept = -(-size // 8) * 8
         if dtype == torch.bfloat16:
             for fast in (64, 128):
-                if kept <= fast and fast * 3 <= kept * 4:
+                if kept <= fast <= kept * most:
                     return fast
         return kept
 

@@ -75,12 +75,17 @@ class GatedMLP(Part):
     fuses_next_norm = True
     takes_normed_input = True
     can_overwrite = True
+    in_two_steps = True
 
     def forward(self, step, h, residual: torch.Tensor, next_norm=None, accumulate: bool = True):
         """``h``: the normalised rows or a half-done norm (:class:`NormedInput`).  With ``next_norm`` the down
         projection may do the first half of that norm; the result is then its :class:`NormedInput`.
         ``accumulate=False``: the result overwrites ``residual`` (a branch buffer) instead of adding to it."""
-        T = residual.shape[0]
+        return self.second_step(step, self.first_step(step, h), residual, next_norm, accumulate)
+
+    def first_step(self, step, h) -> torch.Tensor:
+        """act(gate) * up of the rows ``h``: what does not touch the residual."""
+        T = step.n_tokens
         act = step.ws.buf("ffn_act", (T, self.intermediate), self.dtype)
         normed = isinstance(h, NormedInput)
         rows = h.hb if normed else h
@@ -96,6 +101,9 @@ class GatedMLP(Part):
             self.gate_up(h, gu)
             kernels.gated_act(gu, act, self.spec.activation, interleaved=self.interleaved, limit=self.limit,
                               slope=self.slope)
+        return act
+
+    def second_step(self, step, act: torch.Tensor, residual: torch.Tensor, next_norm=None, accumulate: bool = True):
         if not accumulate:
             self.down(act, residual)
             return None
