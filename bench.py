@@ -1369,6 +1369,15 @@ def run_lilulix(args):
                                    (zero, slopes, "attention with sinks and a distance bias", "attention, every key")):
             ms = timed(lambda: kernels.attention(step, qkv, att_out, H, G, hd, scale, None, io, sinks=sk, slopes=sl))
             report(f"{what}, {tag}", like, ms, att_bytes, att_flops)
+        if decode:
+            # what a decode step launches: the new key and value are made and stored by the attention kernel itself
+            ms = timed(lambda: kernels.attention_with_rope(step, qkv, att_out, H, G, hd, scale, None, io, inv_freq, hd, True))
+            report(f"rotation + cache write + attention in one kernel, {tag}", "-", ms, att_bytes, att_flops)
+            ms = timed(lambda: kernels.attention_with_rope(step, qk, att_out, H, G, hd, scale, None, io, None, 0, True,
+                                                           norm=(hd, 1e-6, wq, wk), values_from_keys=True, sinks=zero,
+                                                           slopes=slopes))
+            report(f"norm of heads + cache write + attention with sinks and a distance bias in one kernel, {tag}",
+                   "rotation + cache write + attention in one kernel", ms, att_bytes, att_flops)
         del k_pages, v_pages
         # the latent's preparation and its attention over one shared head
         K = LC + LR

@@ -85,10 +85,10 @@ class GatedMLP(Part):
 
     def first_step(self, step, h) -> torch.Tensor:
         """act(gate) * up of the rows ``h``: what does not touch the residual."""
-        T = step.n_tokens
-        act = step.ws.buf("ffn_act", (T, self.intermediate), self.dtype)
         normed = isinstance(h, NormedInput)
         rows = h.hb if normed else h
+        T = rows.shape[0]
+        act = step.ws.buf("ffn_act", (T, self.intermediate), self.dtype)
         if self.interleaved and self.spec.activation == "swish_clamped" and not normed:
             fused = kernels.gemm_tc_swish_clamped(rows, self.gate_up.weight, act, self.limit, self.slope,
                                                   bias=self.gate_up.bias)
